@@ -381,6 +381,93 @@ tb_status tb_decoder_create(tb_decoder** out, const tb_model_config* cfg,
                             const float* lm_head_s, tb_space weight_space);
 void tb_decoder_destroy(tb_decoder* dec);
 
+/* ------------------------------------------------------------------------
+ * A decoder described layer by layer (no counterpart in the reference).  It is
+ * a tb_decoder like the others: every tb_decoder_* call below applies unless
+ * its comment says otherwise.  Weights are bfloat16 (the raw 16 bits) in the
+ * layout [out, in]; NULL leaves an optional part out.
+ *
+ *   x = embed[token] * embed_scale (+ pos_table[position])
+ *   per layer:  x += norm1_after(mixer(c(norm1(x))));  x += norm2_after(mlp(c(norm2(x))))
+ *   logits = embed final_norm(x)
+ *
+ * norms are RMS norms with norm_eps inside the root (a missing *_after norm
+ * adds the sublayer's output as it is); c(h) = h + causal convolution of h over
+ * conv_taps positions per channel (conv weights [hidden, conv_taps], the last
+ * tap meets the current position).
+ * Attention: q/k norm over the whole projection, score_scale, no rotation;
+ * position i sees j <= i with i - j < mask_window or j < mask_keep_first;
+ * softmax; the heads' weights are mixed by talk [heads, heads].
+ * Feed-forward: down(a N(z) + b N(z^2) + c N(z^3) + e), z = up h, N dividing by
+ * the root mean square over the features, act = {a, b, c, e}.
+ *
+ * State.  Per layer a KV cache (behind a window a ring of about window +
+ * prefill_rows positions, the kept first positions apart) and per sublayer the
+ * last inputs of the convolution.  A sequence must be fed gap-free; it may be
+ * continued from an earlier position than its last one (speculation) by up to
+ * a little over 100 positions, or from position 0; anything else fails with
+ * TB_ERR_ARG. */
+enum { TB_PRECISION_BF16 = 0, TB_PRECISION_F32 = 1 };
+enum { TB_MIXER_ATTENTION = 0 };
+enum { TB_MLP_NONE = 0, TB_MLP_POLYNORM = 1 };
+typedef struct tb_layered_config {
+  int64_t vocab_size;
+  int64_t hidden_size;
+  int32_t num_layers;
+  int32_t conv_taps;     /* 0 or 1: no neighbours */
+  float norm_eps;
+  float embed_scale;
+  int64_t max_seq_len;   /* also the rows of pos_table */
+  int32_t max_batch;     /* sequences; 0 means 1 */
+  int32_t prefill_rows;  /* positions of one sequence per step; 0 means 512 */
+  int32_t precision;     /* TB_PRECISION_*: products in bf16 with fp32 sums, or everything in fp32 */
+  int32_t flags;         /* TB_DECODER_NO_GRAPH, TB_DECODER_NO_PDL */
+} tb_layered_config;
+typedef struct tb_layered_layer {
+  int32_t mixer;
+  int32_t mlp;
+  int32_t weights_of;    /* use that layer's tensors (sizes must agree); -1: its own */
+  int32_t num_heads;
+  int32_t num_kv_heads;
+  int32_t head_dim;
+  int32_t value_dim;
+  int32_t mask_window;   /* 0: none */
+  int32_t mask_keep_first;
+  float score_scale;
+  int64_t ff;
+  const uint16_t* norm1;
+  const uint16_t* norm1_after;
+  const uint16_t* norm2;
+  const uint16_t* norm2_after;
+  const uint16_t* conv1;
+  const uint16_t* conv2;
+  const uint16_t* q_w;
+  const uint16_t* q_b;
+  const uint16_t* k_w;
+  const uint16_t* k_b;
+  const uint16_t* v_w;
+  const uint16_t* v_b;
+  const uint16_t* q_norm;
+  const uint16_t* k_norm;
+  const uint16_t* talk;
+  const uint16_t* o_w;
+  const uint16_t* o_b;
+  const uint16_t* up_w;
+  const uint16_t* down_w;
+  const uint16_t* act;
+} tb_layered_layer;
+/* embed [vocab, hidden], pos_table [max_seq_len, hidden] or NULL, final_norm [hidden]. */
+tb_status tb_decoder_create_layered(tb_decoder** out, const tb_layered_config* cfg, const tb_layered_layer* layers,
+                                    const uint16_t* embed, const uint16_t* pos_table, const uint16_t* final_norm,
+                                    tb_space weight_space);
+/* The next n tokens of sequence `seq` at positions start_offset.. in as few steps as the decoder's rows
+ * allow; logits_host [n_want, vocab] receives the logits at the places want[i] (indices into tokens, any
+ * order).  With an INT4 decoder seq must be 0. */
+tb_status tb_decoder_extend(tb_decoder* dec, int32_t seq, int64_t start_offset, const int64_t* tokens, int64_t n,
+                            const int64_t* want, int64_t n_want, float* logits_host);
+/* Gives back what sequence `seq` holds; it starts again at position 0. */
+tb_status tb_decoder_reset_sequence(tb_decoder* dec, int32_t seq);
+
 /* step(token_id, offset) -> logits, src/llm/decoder.rs:538-541 / decode_step
  * :729-750.  logits_host [vocab] may be NULL (logits stay on the device; read
  * them with tb_decoder_get_logits).  An out-of-range token or offset yields
@@ -476,7 +563,8 @@ tb_status tb_decoder_speculative_accept(tb_decoder* dec, int64_t offset, const i
 /* Layer-0 intermediates of the last step by name, like debug_step_stages,
  * src/wgpu/profiler.rs:75: "embed", "normed", "qkv", "attn", "x_attn", "h",
  * "x_out".  Only recorded when the decoder was created with TB_DECODER_NO_GRAPH.
- * Writes up to cap floats (sequence 0); *n = element count of the stage. */
+ * Writes up to cap floats (sequence 0); *n = element count of the stage.  A layered decoder records
+ * "layer0", "layer1", ...: the residual stream after that layer for every row of the last step. */
 tb_status tb_decoder_debug_stage(tb_decoder* dec, const char* name, float* out_host, int64_t cap,
                                  int64_t* n);
 /* profile_step_breakdown, src/wgpu/profiler.rs:14-73: CUDA-event milliseconds of

@@ -80,6 +80,60 @@ pub struct tb_model_config {
     pub flags: i32,
 }
 
+/// A decoder described layer by layer (no counterpart in the reference).
+#[repr(C)]
+#[derive(Clone, Copy, Debug)]
+pub struct tb_layered_config {
+    pub vocab_size: i64,
+    pub hidden_size: i64,
+    pub num_layers: i32,
+    pub conv_taps: i32,
+    pub norm_eps: f32,
+    pub embed_scale: f32,
+    pub max_seq_len: i64,
+    pub max_batch: i32,
+    pub prefill_rows: i32,
+    pub precision: i32,
+    pub flags: i32,
+}
+
+/// One of its layers; null pointers leave optional parts out.
+#[repr(C)]
+#[derive(Clone, Copy, Debug)]
+pub struct tb_layered_layer {
+    pub mixer: i32,
+    pub mlp: i32,
+    pub weights_of: i32,
+    pub num_heads: i32,
+    pub num_kv_heads: i32,
+    pub head_dim: i32,
+    pub value_dim: i32,
+    pub mask_window: i32,
+    pub mask_keep_first: i32,
+    pub score_scale: f32,
+    pub ff: i64,
+    pub norm1: *const u16,
+    pub norm1_after: *const u16,
+    pub norm2: *const u16,
+    pub norm2_after: *const u16,
+    pub conv1: *const u16,
+    pub conv2: *const u16,
+    pub q_w: *const u16,
+    pub q_b: *const u16,
+    pub k_w: *const u16,
+    pub k_b: *const u16,
+    pub v_w: *const u16,
+    pub v_b: *const u16,
+    pub q_norm: *const u16,
+    pub k_norm: *const u16,
+    pub talk: *const u16,
+    pub o_w: *const u16,
+    pub o_b: *const u16,
+    pub up_w: *const u16,
+    pub down_w: *const u16,
+    pub act: *const u16,
+}
+
 /// Per-layer weights in the capsule order of `create_rust_qwen_decoder`.
 #[repr(C)]
 #[derive(Clone, Copy, Debug)]
@@ -165,6 +219,9 @@ extern "C" {
     pub fn tb_fused_attention_step(qkv: *mut tb_linear, o: *mut tb_linear, x: *const f32, k_cache: *mut f32, v_cache: *mut f32, cos_p: *const f32, sin_p: *const f32, offset: i64, num_heads: i32, num_kv_heads: i32, head_dim: i32, max_seq_len: i64, out: *mut f32, io_space: tb_space, stream: *mut c_void) -> tb_status;
     pub fn tb_fused_transformer_layer_step(x: *mut f32, w: *const tb_layer_step_weights, k_cache: *mut f32, v_cache: *mut f32, cos_p: *const f32, sin_p: *const f32, offset: i64, hidden_size: i64, intermediate_size: i64, num_heads: i32, num_kv_heads: i32, head_dim: i32, max_seq_len: i64, group_size: i32, eps: f32, io_space: tb_space, stream: *mut c_void) -> tb_status;
     pub fn tb_decoder_create(out: *mut *mut tb_decoder, cfg: *const tb_model_config, embed_tokens: *const f32, layers: *const tb_layer_weights, final_norm_w: *const f32, lm_head_w: *const u8, lm_head_s: *const f32, weight_space: tb_space) -> tb_status;
+    pub fn tb_decoder_create_layered(out: *mut *mut tb_decoder, cfg: *const tb_layered_config, layers: *const tb_layered_layer, embed: *const u16, pos_table: *const u16, final_norm: *const u16, weight_space: tb_space) -> tb_status;
+    pub fn tb_decoder_extend(dec: *mut tb_decoder, seq: i32, start_offset: i64, tokens: *const i64, n: i64, want: *const i64, n_want: i64, logits_host: *mut f32) -> tb_status;
+    pub fn tb_decoder_reset_sequence(dec: *mut tb_decoder, seq: i32) -> tb_status;
     pub fn tb_decoder_destroy(dec: *mut tb_decoder);
     pub fn tb_decoder_step(dec: *mut tb_decoder, token_id: i64, offset: i64, logits_host: *mut f32) -> tb_status;
     pub fn tb_decoder_step_batch(dec: *mut tb_decoder, token_ids: *const i64, offsets: *const i64, batch: i32, logits_host: *mut f32) -> tb_status;

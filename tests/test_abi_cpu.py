@@ -53,7 +53,7 @@ def test_rust_sys_crate_declares_exactly_the_header(tb):
     assert set(c_fns) == set(r_fns), (sorted(set(c_fns) - set(r_fns)), sorted(set(r_fns) - set(c_fns)))
     assert c_fns == r_fns, {k: (c_fns[k], r_fns[k]) for k in c_fns if c_fns[k] != r_fns[k]}
     # struct fields, in order
-    for name in ("tb_model_config", "tb_layer_weights", "tb_layer_step_weights"):
+    for name in ("tb_model_config", "tb_layer_weights", "tb_layer_step_weights", "tb_layered_config", "tb_layered_layer"):
         c_body = re.search(r"typedef struct %s \{(.*?)\} %s;" % (name, name), hdr, flags=re.S).group(1)
         c_fields = re.findall(r"(\w+)\s*;", c_body)
         r_body = re.search(r"pub struct %s \{(.*?)\n\}" % name, rs_code, flags=re.S).group(1)

@@ -39,6 +39,31 @@ class LayerWeights(C.Structure):
         "up_s", "down_w", "down_s", "qkv_b")]
 
 
+TB_PRECISION = {"bfloat16": 0, "float32": 1}
+TB_MIXER_ATTENTION = 0
+TB_MLP_NONE, TB_MLP_POLYNORM = 0, 1
+
+
+class LayeredConfig(C.Structure):
+    _fields_ = [
+        ("vocab_size", C.c_int64), ("hidden_size", C.c_int64), ("num_layers", C.c_int32), ("conv_taps", C.c_int32),
+        ("norm_eps", C.c_float), ("embed_scale", C.c_float), ("max_seq_len", C.c_int64), ("max_batch", C.c_int32),
+        ("prefill_rows", C.c_int32), ("precision", C.c_int32), ("flags", C.c_int32),
+    ]
+
+
+LAYERED_TENSORS = ("norm1", "norm1_after", "norm2", "norm2_after", "conv1", "conv2", "q_w", "q_b", "k_w", "k_b", "v_w", "v_b",
+                   "q_norm", "k_norm", "talk", "o_w", "o_b", "up_w", "down_w", "act")
+
+
+class LayeredLayer(C.Structure):
+    _fields_ = [
+        ("mixer", C.c_int32), ("mlp", C.c_int32), ("weights_of", C.c_int32), ("num_heads", C.c_int32), ("num_kv_heads", C.c_int32),
+        ("head_dim", C.c_int32), ("value_dim", C.c_int32), ("mask_window", C.c_int32), ("mask_keep_first", C.c_int32),
+        ("score_scale", C.c_float), ("ff", C.c_int64),
+    ] + [(k, C.c_void_p) for k in LAYERED_TENSORS]
+
+
 class LayerStepWeights(C.Structure):
     _fields_ = [(k, C.c_void_p) for k in (
         "input_norm_w", "qkv_w", "qkv_s", "qkv_b", "o_w", "o_s", "o_b", "post_norm_w", "gate_w", "gate_s", "gate_b",
@@ -89,6 +114,9 @@ SIGNATURES = {
     "tb_fused_attention_step": (_i32, [_p, _p, _p, _p, _p, _p, _p, _i64, _i32, _i32, _i32, _i64, _p, _i32, _p]),
     "tb_fused_transformer_layer_step": (_i32, [_p, _p, _p, _p, _p, _p, _i64, _i64, _i64, _i32, _i32, _i32, _i64, _i32, _f32, _i32, _p]),
     "tb_decoder_create": (_i32, [_PP, C.POINTER(ModelConfig), _p, _p, _p, _p, _p, _i32]),
+    "tb_decoder_create_layered": (_i32, [_PP, C.POINTER(LayeredConfig), _p, _p, _p, _p, _i32]),
+    "tb_decoder_extend": (_i32, [_p, _i32, _i64, _p, _i64, _p, _i64, _p]),
+    "tb_decoder_reset_sequence": (_i32, [_p, _i32]),
     "tb_decoder_destroy": (None, [_p]),
     "tb_decoder_step": (_i32, [_p, _i64, _i64, _p]),
     "tb_decoder_step_batch": (_i32, [_p, _p, _p, _i32, _p]),
@@ -124,6 +152,13 @@ SIGNATURES = {
 }
 
 _lib = None
+
+
+def select(path: str) -> None:
+    """Uses the library at ``path`` (see ``build.ensure``); before the first call only."""
+    global LIB_PATH
+    if _lib is None and not os.environ.get("TORCHBURN_B200_LIB"):
+        LIB_PATH = path
 
 
 def lib():

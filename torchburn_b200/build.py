@@ -1,13 +1,18 @@
 """Builds libtorchburn_b200.so (sm_100a) from csrc/ with nvcc.
 
-    python -m torchburn_b200.build [--force] [--verbose]
+    python -m torchburn_b200.build [--force] [--verbose] [--profile full|dense]
 
 The library is written in-tree (torchburn_b200/lib/); it is the only compute
 path of the package - nothing falls back to the CPU when it is missing.
+
+Profile "full" (the default) is the whole library.  Profile "dense" leaves the
+INT4 kernels out (its INT4 entry points answer TB_ERR_UNSUPPORTED) and is what a
+layered model needs; ``ensure`` builds it only where no full library is at hand.
 """
 from __future__ import annotations
 
 import concurrent.futures as cf
+import fcntl
 import os
 import shutil
 import subprocess
@@ -17,6 +22,9 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "lib", "obj")
 LIB = os.path.join(HERE, "lib", "libtorchburn_b200.so")
+PROFILES = {"full": LIB, "dense": os.path.join(HERE, "lib", "libtorchburn_b200_dense.so")}
+INT4_SOURCES = ("w4_step.cu", "w4_stream.cu", "w4_gemv.cu", "w4_mma.cu", "w4_tc5.cu", "attention.cu")
+INT4_ABSENT = "w4_absent.cpp"
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -31,8 +39,9 @@ def _nvcc() -> str:
     raise RuntimeError("nvcc not found: the sm_100a library cannot be built")
 
 
-def sources():
-    return sorted(f for f in os.listdir(CSRC) if f.endswith((".cu", ".cpp")))
+def sources(profile: str = "full"):
+    drop = (INT4_ABSENT,) if profile == "full" else INT4_SOURCES
+    return sorted(f for f in os.listdir(CSRC) if f.endswith((".cu", ".cpp")) and f not in drop)
 
 
 def _newest_header() -> float:
@@ -41,13 +50,36 @@ def _newest_header() -> float:
     return max(os.path.getmtime(h) for h in hdrs)
 
 
-def build(force: bool = False, verbose: bool = False) -> str:
+def up_to_date(profile: str = "full") -> bool:
+    lib = PROFILES[profile]
+    if not os.path.exists(lib):
+        return False
+    newest = max(_newest_header(), *(os.path.getmtime(os.path.join(CSRC, f)) for f in sources(profile)))
+    return os.path.getmtime(lib) >= newest
+
+
+def ensure(profile: str) -> str:
+    """The library a model of this profile runs on: the full one if it is built, else the profile's own,
+    compiled now if need be."""
+    if up_to_date("full"):
+        return PROFILES["full"]
+    return PROFILES[profile] if up_to_date(profile) else build(profile=profile)
+
+
+def build(force: bool = False, verbose: bool = False, profile: str = "full") -> str:
     os.makedirs(OBJ, exist_ok=True)
+    with open(os.path.join(HERE, "lib", ".lock"), "w") as lock:   # two processes of a fresh checkout
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return _build(force, verbose, profile)
+
+
+def _build(force: bool, verbose: bool, profile: str) -> str:
+    LIB = PROFILES[profile]
     nvcc = _nvcc()
     hdr_time = _newest_header()
     jobs = []
     objs = []
-    for src in sources():
+    for src in sources(profile):
         sp = os.path.join(CSRC, src)
         op = os.path.join(OBJ, os.path.splitext(src)[0] + ".o")
         objs.append(op)
@@ -79,5 +111,6 @@ def build(force: bool = False, verbose: bool = False) -> str:
 
 
 if __name__ == "__main__":
-    path = build(force="--force" in sys.argv, verbose="--verbose" in sys.argv)
+    prof = sys.argv[sys.argv.index("--profile") + 1] if "--profile" in sys.argv else "full"
+    path = build(force="--force" in sys.argv, verbose="--verbose" in sys.argv, profile=prof)
     print(path)

@@ -17,6 +17,7 @@
 #include <new>
 #include <vector>
 
+#include "layered.cuh"
 #include "tb_common.cuh"
 #include "tp.cuh"
 
@@ -109,6 +110,12 @@ struct tb_decoder {
   int launches_per_step = 0;
   TpState* tpst = nullptr;
   std::vector<float> host_logits;  // sampling on the host
+  // A model described layer by layer (layered.cu) instead of the INT4 weights and caches above.
+  LayeredModel* lay = nullptr;
+  int32_t *d_slots = nullptr, *d_row_map = nullptr;
+  int logit_rows = 1;                        // rows of `logits`
+  int debug_rows = 0;                        // rows of the last step (its snapshots)
+  std::vector<int64_t> seq_len, seq_high;    // per sequence: next position, one past the furthest position its rings have held
 };
 
 namespace {
@@ -146,6 +153,14 @@ size_t kv_layer_stride(const tb_decoder* d) { return (size_t)d->B * d->nkv_l * d
 tb_status enqueue_step(tb_decoder* d, int b, bool debug, cudaEvent_t before_lm_head = nullptr) {
   cudaStream_t st = d->stream;
   const bool pdl = d->pdl;
+  if (d->lay) {
+    LayeredStep s;
+    s.r.tokens = d->d_tokens; s.r.slots = d->d_slots; s.r.offsets = d->d_offsets; s.r.rows = b;
+    s.logit_rows = b; s.logits = d->logits; s.pdl = pdl && before_lm_head == nullptr; s.snapshots = debug;
+    s.before_lm_head = before_lm_head;
+    d->debug_rows = b;
+    return layered_enqueue(d->lay, s, st, &d->launches_per_step);
+  }
   const int pm = d->pdl_mask;
   int launches = 0;
   if (d->fused_step && b == 1 && !debug && before_lm_head == nullptr) {
@@ -445,7 +460,41 @@ void note_kv(tb_decoder* d, int64_t token, int64_t offset) {
 
 int32_t clamp_i32(int64_t v) { return v < -1 ? -1 : (v > 0x7ffffff0 ? 0x7ffffff0 : (int32_t)v); }
 
+// Can sequence `seq` of a layered decoder go on at `start`?  Its rings hold a window and some room to go back,
+// not every position; and the convolution needs every position in front.
+tb_status check_sequence(const tb_decoder* d, int seq, int64_t start) {
+  if (!d->lay || start == 0) return TB_OK;
+  const int64_t len = d->seq_len[(size_t)seq], high = d->seq_high[(size_t)seq];
+  if (start > len) return fail(TB_ERR_ARG, "sequence %d has %lld positions and cannot go on at position %lld", seq, (long long)len, (long long)start);
+  if (high - start > layered_rollback(d->lay))
+    return fail(TB_ERR_ARG, "sequence %d was fed up to position %lld and cannot go back to %lld (at most %lld positions)", seq, (long long)high,
+                (long long)start, (long long)layered_rollback(d->lay));
+  return TB_OK;
+}
+void advance_sequence(tb_decoder* d, int seq, int64_t start, int64_t n) {
+  if (!d->lay) return;
+  const int64_t end = start + n;
+  int64_t &len = d->seq_len[(size_t)seq], &high = d->seq_high[(size_t)seq];
+  high = start == 0 || end > high ? end : high;
+  len = end;
+}
+
+tb_status feed_slots(tb_decoder* d, int b) {
+  if (!d->lay) return TB_OK;
+  for (int i = 0; i < b; ++i) d->h_io[2 * kMaxBatch + i] = i;
+  DEC_CUDA(d, cudaMemcpyAsync(d->d_slots, d->h_io + 2 * kMaxBatch, sizeof(int32_t) * b, cudaMemcpyHostToDevice, d->stream));
+  return TB_OK;
+}
+
 tb_status feed_and_step(tb_decoder* d, const int64_t* tokens, const int64_t* offsets, int b) {
+  if (d->lay) {
+    auto live = [&](int i) { return tokens[i] >= 0 && tokens[i] < d->V && offsets[i] >= 0 && offsets[i] < d->S; };
+    for (int i = 0; i < b; ++i)
+      if (live(i)) TB_TRY(check_sequence(d, i, offsets[i]));
+    for (int i = 0; i < b; ++i)
+      if (live(i)) advance_sequence(d, i, offsets[i], 1);
+    TB_TRY(feed_slots(d, b));
+  }
   for (int i = 0; i < b; ++i) {
     d->h_io[i] = clamp_i32(tokens[i]);
     d->h_io[kMaxBatch + i] = clamp_i32(offsets[i]);
@@ -457,12 +506,81 @@ tb_status feed_and_step(tb_decoder* d, const int64_t* tokens, const int64_t* off
   return run_step(d, b, false);
 }
 
+// The same for sequence `seq` of a layered decoder: up to its prefill rows per step, each token at its own
+// position, logits only for the wanted places (want == nullptr: of every position when rows_host is given;
+// the last position's logits always end up in the decoder's own buffer).
+tb_status run_positions_layered(tb_decoder* d, int seq, const int64_t* tokens, int64_t n, int64_t start_offset, const int64_t* want,
+                                int64_t n_want, float* rows_host) {
+  for (int64_t i = 0; i < n; ++i)
+    if (tokens[i] < 0 || tokens[i] >= d->V) return fail(TB_ERR_ARG, "token %lld outside the vocabulary", (long long)tokens[i]);
+  TB_TRY(check_sequence(d, seq, start_offset));
+  if (n > d->feed_cap) {
+    cudaFreeHost(d->h_feed);
+    d->h_feed = nullptr;
+    d->feed_cap = 0;
+    DEC_CUDA(d, cudaMallocHost((void**)&d->h_feed, sizeof(int32_t) * 4 * n));
+    d->feed_cap = n;
+  }
+  const bool all = want == nullptr && rows_host != nullptr;
+  std::vector<uint8_t> wanted((size_t)n, all ? 1 : 0);
+  for (int64_t i = 0; i < n_want; ++i) wanted[(size_t)want[i]] = 1;
+  wanted[(size_t)(n - 1)] = 1;
+  int32_t *tok = d->h_feed, *off = tok + n, *slot = off + n, *map = slot + n;
+  std::vector<int32_t> row_of((size_t)n, -1);
+  const int max_rows = layered_max_rows(d->lay);
+  const bool debug = (d->cfg.flags & TB_DECODER_NO_GRAPH) != 0;
+  int64_t i = 0;
+  while (i < n) {
+    int m = 0, lr = 0;
+    for (; i + m < n && m < max_rows; ++m) {
+      const int64_t j = i + m;
+      if (wanted[(size_t)j] && lr == d->logit_rows) break;
+      tok[j] = (int32_t)tokens[j];
+      off[j] = clamp_i32(start_offset + j);
+      slot[j] = seq;
+      map[j] = row_of[(size_t)j] = wanted[(size_t)j] ? lr++ : -1;
+    }
+    DEC_CUDA(d, cudaMemcpyAsync(d->d_tokens, tok + i, sizeof(int32_t) * m, cudaMemcpyHostToDevice, d->stream));
+    DEC_CUDA(d, cudaMemcpyAsync(d->d_offsets, off + i, sizeof(int32_t) * m, cudaMemcpyHostToDevice, d->stream));
+    DEC_CUDA(d, cudaMemcpyAsync(d->d_slots, slot + i, sizeof(int32_t) * m, cudaMemcpyHostToDevice, d->stream));
+    if (m == 1 && lr == 1) {
+      TB_TRY(run_step(d, 1, false));
+    } else {
+      DEC_CUDA(d, cudaMemcpyAsync(d->d_row_map, map + i, sizeof(int32_t) * m, cudaMemcpyHostToDevice, d->stream));
+      LayeredStep s;
+      s.r.tokens = d->d_tokens; s.r.slots = d->d_slots; s.r.offsets = d->d_offsets; s.r.rows = m;
+      s.one_sequence = true; s.last_pos = (int)(start_offset + i + m - 1);
+      s.row_map = d->d_row_map; s.logit_rows = lr; s.logits = d->logits; s.pdl = d->pdl; s.snapshots = debug;
+      d->debug_rows = m;
+      int launches = 0;
+      TB_TRY(layered_enqueue(d->lay, s, d->stream, &launches));
+    }
+    advance_sequence(d, seq, start_offset + i, m);
+    note_kv(d, tokens[i], start_offset + i + m - 1);
+    if (all) {
+      DEC_CUDA(d, cudaMemcpyAsync(rows_host + i * d->V, d->logits, sizeof(float) * (size_t)m * d->V, cudaMemcpyDeviceToHost, d->stream));
+    } else if (rows_host) {
+      for (int64_t w = 0; w < n_want; ++w)
+        if (want[w] >= i && want[w] < i + m)
+          DEC_CUDA(d, cudaMemcpyAsync(rows_host + w * d->V, d->logits + (size_t)row_of[(size_t)want[w]] * d->V, sizeof(float) * d->V, cudaMemcpyDeviceToHost, d->stream));
+    }
+    if (i + m == n && lr > 1)
+      DEC_CUDA(d, cudaMemcpyAsync(d->logits, d->logits + (size_t)(lr - 1) * d->V, sizeof(float) * d->V, cudaMemcpyDeviceToDevice, d->stream));
+    i += m;
+  }
+  d->last_batch = 1;
+  DEC_CUDA(d, cudaStreamSynchronize(d->stream));
+  return TB_OK;
+}
+
 // n consecutive positions of sequence 0, max_batch of them per step: the rows of a step are positions of the
 // ONE sequence (batched products, attention rows sharing sequence 0's cache, causal inside the block).  All
 // tokens and offsets are staged in pinned memory first, every step copying from its own part, so that the host
 // never rewrites words an earlier, still queued copy has yet to read.  rows_host (optional) receives the
 // logits of every position.  Afterwards the decoder's own logits are those of the last position.
-tb_status run_positions(tb_decoder* d, const int64_t* tokens, int64_t n, int64_t start_offset, float* rows_host) {
+tb_status run_positions(tb_decoder* d, const int64_t* tokens, int64_t n, int64_t start_offset, float* rows_host,
+                        const int64_t* want = nullptr, int64_t n_want = 0) {
+  if (d->lay) return run_positions_layered(d, 0, tokens, n, start_offset, want, n_want, rows_host);
   if (n > d->feed_cap) {
     cudaFreeHost(d->h_feed);
     d->h_feed = nullptr;
@@ -485,8 +603,11 @@ tb_status run_positions(tb_decoder* d, const int64_t* tokens, int64_t n, int64_t
     const tb_status s = run_step(d, m, false);
     d->verify_shared = false;
     TB_TRY(s);
-    if (rows_host)
+    if (rows_host && !want)
       DEC_CUDA(d, cudaMemcpyAsync(rows_host + i * d->V, d->logits, sizeof(float) * (size_t)m * d->V, cudaMemcpyDeviceToHost, d->stream));
+    for (int64_t w = 0; rows_host && w < n_want; ++w)
+      if (want[w] >= i && want[w] < i + m)
+        DEC_CUDA(d, cudaMemcpyAsync(rows_host + w * d->V, d->logits + (size_t)(want[w] - i) * d->V, sizeof(float) * d->V, cudaMemcpyDeviceToHost, d->stream));
     last_m = m;
     i += m;
   }
@@ -673,6 +794,65 @@ tb_status tb_decoder_create(tb_decoder** out, const tb_model_config* cfg,
   return TB_OK;
 }
 
+tb_status tb_decoder_create_layered(tb_decoder** out, const tb_layered_config* cfg, const tb_layered_layer* layers,
+                                    const uint16_t* embed, const uint16_t* pos_table, const uint16_t* final_norm, tb_space ws) {
+  if (!out) return fail(TB_ERR_ARG, "tb_decoder_create_layered: null out");
+  *out = nullptr;
+  if (!cfg || !layers || !embed || !final_norm) return fail(TB_ERR_ARG, "tb_decoder_create_layered: null argument");
+  tb_layered_config c = *cfg;
+  if (c.max_batch <= 0) c.max_batch = 1;
+  if (c.prefill_rows <= 0) c.prefill_rows = 512;
+  if (c.max_batch > kMaxBatch) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: max_batch %d (max %d)", c.max_batch, kMaxBatch);
+  if (c.prefill_rows > 8192) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: prefill_rows %d (max 8192)", c.prefill_rows);
+  tb_decoder* d = new (std::nothrow) tb_decoder();
+  if (!d) return fail(TB_ERR_OOM, "tb_decoder_create_layered: host allocation failed");
+  memset(&d->cfg, 0, sizeof(d->cfg));
+  d->cfg.vocab_size = c.vocab_size; d->cfg.hidden_size = c.hidden_size; d->cfg.num_layers = c.num_layers;
+  d->cfg.rms_norm_eps = c.norm_eps; d->cfg.max_seq_len = c.max_seq_len; d->cfg.max_batch = c.max_batch; d->cfg.flags = c.flags;
+  d->V = d->V_l = c.vocab_size; d->H = c.hidden_size; d->S = c.max_seq_len; d->L = c.num_layers; d->B = c.max_batch;
+  d->use_graph = !(c.flags & TB_DECODER_NO_GRAPH);
+  d->pdl = !(c.flags & TB_DECODER_NO_PDL);
+  auto fin = [&](tb_status st) -> tb_status {
+    tb_decoder_destroy(d);
+    return st;
+  };
+#define CR(expr) do { const tb_status _st = (expr); if (_st != TB_OK) return fin(_st); } while (0)
+#define CRC(expr) do { cudaError_t _e = (expr); if (_e != cudaSuccess) return fin(fail(_e == cudaErrorMemoryAllocation ? TB_ERR_OOM : TB_ERR_CUDA, "%s failed: %s", #expr, cudaGetErrorString(_e))); } while (0)
+  CR(layered_create(&d->lay, c, layers, embed, pos_table, final_norm, ws, (c.flags & TB_DECODER_NO_GRAPH) != 0));
+  cudaGetDevice(&d->device);
+  CRC(cudaStreamCreateWithFlags(&d->stream, cudaStreamNonBlocking));
+  d->seq_len.assign((size_t)d->B, 0);
+  d->seq_high.assign((size_t)d->B, 0);
+  d->logit_rows = kMaxBatch;
+  const size_t rows = (size_t)(layered_max_rows(d->lay) > kMaxBatch ? layered_max_rows(d->lay) : kMaxBatch);
+  CR(dalloc(&d->logits, (size_t)d->logit_rows * d->V));
+  CRC(cudaMemset(d->logits, 0, (size_t)d->logit_rows * d->V * sizeof(float)));
+  CR(dalloc(&d->d_tokens, rows));
+  CR(dalloc(&d->d_offsets, rows));
+  CR(dalloc(&d->d_slots, rows));
+  CR(dalloc(&d->d_row_map, rows));
+  CR(dalloc(&d->d_hist_pos, (size_t)1));
+  CRC(cudaMemset(d->d_hist_pos, 0, sizeof(int32_t)));
+  CRC(cudaMallocHost((void**)&d->h_io, sizeof(int32_t) * 3 * kMaxBatch));
+  CRC(cudaMalloc(&d->argmax_scratch, 16 * kMaxBatch));
+  CRC(cudaMemset(d->argmax_scratch, 0, 16 * kMaxBatch));
+  // warm-up with an out-of-range token, like tb_decoder_create
+  int64_t tok = -1, off = 0;
+  const bool g = d->use_graph;
+  const int flags = d->cfg.flags;
+  d->use_graph = false;
+  d->cfg.flags &= ~TB_DECODER_NO_GRAPH;
+  const tb_status s = feed_and_step(d, &tok, &off, 1);
+  d->cfg.flags = flags;
+  d->use_graph = g;
+  if (s != TB_OK) return fin(s);
+  CRC(cudaStreamSynchronize(d->stream));
+#undef CR
+#undef CRC
+  *out = d;
+  return TB_OK;
+}
+
 void tb_decoder_destroy(tb_decoder* d) {
   if (!d) return;
   if (d->stream) cudaStreamSynchronize(d->stream);
@@ -682,6 +862,8 @@ void tb_decoder_destroy(tb_decoder* d) {
     if (d->graphs_verify[i]) cudaGraphExecDestroy(d->graphs_verify[i]);
   }
   if (d->tpst) tp_destroy(d->tpst);
+  layered_destroy(d->lay);
+  cudaFree(d->d_slots); cudaFree(d->d_row_map);
   cudaFree(d->embed); cudaFree(d->final_norm_w); cudaFree(d->lm_w); cudaFree(d->lm_s);
   for (LayerDev& o : d->layers) {
     cudaFree(o.input_norm_w); cudaFree(o.qkv_w); cudaFree(o.qkv_s); cudaFree(o.o_w); cudaFree(o.o_s);
@@ -732,7 +914,7 @@ tb_status tb_decoder_prefill_tokens(tb_decoder* d, const int64_t* tokens, int64_
   if (!tokens || n < 0 || start_offset < 0) return fail(TB_ERR_ARG, "tb_decoder_prefill_tokens: bad arguments");
   if (start_offset + n > d->S)
     return fail(TB_ERR_ARG, "prefill %lld tokens at offset %lld exceeds max_seq_len %lld", (long long)n, (long long)start_offset, (long long)d->S);
-  if (d->B > 1 && n > 1) {
+  if (d->lay || (d->B > 1 && n > 1)) {
     // A decoder built for several rows takes max_batch positions of the prompt per step, like
     // tb_decoder_verify_tokens: one pass over the weights for every max_batch tokens instead of one per token
     // (the reference steps token by token, src/llm/decoder.rs:436-445; the cache rows and the last logits are
@@ -786,6 +968,32 @@ tb_status tb_decoder_verify_tokens(tb_decoder* d, int64_t start_offset, const in
   return run_positions(d, tokens, n, start_offset, logits_host);
 }
 
+tb_status tb_decoder_extend(tb_decoder* d, int32_t seq, int64_t start_offset, const int64_t* tokens, int64_t n,
+                            const int64_t* want, int64_t n_want, float* logits_host) {
+  TB_TRY(check_alive(d, "tb_decoder_extend"));
+  if (n == 0 && n_want == 0) return TB_OK;
+  if (!tokens || n <= 0 || start_offset < 0 || n_want < 0 || (n_want > 0 && (!want || !logits_host)))
+    return fail(TB_ERR_ARG, "tb_decoder_extend: bad arguments");
+  if (seq < 0 || seq >= d->B || (!d->lay && seq != 0)) return fail(TB_ERR_ARG, "tb_decoder_extend: sequence %d", seq);
+  if (start_offset + n > d->S)
+    return fail(TB_ERR_ARG, "extend %lld tokens at offset %lld exceeds max_seq_len %lld", (long long)n, (long long)start_offset, (long long)d->S);
+  for (int64_t i = 0; i < n_want; ++i)
+    if (want[i] < 0 || want[i] >= n) return fail(TB_ERR_ARG, "tb_decoder_extend: place %lld of %lld tokens", (long long)want[i], (long long)n);
+  const int64_t none = 0;
+  if (n_want == 0) want = &none;   // not "every position"
+  if (d->lay) return run_positions_layered(d, seq, tokens, n, start_offset, want, n_want, logits_host);
+  return run_positions(d, tokens, n, start_offset, logits_host, want, n_want);
+}
+
+tb_status tb_decoder_reset_sequence(tb_decoder* d, int32_t seq) {
+  TB_TRY(check_alive(d, "tb_decoder_reset_sequence"));
+  if (seq < 0 || seq >= d->B) return fail(TB_ERR_ARG, "tb_decoder_reset_sequence: sequence %d", seq);
+  // Nothing to clear: a sequence that starts at position 0 again reads only rows it has written since (INT4
+  // caches: rows in front of its offset; rings: positions of its own window; the convolution: zeros in front).
+  if (d->lay) d->seq_len[(size_t)seq] = d->seq_high[(size_t)seq] = 0;
+  return TB_OK;
+}
+
 tb_status tb_decoder_speculative_accept(tb_decoder* d, int64_t offset, const int64_t* draft_tokens, int64_t k,
                                         const float* draft_probs, float temperature, float top_p,
                                         uint64_t* rng_state, int64_t* accepted, int64_t* bonus) {
@@ -810,6 +1018,13 @@ tb_status tb_decoder_speculative_accept(tb_decoder* d, int64_t offset, const int
 
 tb_status tb_decoder_reset_kv_cache(tb_decoder* d) {
   TB_TRY(check_alive(d, "tb_decoder_reset_kv_cache"));
+  if (d->lay) {
+    DEC_CUDA(d, cudaStreamSynchronize(d->stream));
+    d->seq_len.assign((size_t)d->B, 0);
+    d->seq_high.assign((size_t)d->B, 0);
+    d->kv_used = 0;
+    return TB_OK;
+  }
   const int64_t used = d->kv_used < d->S ? d->kv_used : d->S;
   if (used == 0) return TB_OK;  // src/llm/decoder.rs:452-455
   const size_t pitch = (size_t)d->S * d->hd * sizeof(float);
@@ -826,6 +1041,7 @@ tb_status tb_decoder_copy_kv_cache_from(tb_decoder* d, const float* const* k, co
                                         int32_t num_given, int64_t seq_len, int64_t src_max_len,
                                         int32_t seq, tb_space space) {
   TB_TRY(check_alive(d, "tb_decoder_copy_kv_cache_from"));
+  if (d->lay) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: a layered decoder's state is more than its K and V rows; prefill instead");
   if (!k || !v || num_given < 0 || seq < 0 || seq >= d->B) return fail(TB_ERR_ARG, "tb_decoder_copy_kv_cache_from: bad arguments");
   if (seq_len < 0 || seq_len > d->S || seq_len > src_max_len) return fail(TB_ERR_ARG, "KV cache copy out of bounds");
   const int nl = num_given < d->L ? num_given : d->L;  // src/llm/decoder.rs:486
@@ -847,6 +1063,7 @@ tb_status tb_decoder_copy_kv_cache_from(tb_decoder* d, const float* const* k, co
 
 tb_status tb_decoder_read_kv_cache(tb_decoder* d, int32_t layer, int32_t seq, float* k_host, float* v_host) {
   TB_TRY(check_alive(d, "tb_decoder_read_kv_cache"));
+  if (d->lay) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: the caches of a layered decoder are rings of its own layout");
   if (layer < 0 || layer >= d->L || seq < 0 || seq >= d->B || !k_host || !v_host) return fail(TB_ERR_ARG, "tb_decoder_read_kv_cache: bad arguments");
   const size_t n = (size_t)d->nkv_l * d->S * d->hd;
   const size_t base = (size_t)layer * kv_layer_stride(d) + (size_t)seq * n;
@@ -874,6 +1091,8 @@ tb_status tb_decoder_generate_greedy(tb_decoder* d, int64_t first_token, int64_t
   if (n_new == 0) return TB_OK;
   if (!out_tokens || n_new < 0 || start_offset < 0) return fail(TB_ERR_ARG, "tb_decoder_generate_greedy: bad arguments");
   if (start_offset + n_new > d->S) return fail(TB_ERR_ARG, "generate exceeds max_seq_len");
+  if (d->lay && (first_token < 0 || first_token >= d->V)) return fail(TB_ERR_ARG, "token %lld outside the vocabulary", (long long)first_token);
+  TB_TRY(check_sequence(d, 0, start_offset));
   if (n_new > d->hist_cap) {
     // First use: room for the longest possible run (max_seq_len tokens), so that the graphs, which
     // hold this pointer, are never rebuilt in the middle of a generation.
@@ -891,7 +1110,9 @@ tb_status tb_decoder_generate_greedy(tb_decoder* d, int64_t first_token, int64_t
   d->h_io[kMaxBatch] = clamp_i32(start_offset);
   DEC_CUDA(d, cudaMemcpyAsync(d->d_tokens, d->h_io, sizeof(int32_t), cudaMemcpyHostToDevice, d->stream));
   DEC_CUDA(d, cudaMemcpyAsync(d->d_offsets, d->h_io + kMaxBatch, sizeof(int32_t), cudaMemcpyHostToDevice, d->stream));
+  TB_TRY(feed_slots(d, 1));
   DEC_CUDA(d, cudaMemsetAsync(d->d_hist_pos, 0, sizeof(int32_t), d->stream));
+  advance_sequence(d, 0, start_offset, n_new);
   d->last_batch = 1;
   for (int64_t i = 0; i < n_new; ++i) TB_TRY(run_step(d, 1, true));
   std::vector<int32_t> hist((size_t)n_new);
@@ -974,6 +1195,18 @@ tb_status tb_decoder_debug_stage(tb_decoder* d, const char* name, float* out_hos
     return fail(TB_ERR_UNSUPPORTED, "debug stages are recorded only by a decoder created with TB_DECODER_NO_GRAPH");
   const float* src = nullptr;
   int64_t cnt = 0;
+  if (d->lay) {
+    int64_t stride = 0;
+    src = strncmp(name, "layer", 5) == 0 && name[5] >= '0' && name[5] <= '9' ? layered_snapshot(d->lay, atoi(name + 5), &stride) : nullptr;
+    if (!src) return fail(TB_ERR_ARG, "unknown stage '%s'", name);
+    *n = (int64_t)d->debug_rows * d->H;
+    if (out_host && cap >= *n) {
+      DEC_CUDA(d, cudaMemcpy2DAsync(out_host, sizeof(float) * d->H, src, sizeof(float) * stride, sizeof(float) * d->H, d->debug_rows,
+                                    cudaMemcpyDeviceToHost, d->stream));
+      DEC_CUDA(d, cudaStreamSynchronize(d->stream));
+    }
+    return TB_OK;
+  }
   if (!strcmp(name, "embed")) { src = d->dbg_embed; cnt = d->H; }
   else if (!strcmp(name, "normed")) { src = d->dbg_normed; cnt = d->H; }
   else if (!strcmp(name, "qkv")) { src = d->dbg_qkv; cnt = d->tq_l; }
@@ -1000,6 +1233,13 @@ tb_status tb_decoder_step_timed(tb_decoder* d, int64_t token_id, int64_t offset,
   d->h_io[kMaxBatch] = clamp_i32(offset);
   note_kv(d, token_id, offset);
   d->last_batch = 1;
+  if (d->lay) {
+    if (token_id >= 0 && token_id < d->V && offset >= 0 && offset < d->S) {
+      TB_TRY(check_sequence(d, 0, offset));
+      advance_sequence(d, 0, offset, 1);
+    }
+    TB_TRY(feed_slots(d, 1));
+  }
   DEC_CUDA(d, cudaMemcpyAsync(d->d_tokens, d->h_io, sizeof(int32_t), cudaMemcpyHostToDevice, d->stream));
   DEC_CUDA(d, cudaMemcpyAsync(d->d_offsets, d->h_io + kMaxBatch, sizeof(int32_t), cudaMemcpyHostToDevice, d->stream));
   DEC_CUDA(d, cudaEventRecord(ev[0], d->stream));

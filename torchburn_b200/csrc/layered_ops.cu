@@ -1,0 +1,318 @@
+// Row kernels of the layered decoder, between the projections: residual + norms + the causal convolution
+// in front of a sublayer (glue), query/key norm with the cache append, and PolyNorm.  All arithmetic is
+// fp32; the results are written as the next projection's operand.
+//
+// A row is handled by a cluster of 1..8 CTAs (few rows: more CTAs, so that a decode row of several thousand
+// features is not one SM's work); block sums meet through distributed shared memory and are added in rank
+// order, so a result does not depend on timing.  The partial sums of a K-split projection are added here.
+#include <cooperative_groups.h>
+
+#include "dense.cuh"
+
+namespace cg = cooperative_groups;
+
+namespace tb {
+
+namespace {
+
+constexpr int kThreads = 256;
+
+// Sum over the cluster of N values per thread.  `slot` alternates 0, 1, 0, ... from call to call: a CTA that
+// has passed the barrier of call i has finished reading the slot of call i - 1.
+template <int N>
+struct ClusterSum {
+  float part[N][kThreads / 32];
+  float all[2][8][N];
+};
+template <int N>
+__device__ __forceinline__ void cluster_sum(ClusterSum<N>& s, int slot, int csize, int crank, float (&v)[N]) {
+#pragma unroll
+  for (int i = 0; i < N; ++i)
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v[i] += __shfl_xor_sync(0xffffffffu, v[i], o);
+  if ((threadIdx.x & 31) == 0)
+#pragma unroll
+    for (int i = 0; i < N; ++i) s.part[i][threadIdx.x >> 5] = v[i];
+  __syncthreads();
+  if (csize == 1) {
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      float t = 0.f;
+#pragma unroll
+      for (int w = 0; w < kThreads / 32; ++w) t += s.part[i][w];
+      v[i] = t;
+    }
+    __syncthreads();   // `part` may be rewritten
+    return;
+  }
+  cg::cluster_group cl = cg::this_cluster();
+  if (threadIdx.x < (unsigned)csize) {
+    ClusterSum<N>* peer = cl.map_shared_rank(&s, threadIdx.x);
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+      float t = 0.f;
+#pragma unroll
+      for (int w = 0; w < kThreads / 32; ++w) t += s.part[i][w];
+      peer->all[slot][crank][i] = t;
+    }
+  }
+  cl.sync();
+#pragma unroll
+  for (int i = 0; i < N; ++i) {
+    float t = 0.f;
+    for (int r = 0; r < csize; ++r) t += s.all[slot][r][i];
+    v[i] = t;
+  }
+}
+
+__device__ __forceinline__ float4 f4(float v) { return make_float4(v, v, v, v); }
+__device__ __forceinline__ float4 ld4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+__device__ __forceinline__ float dot4(float4 a) { return fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(a.z, a.z, a.w * a.w))); }
+__device__ __forceinline__ float4 mul4(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
+__device__ __forceinline__ float4 scale4(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
+__device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) {
+  return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w));
+}
+__device__ __forceinline__ float4 sum_partials(const PartialSums& y, int row, int col) {
+  const float* p = y.y + (size_t)row * y.ldy + col;
+  float4 v = ld4(p);
+  for (int s = 1; s < y.splits; ++s) v = add4(v, ld4(p + (size_t)s * y.split_stride));
+  return v;
+}
+
+// grid: (rows / rows_per * csize); rows_per consecutive rows per cluster, after up to taps - 1 rows of the same
+// sequence in front of them whose convolution inputs are computed again.
+template <bool BF16>
+__global__ void __launch_bounds__(kThreads) glue_kernel(const GlueArgs a, const int rows_per, const int e4) {
+  extern __shared__ float4 s_dyn[];        // [1 + taps][e4][kThreads]: x' of the row, then h of the last taps rows
+  __shared__ ClusterSum<1> s_sum;
+  const int tid = threadIdx.x;
+  const int csize = (int)cg::this_cluster().num_blocks();
+  const int crank = (int)cg::this_cluster().block_rank();
+  const int xs4 = a.xs >> 2, lane4 = crank * kThreads + tid, step4 = csize * kThreads;
+  const int r0 = a.row0 + ((int)blockIdx.x / csize) * rows_per;
+  const int r1 = min(a.r.rows, r0 + rows_per);
+  float4* s_x = s_dyn;
+  float4* s_h = s_dyn + (size_t)e4 * kThreads;
+  const int hist = e4 * kThreads;
+  if (csize > 1) cg::this_cluster().sync();   // every CTA of the cluster runs before its shared memory is written
+  grid_dep_launch();
+  grid_dep_wait();
+  const int taps = a.conv_w != nullptr ? a.taps : 1;
+  const bool emb = a.embed != nullptr;
+  int slot = 0;
+  const int32_t* posv = emb ? a.r.offsets : a.r.pos;   // the embedding kernel is the one that writes r.pos
+  auto same_run = [&](int q, int r) { return q >= 0 && a.r.slots[q] == a.r.slots[r] && posv[q] >= 0 && posv[q] == posv[r] - (r - q); };
+
+  for (int r = max(0, r0 - (taps - 1)); r < r1; ++r) {
+    if (r < r0 && !same_run(r, r0)) continue;
+    // ---- x' ----
+    int tok = 0, pos = posv[r];
+    bool live = pos >= 0;
+    if (emb) {
+      tok = a.r.tokens[r];
+      live = tok >= 0 && tok < a.vocab && pos >= 0 && pos < a.max_pos;
+      if (!live) pos = -1;
+      if (r >= r0 && tid == 0 && crank == 0) a.r.pos[r] = pos;
+    }
+    float inv = 1.f;
+    if (!emb && a.y.y != nullptr) {
+      float ss[1] = {0.f};
+      for (int e = 0, i = lane4; i < xs4; ++e, i += step4) {
+        float4 v = sum_partials(a.y, r, i * 4);
+        if (a.y_bias) v = add4(v, ld4(a.y_bias + i * 4));
+        s_x[e * kThreads + tid] = v;
+        ss[0] += dot4(v);
+      }
+      if (a.post_w) {
+        cluster_sum<1>(s_sum, slot, csize, crank, ss);
+        slot ^= 1;
+        inv = 1.0f / sqrtf(ss[0] / (float)a.width + a.eps);
+      }
+    }
+    float ss[1] = {0.f};
+    for (int e = 0, i = lane4; i < xs4; ++e, i += step4) {
+      float4 v = f4(0.f);
+      if (emb) {
+        if (live) {
+          const int k = i * 4;
+          // embedding row from the tile images of the tied output matrix
+          const unsigned char* t = static_cast<const unsigned char*>(a.embed->img) + ((size_t)(tok >> 7) * (a.embed->kp >> 6) + (k >> 6)) * 16384 +
+                                   (size_t)(tok & 127) * 128 + ((((k >> 3) & 7) ^ (tok & 7)) << 4) + ((k & 7) << 1);
+          const uint2 u = *reinterpret_cast<const uint2*>(t);
+          v = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
+          v = scale4(v, a.embed_scale);
+          if (a.pos_table) {
+            const __nv_bfloat16* pr = a.pos_table + (size_t)pos * a.width;
+            if (k < a.width) v.x += __bfloat162float(pr[k]);
+            if (k + 1 < a.width) v.y += __bfloat162float(pr[k + 1]);
+            if (k + 2 < a.width) v.z += __bfloat162float(pr[k + 2]);
+            if (k + 3 < a.width) v.w += __bfloat162float(pr[k + 3]);
+          }
+        }
+      } else {
+        v = ld4(a.x_in + (size_t)r * a.xs + i * 4);
+        if (a.y.y != nullptr) {
+          const float4 y = s_x[e * kThreads + tid];
+          v = a.post_w ? fma4(scale4(y, inv), ld4(a.post_w + i * 4), v) : add4(v, y);
+        }
+      }
+      s_x[e * kThreads + tid] = v;
+      ss[0] += dot4(v);
+      if (r >= r0 && a.x_out) *reinterpret_cast<float4*>(a.x_out + (size_t)r * a.xs + i * 4) = v;
+      if (r >= r0 && a.snapshot) *reinterpret_cast<float4*>(a.snapshot + (size_t)r * a.xs + i * 4) = v;
+    }
+    // ---- h = norm(x') ----
+    cluster_sum<1>(s_sum, slot, csize, crank, ss);
+    slot ^= 1;
+    inv = 1.0f / sqrtf(ss[0] / (float)a.width + a.eps);
+    const int orow = (a.row_map != nullptr && r >= r0) ? a.row_map[r] : r;
+    uint32_t in_step = 0;   // bit j: the input j positions back is a row of this step (else it is in the state)
+    for (int j = 1; j < taps; ++j) in_step |= same_run(r - j, r) ? 1u << j : 0u;
+    float4* h_cur = s_h + (size_t)(r % taps) * hist;
+    for (int e = 0, i = lane4; i < xs4; ++e, i += step4) {
+      const float4 h = mul4(scale4(s_x[e * kThreads + tid], inv), ld4(a.pre_w + i * 4));
+      h_cur[e * kThreads + tid] = h;
+      if (r < r0) continue;
+      if (a.write_state && pos >= 0)
+        *reinterpret_cast<float4*>(a.conv_state + ((size_t)a.r.slots[r] * a.ring + (pos & (a.ring - 1))) * a.xs + i * 4) = h;
+      if (a.out.data == nullptr || orow < 0) continue;
+      float4 o = h;
+      if (a.conv_w != nullptr && pos >= 0) {
+        for (int j = 0; j < taps && j <= pos; ++j) {   // tap taps - 1 - j meets the input j positions back
+          float4 hp = h;
+          if (j > 0) {
+            if ((in_step >> j) & 1u) hp = s_h[(size_t)((r - j) % taps) * hist + e * kThreads + tid];
+            else hp = ld4(a.conv_state + ((size_t)a.r.slots[r] * a.ring + ((pos - j) & (a.ring - 1))) * a.xs + i * 4);
+          }
+          o = fma4(ld4(a.conv_w + (size_t)(taps - 1 - j) * a.xs + i * 4), hp, o);
+        }
+      }
+      if (pos < 0) o = f4(0.f);
+      act_store4<BF16>(a.out, orow, i * 4, o);
+    }
+  }
+}
+
+// Query/key norm over the whole projection, biases, heads split and padded, k and v into the cache.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) qkv_prep_kernel(const QkvPrepArgs a) {
+  __shared__ ClusterSum<2> s_sum;
+  const int tid = threadIdx.x;
+  const int csize = (int)cg::this_cluster().num_blocks();
+  const int crank = (int)cg::this_cluster().block_rank();
+  const int r = (int)blockIdx.x / csize;
+  const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
+  const int first = crank * kThreads + tid, step = csize * kThreads;
+  if (csize > 1) cg::this_cluster().sync();
+  grid_dep_launch();
+  grid_dep_wait();
+  const int pos = a.r.pos[r];
+  auto value = [&](int col) {
+    const float* p = a.y.y + (size_t)r * a.y.ldy + col;
+    float v = p[0];
+    for (int s = 1; s < a.y.splits; ++s) v += p[(size_t)s * a.y.split_stride];
+    return a.bias ? v + a.bias[col] : v;
+  };
+  float ss[2] = {0.f, 0.f};
+  for (int i = first; i < nq; i += step) { const float v = value(a.q_off + i); ss[0] = fmaf(v, v, ss[0]); }
+  for (int i = first; i < nk; i += step) { const float v = value(a.k_off + i); ss[1] = fmaf(v, v, ss[1]); }
+  cluster_sum<2>(s_sum, 0, csize, crank, ss);
+  const float iq = a.q_norm ? 1.0f / sqrtf(ss[0] / (float)nq + a.eps) : 1.f;
+  const float ik = a.k_norm ? 1.0f / sqrtf(ss[1] / (float)nk + a.eps) : 1.f;
+  for (int i = first; i < nq; i += step) {
+    float v = value(a.q_off + i) * iq;
+    if (a.q_norm) v *= a.q_norm[i];
+    const size_t o = (size_t)r * a.heads * a.dpad + (size_t)(i / a.dim) * a.dpad + i % a.dim;
+    if (a.q) a.q[o] = v;
+    if (a.q16) a.q16[o] = __float2bfloat16_rn(v);
+  }
+  if (pos < 0) return;
+  const size_t crow = (size_t)a.r.slots[r] * a.geom.rows + a.geom.row_of(pos);
+  T* kc = static_cast<T*>(a.k_cache) + crow * (size_t)(a.kv_heads * a.dpad);
+  T* vc = static_cast<T*>(a.v_cache) + crow * (size_t)(a.kv_heads * a.vpad);
+  for (int i = first; i < nk; i += step) {
+    float v = value(a.k_off + i) * ik;
+    if (a.k_norm) v *= a.k_norm[i];
+    kc[(i / a.dim) * a.dpad + i % a.dim] = (T)v;
+  }
+  for (int i = first; i < nv; i += step) vc[(i / a.vdim) * a.vpad + i % a.vdim] = (T)value(a.v_off + i);
+}
+
+template <bool BF16>
+__global__ void __launch_bounds__(kThreads) poly_norm_kernel(const PolyNormArgs a, const int e4) {
+  extern __shared__ float4 s_z[];   // [e4][kThreads]
+  __shared__ ClusterSum<3> s_sum;
+  const int tid = threadIdx.x;
+  const int csize = (int)cg::this_cluster().num_blocks();
+  const int crank = (int)cg::this_cluster().block_rank();
+  const int r = (int)blockIdx.x / csize;
+  const int k4 = a.out.kp >> 2, lane4 = crank * kThreads + tid, step4 = csize * kThreads;
+  if (csize > 1) cg::this_cluster().sync();
+  grid_dep_launch();
+  grid_dep_wait();
+  float ss[3] = {0.f, 0.f, 0.f};
+  for (int e = 0, i = lane4; i < k4; ++e, i += step4) {
+    const float4 z = sum_partials(a.z, r, i * 4);
+    s_z[e * kThreads + tid] = z;
+    const float4 z2 = mul4(z, z), z3 = mul4(z2, z);
+    ss[0] += dot4(z);
+    ss[1] += dot4(z2);
+    ss[2] += dot4(z3);
+  }
+  cluster_sum<3>(s_sum, 0, csize, crank, ss);
+  const float n = (float)a.width;
+  const float c1 = a.coef[0] / sqrtf(ss[0] / n + a.eps), c2 = a.coef[1] / sqrtf(ss[1] / n + a.eps), c3 = a.coef[2] / sqrtf(ss[2] / n + a.eps);
+  const float c0 = a.coef[3];
+  auto f = [&](float z, int k) { return k < a.width ? fmaf(z, fmaf(z, fmaf(z, c3, c2), c1), c0) : 0.f; };
+  for (int e = 0, i = lane4; i < k4; ++e, i += step4) {
+    const float4 z = s_z[e * kThreads + tid];
+    const int k = i * 4;
+    act_store4<BF16>(a.out, r, k, make_float4(f(z.x, k), f(z.y, k + 1), f(z.z, k + 2), f(z.w, k + 3)));
+  }
+}
+
+// CTAs per row: enough to spread a few rows over the SMs, never more than there are 4-element pieces for.
+int row_cluster(int rows, int64_t n4) {
+  int c = 1;
+  while (c < 8 && (int64_t)c * kThreads < n4 && rows * c * 2 <= sm_count()) c *= 2;
+  return c;
+}
+
+}  // namespace
+
+tb_status launch_glue(Precision p, const GlueArgs& a, cudaStream_t st) {
+  const int n = a.r.rows - a.row0;
+  if (n < 1) return TB_OK;
+  const int c = row_cluster(n, a.xs / 4);
+  int per = 1;
+  if (c == 1)
+    while (per < 4 && n / (per * 2) >= sm_count()) per *= 2;   // fewer rows computed again in front of each block
+  const int e4 = (a.xs / 4 + c * kThreads - 1) / (c * kThreads);
+  const int taps = a.conv_w ? a.taps : 1;
+  const size_t smem = (size_t)(1 + taps) * e4 * kThreads * sizeof(float4);
+  if (smem > 200 * 1024 || taps > 32) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: hidden size %d with %d taps", a.width, a.taps);
+  const dim3 grid((unsigned)((n + per - 1) / per * c));
+  if (p == Precision::kBf16) return launch_kernel(glue_kernel<true>, grid, dim3(kThreads), smem, st, a.pdl, c, a, per, e4);
+  return launch_kernel(glue_kernel<false>, grid, dim3(kThreads), smem, st, a.pdl, c, a, per, e4);
+}
+
+tb_status launch_qkv_prep(Precision p, const QkvPrepArgs& a, cudaStream_t st) {
+  const int c = row_cluster(a.r.rows, (int64_t)(a.heads + 2 * a.kv_heads) * a.dim / 2);
+  const dim3 grid((unsigned)(a.r.rows * c));
+  if (p == Precision::kBf16) return launch_kernel(qkv_prep_kernel<__nv_bfloat16>, grid, dim3(kThreads), 0, st, a.pdl, c, a);
+  return launch_kernel(qkv_prep_kernel<float>, grid, dim3(kThreads), 0, st, a.pdl, c, a);
+}
+
+tb_status launch_poly_norm(Precision p, const PolyNormArgs& a, cudaStream_t st) {
+  const int c = row_cluster(a.rows, a.out.kp / 4);
+  const int e4 = (a.out.kp / 4 + c * kThreads - 1) / (c * kThreads);
+  const size_t smem = (size_t)e4 * kThreads * sizeof(float4);
+  if (smem > 200 * 1024) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: feed-forward width %d", a.width);
+  const dim3 grid((unsigned)(a.rows * c));
+  if (p == Precision::kBf16) return launch_kernel(poly_norm_kernel<true>, grid, dim3(kThreads), smem, st, a.pdl, c, a, e4);
+  return launch_kernel(poly_norm_kernel<false>, grid, dim3(kThreads), smem, st, a.pdl, c, a, e4);
+}
+
+}  // namespace tb

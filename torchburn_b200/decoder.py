@@ -48,60 +48,17 @@ class _Operands:
         return p
 
 
-class B200QwenDecoder:
-    """The reference's decoder class on a B200.
+class DecoderHandle:
+    """A ``tb_decoder`` and its calls, whatever model is behind it.  Subclasses create the handle in their
+    constructor and call ``_adopt``."""
 
-    Constructor arguments follow RustQwenDecoder::new (src/llm/decoder.rs:176-210):
-    ``layers_data`` is a list of per-layer sequences in the order
-    [input_norm, qkv_w, qkv_s, o_w, o_s, post_norm, gate_w, gate_s, up_w, up_s,
-    down_w, down_s, (qkv_b)] (numpy arrays or torch tensors; dicts keyed by those
-    names are accepted too).  ``max_batch``, ``tp_size``/``tp_rank``, ``debug`` and
-    ``fused_step`` (True: batch-1 steps as the one persistent step kernel; False: as a chain of single
-    kernels; None: the faster of the two - the step kernel with tensor parallelism, the chain on one
-    GPU) have no counterpart in the reference.
-    """
-
-    def __init__(self, embed_tokens, layers_data: Sequence, final_norm_w, lm_head_w, lm_head_s,
-                 num_layers: int, hidden_size: int, intermediate_size: int, num_heads: int,
-                 num_kv_heads: int, head_dim: int, group_size: int = 64, rms_norm_eps: float = 1e-6,
-                 max_seq_len: int = 2048, rope_theta: float = 1000000.0, max_batch: int = 1,
-                 tp_size: int = 1, tp_rank: int = 0, debug: bool = False, vocab_size: Optional[int] = None,
-                 nccl_only: bool = False, pdl: bool = True, fused_step: Optional[bool] = None):
-        self._h = None
-        ops = _Operands()
-        emb_p = ops.ptr(embed_tokens, np.float32)
-        self.vocab_size = int(vocab_size if vocab_size is not None else embed_tokens.shape[0])
-        arr = (LayerWeights * num_layers)()
-        if len(layers_data) != num_layers:
-            raise ValueError(f"layers_data has {len(layers_data)} entries, num_layers is {num_layers}")
-        for i, ld in enumerate(layers_data):
-            if isinstance(ld, dict):
-                items = [ld.get(k) for k in _LAYER_ORDER]
-            else:
-                items = list(ld) + [None] * (13 - len(ld))
-                if len(ld) < 12:
-                    raise _lib.TorchBurnB200Error(2, "Each layer requires 12 capsules: input_norm, qkv_w, qkv_s, o_w, o_s, post_norm, gate_w, gate_s, up_w, up_s, down_w, down_s")
-            for key, item in zip(_LAYER_ORDER, items):
-                setattr(arr[i], key, ops.ptr(item, np.uint8 if key in _U8 else np.float32))
-        fn_p = ops.ptr(final_norm_w, np.float32)
-        lw_p = ops.ptr(lm_head_w, np.uint8)
-        ls_p = ops.ptr(lm_head_s, np.float32)
-        flags = ((_lib.TB_DECODER_NO_GRAPH if debug else 0) | (_lib.TB_DECODER_NCCL_ONLY if nccl_only else 0)
-                 | (0 if pdl else _lib.TB_DECODER_NO_PDL) | (0 if fused_step is None else (_lib.TB_DECODER_FUSED_STEP if fused_step else _lib.TB_DECODER_NO_FUSED_STEP)))
-        cfg = ModelConfig(vocab_size=self.vocab_size, hidden_size=hidden_size, intermediate_size=intermediate_size,
-                          num_layers=num_layers, num_heads=num_heads, num_kv_heads=num_kv_heads, head_dim=head_dim,
-                          group_size=group_size, rms_norm_eps=rms_norm_eps, max_seq_len=max_seq_len,
-                          rope_theta=rope_theta, max_batch=max_batch, tp_size=tp_size, tp_rank=tp_rank, flags=flags)
-        self.cfg = cfg
-        h = C.c_void_p()
-        check(lib().tb_decoder_create(C.byref(h), C.byref(cfg), emb_p, C.cast(arr, C.c_void_p), fn_p, lw_p, ls_p,
-                                      ops.space if ops.space is not None else TB_HOST))
-        self._h = h
+    def _adopt(self, handle, vocab_size: int, max_batch: int, max_seq_len: int) -> None:
+        self._h = handle
+        self.vocab_size = vocab_size
         self.max_batch = max_batch
         self.max_seq_len = max_seq_len
-        self._logits = np.empty((max_batch, self.vocab_size), np.float32)
+        self._logits = np.empty((max_batch, vocab_size), np.float32)
         self._rng = C.c_uint64(0x9E3779B97F4A7C15)
-        del ops  # the library copied everything to the device
 
     def __del__(self):
         self.close()
@@ -166,6 +123,25 @@ class B200QwenDecoder:
         check(lib().tb_decoder_verify_tokens(self._h, start_offset, t.ctypes.data, t.size, out.ctypes.data))
         return out
 
+    def extend(self, tokens: Sequence[int], start_offset: int, want: Sequence[int] = (), seq: int = 0) -> np.ndarray:
+        """The next tokens of sequence ``seq`` in as few steps as the decoder's rows allow; returns the logits
+        at the places ``want`` among them, [len(want), vocab]."""
+        t = np.ascontiguousarray(tokens, dtype=np.int64)
+        w = np.ascontiguousarray(want, dtype=np.int64)
+        out = np.empty((w.size, self.vocab_size), np.float32)
+        check(lib().tb_decoder_extend(self._h, seq, start_offset, t.ctypes.data, t.size, w.ctypes.data, w.size, out.ctypes.data))
+        return out
+
+    def reset_sequence(self, seq: int = 0) -> None:
+        """Gives back what a sequence holds; it starts again at position 0."""
+        check(lib().tb_decoder_reset_sequence(self._h, seq))
+
+    def generate_greedy(self, first_token: int, start_offset: int, n_new: int) -> List[int]:
+        """n_new tokens, each argmax fed back on the device; ``first_token`` sits at ``start_offset``."""
+        out = np.empty(max(n_new, 1), np.int64)
+        check(lib().tb_decoder_generate_greedy(self._h, int(first_token), int(start_offset), int(n_new), out.ctypes.data))
+        return [int(t) for t in out[:n_new]]
+
     def decode_and_sample(self, token_id: int, offset: int, temperature: float = 0.7, top_k: int = 40,
                           repetition_penalty: float = 1.0, recent_tokens: Optional[Sequence[int]] = None,
                           top_p: float = 1.0) -> int:
@@ -210,13 +186,6 @@ class B200QwenDecoder:
         self._rng = C.c_uint64(value or 1)
 
     # ---- extras -------------------------------------------------------------
-    def read_kv_cache(self, layer: int, seq: int = 0):
-        shape = (self.cfg.num_kv_heads // max(self.cfg.tp_size, 1), self.max_seq_len, self.cfg.head_dim)
-        k = np.empty(shape, np.float32)
-        v = np.empty(shape, np.float32)
-        check(lib().tb_decoder_read_kv_cache(self._h, layer, seq, k.ctypes.data, v.ctypes.data))
-        return k, v
-
     def debug_stage(self, name: str) -> np.ndarray:
         n = C.c_int64()
         check(lib().tb_decoder_debug_stage(self._h, name.encode(), None, 0, C.byref(n)))
@@ -241,6 +210,65 @@ class B200QwenDecoder:
     @property
     def handle(self):
         return self._h
+
+
+class B200QwenDecoder(DecoderHandle):
+    """The reference's decoder class on a B200.
+
+    Constructor arguments follow RustQwenDecoder::new (src/llm/decoder.rs:176-210):
+    ``layers_data`` is a list of per-layer sequences in the order
+    [input_norm, qkv_w, qkv_s, o_w, o_s, post_norm, gate_w, gate_s, up_w, up_s,
+    down_w, down_s, (qkv_b)] (numpy arrays or torch tensors; dicts keyed by those
+    names are accepted too).  ``max_batch``, ``tp_size``/``tp_rank``, ``debug`` and
+    ``fused_step`` (True: batch-1 steps as the one persistent step kernel; False: as a chain of single
+    kernels; None: the faster of the two - the step kernel with tensor parallelism, the chain on one
+    GPU) have no counterpart in the reference.
+    """
+
+    def __init__(self, embed_tokens, layers_data: Sequence, final_norm_w, lm_head_w, lm_head_s,
+                 num_layers: int, hidden_size: int, intermediate_size: int, num_heads: int,
+                 num_kv_heads: int, head_dim: int, group_size: int = 64, rms_norm_eps: float = 1e-6,
+                 max_seq_len: int = 2048, rope_theta: float = 1000000.0, max_batch: int = 1,
+                 tp_size: int = 1, tp_rank: int = 0, debug: bool = False, vocab_size: Optional[int] = None,
+                 nccl_only: bool = False, pdl: bool = True, fused_step: Optional[bool] = None):
+        self._h = None
+        ops = _Operands()
+        emb_p = ops.ptr(embed_tokens, np.float32)
+        self.vocab_size = int(vocab_size if vocab_size is not None else embed_tokens.shape[0])
+        arr = (LayerWeights * num_layers)()
+        if len(layers_data) != num_layers:
+            raise ValueError(f"layers_data has {len(layers_data)} entries, num_layers is {num_layers}")
+        for i, ld in enumerate(layers_data):
+            if isinstance(ld, dict):
+                items = [ld.get(k) for k in _LAYER_ORDER]
+            else:
+                items = list(ld) + [None] * (13 - len(ld))
+                if len(ld) < 12:
+                    raise _lib.TorchBurnB200Error(2, "Each layer requires 12 capsules: input_norm, qkv_w, qkv_s, o_w, o_s, post_norm, gate_w, gate_s, up_w, up_s, down_w, down_s")
+            for key, item in zip(_LAYER_ORDER, items):
+                setattr(arr[i], key, ops.ptr(item, np.uint8 if key in _U8 else np.float32))
+        fn_p = ops.ptr(final_norm_w, np.float32)
+        lw_p = ops.ptr(lm_head_w, np.uint8)
+        ls_p = ops.ptr(lm_head_s, np.float32)
+        flags = ((_lib.TB_DECODER_NO_GRAPH if debug else 0) | (_lib.TB_DECODER_NCCL_ONLY if nccl_only else 0)
+                 | (0 if pdl else _lib.TB_DECODER_NO_PDL) | (0 if fused_step is None else (_lib.TB_DECODER_FUSED_STEP if fused_step else _lib.TB_DECODER_NO_FUSED_STEP)))
+        cfg = ModelConfig(vocab_size=self.vocab_size, hidden_size=hidden_size, intermediate_size=intermediate_size,
+                          num_layers=num_layers, num_heads=num_heads, num_kv_heads=num_kv_heads, head_dim=head_dim,
+                          group_size=group_size, rms_norm_eps=rms_norm_eps, max_seq_len=max_seq_len,
+                          rope_theta=rope_theta, max_batch=max_batch, tp_size=tp_size, tp_rank=tp_rank, flags=flags)
+        self.cfg = cfg
+        h = C.c_void_p()
+        check(lib().tb_decoder_create(C.byref(h), C.byref(cfg), emb_p, C.cast(arr, C.c_void_p), fn_p, lw_p, ls_p,
+                                      ops.space if ops.space is not None else TB_HOST))
+        self._adopt(h, self.vocab_size, max_batch, max_seq_len)
+        del ops  # the library copied everything to the device
+
+    def read_kv_cache(self, layer: int, seq: int = 0):
+        shape = (self.cfg.num_kv_heads // max(self.cfg.tp_size, 1), self.max_seq_len, self.cfg.head_dim)
+        k = np.empty(shape, np.float32)
+        v = np.empty(shape, np.float32)
+        check(lib().tb_decoder_read_kv_cache(self._h, layer, seq, k.ctypes.data, v.ctypes.data))
+        return k, v
 
 
 def create_b200_qwen_decoder(model: Any, max_seq_len: int = 4096, group_size: Optional[int] = None,

@@ -132,7 +132,7 @@ struct StepRows {
 struct GlueArgs {
   StepRows r;
   // source
-  const DenseWeight* embed = nullptr;    // embedding mode when not null
+  DenseWeight embed;                     // embedding mode when it has an image
   float embed_scale = 1.f;
   const __nv_bfloat16* pos_table = nullptr;  // [max positions, width] or null
   int64_t vocab = 0, max_pos = 0;

@@ -396,7 +396,7 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
   };
 
   reset_glue();
-  g.embed = &m->embed; g.embed_scale = m->cfg.embed_scale; g.pos_table = m->pos_table; g.vocab = m->cfg.vocab_size; g.max_pos = m->cfg.max_seq_len;
+  g.embed = m->embed; g.embed_scale = m->cfg.embed_scale; g.pos_table = m->pos_table; g.vocab = m->cfg.vocab_size; g.max_pos = m->cfg.max_seq_len;
   for (int l = 0; l < m->L; ++l) {
     const LayerRun& run = m->runs[(size_t)l];
     const LayerWeights& w = m->w[(size_t)run.weights];

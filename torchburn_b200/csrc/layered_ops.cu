@@ -100,7 +100,7 @@ __global__ void __launch_bounds__(kThreads) glue_kernel(const GlueArgs a, const 
   grid_dep_launch();
   grid_dep_wait();
   const int taps = a.conv_w != nullptr ? a.taps : 1;
-  const bool emb = a.embed != nullptr;
+  const bool emb = a.embed.img != nullptr;
   int slot = 0;
   const int32_t* posv = emb ? a.r.offsets : a.r.pos;   // the embedding kernel is the one that writes r.pos
   auto same_run = [&](int q, int r) { return q >= 0 && a.r.slots[q] == a.r.slots[r] && posv[q] >= 0 && posv[q] == posv[r] - (r - q); };
@@ -138,7 +138,7 @@ __global__ void __launch_bounds__(kThreads) glue_kernel(const GlueArgs a, const 
         if (live) {
           const int k = i * 4;
           // embedding row from the tile images of the tied output matrix
-          const unsigned char* t = static_cast<const unsigned char*>(a.embed->img) + ((size_t)(tok >> 7) * (a.embed->kp >> 6) + (k >> 6)) * 16384 +
+          const unsigned char* t = static_cast<const unsigned char*>(a.embed.img) + ((size_t)(tok >> 7) * (a.embed.kp >> 6) + (k >> 6)) * 16384 +
                                    (size_t)(tok & 127) * 128 + ((((k >> 3) & 7) ^ (tok & 7)) << 4) + ((k & 7) << 1);
           const uint2 u = *reinterpret_cast<const uint2*>(t);
           v = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));

@@ -7,7 +7,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any, Callable, List, Mapping, Optional
 
-from . import _lib, build as _build, checkpoint
+from . import _lib, checkpoint
 from .decoder import DecoderHandle
 
 
@@ -48,6 +48,8 @@ def load_model(model_dir: str, dtype: Optional[str] = None, max_seq_len: Optiona
     if dtype not in d.dtypes:
         raise NotImplementedError(f"{d.name} is served in {', '.join(d.dtypes)}, not in {dtype}")
     if build:
+        from . import build as _build
+
         _lib.select(_build.ensure(d.profile))
     return d.load(model_dir, config, dtype, max_seq_len, **options)
 

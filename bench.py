@@ -1,6 +1,7 @@
 """Headline benchmark: INT4 decode tokens/s of a Llama-3-8B-shaped model on B200(s).
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--batch B] [--impl reference]
+    python bench.py --design dabevik     # a layered design beside the INT4 decoder (another JSON line)
 
 N=1 workload: the headline configuration "Llama-3-8B-architecture INT4 decode" - hidden 4096,
 32 layers, 32 q / 8 kv heads, head_dim 128, intermediate 14336, vocab 128256,
@@ -769,6 +770,112 @@ def time_config3(torch, tb, device, args):
     return out
 
 
+# ----------------------------------------------------------------- layered designs (--design)
+# Layers like a real model's, random weights.  The feed-forward of the design has two matrices where the INT4
+# model has three: 1.5 times the width gives both the same number of weights.
+DESIGN_SIZES = {
+    "llama-3-8b-layers": dict(width=4096, layers=8, heads=32, kv_heads=8, dim=128, ff=21504, vocab=128256),
+    "qwen2.5-0.5b": dict(width=896, layers=24, heads=14, kv_heads=2, dim=64, ff=7296, vocab=151936),
+}
+
+
+def build_dabevik(torch, tb, z, device, context, max_batch, prefill_rows, seed=3, dtype="bfloat16"):
+    """A Dabevik model of these sizes; the window spans the context, four first tokens are kept."""
+    gen = torch.Generator(device).manual_seed(seed)
+
+    def rnd(*shape, std=0.02, mean=0.0):
+        return (mean + std * torch.randn(*shape, device=device, generator=gen)).to(torch.bfloat16)
+
+    w, h, kv, d, ff = z["width"], z["heads"], z["kv_heads"], z["dim"], z["ff"]
+    positions = context + 512
+    specs = []
+    for _ in range(z["layers"]):
+        t = {n: rnd(w, mean=1.0) for n in ("norm1", "norm1_after", "norm2", "norm2_after")}
+        t.update(conv1=rnd(w, 4, std=0.2), conv2=rnd(w, 4, std=0.2), q_w=rnd(h * d, w), q_b=rnd(h * d), k_w=rnd(kv * d, w), k_b=rnd(kv * d),
+                 v_w=rnd(kv * d, w), v_b=rnd(kv * d), q_norm=rnd(h * d, mean=1.0), k_norm=rnd(kv * d, mean=1.0), talk=rnd(h, h, std=0.2),
+                 o_w=rnd(w, h * d), o_b=rnd(w), up_w=rnd(ff, w), down_w=rnd(w, ff), act=rnd(4, std=0.5))
+        specs.append(tb.LayerSpec(h, kv, d, d, d ** -0.5, context, 4, ff, None, t))
+    return tb.LayeredDecoder(specs, rnd(z["vocab"], w, std=1.0), rnd(w, mean=1.0), rnd(positions, w), hidden_size=w, vocab_size=z["vocab"],
+                             norm_eps=1e-5, max_seq_len=positions, embed_scale=1.0, conv_taps=4, max_batch=max_batch,
+                             prefill_rows=prefill_rows, dtype=dtype)
+
+
+def run_design(args):
+    """Decode and prompt throughput of a layered design beside the INT4 decoder of equal size: CUDA events on the
+    decoder's stream around K steps (decode), wall clock around whole prompts (token ids in, last logits left on the device)."""
+    import torch
+
+    import torchburn_b200 as tb
+
+    torch.cuda.set_device(0)
+    device = torch.device("cuda", 0)
+    K, W, ctx = args.steps, max(args.warmup, 3), CONTEXT
+    peak, kind = measured_peak()
+    try:
+        tflops = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+    except Exception:
+        tflops = 1590.0
+    batches = (1, 8, 32)
+    out = []
+
+    def prompt_ms(fn, reps=3):
+        fn()
+        torch.cuda.synchronize(device)
+        times = []
+        for _ in range(reps):
+            t0 = time.perf_counter()
+            fn()
+            torch.cuda.synchronize(device)
+            times.append((time.perf_counter() - t0) * 1e3)
+        return float(np.median(times))
+
+    with ClockSampler(0) as clocks:
+        for name, z in DESIGN_SIZES.items():
+            ids = np.random.default_rng(1).integers(0, z["vocab"], ctx).tolist()
+            r = {"size": name, "layers": z["layers"], "context": ctx, "decode": {}, "prompt": {}}
+            body = z["layers"] * (z["width"] * z["dim"] * (2 * z["heads"] + 2 * z["kv_heads"]) + 2 * z["width"] * z["ff"])
+            head = z["vocab"] * z["width"]
+            # keys the positions of the prompt see, on average, times the query/key and value products of a position and key
+            attn_flops = 4.0 * z["layers"] * z["heads"] * z["dim"] * (ctx / 2)
+            for rows in (512, 1024):
+                dec = build_dabevik(torch, tb, z, device, ctx, 1, rows)
+                ms = prompt_ms(lambda: dec.prefill_tokens(ids, 0))
+                r["prompt"][f"dabevik_{rows}_rows"] = {"tokens": ctx, "ms": ms, "tokens_per_s": ctx * 1e3 / ms,
+                                                      "frac_of_bf16_peak": ctx * (2.0 * body + attn_flops) / (ms * 1e-3) / 1e12 / tflops}
+                dec.close()
+            dec = build_dabevik(torch, tb, z, device, ctx, max(batches), 512)
+            for s in range(max(batches)):
+                dec.extend(ids[:ctx - 256], 0, seq=s)
+            for b in batches:
+                start = ctx - 256 + W
+                ms = float(np.median(timed_steps(torch, None, tb, dec, device, 1, b, ctx - 256, K, W, args.repeats))) / K
+                kv = z["layers"] * b * (start + K // 2) * 2 * z["kv_heads"] * z["dim"] * 2
+                by = 2.0 * (body + head) + kv
+                r["decode"][f"dabevik_batch{b}"] = {"tokens_per_s": b * 1e3 / ms, "ms_per_step": ms, "launches_per_step": dec.launches_per_step(),
+                                                    "frac_of_hbm_peak": by / (ms * 1e-3) / 1e9 / peak}
+            dec.close()
+            # the INT4 decoder with the same weights count, heads and context
+            c = dict(vocab_size=z["vocab"], hidden_size=z["width"], intermediate_size=z["ff"] * 2 // 3, num_layers=z["layers"], num_heads=z["heads"],
+                     num_kv_heads=z["kv_heads"], head_dim=z["dim"], group_size=32, rms_norm_eps=1e-6, rope_theta=500000.0)
+            model = build_model(torch, tb, c, device, 1, 0)
+            dec = make_decoder(tb, c, model, ctx + 512, max(batches), 1, 0, args)
+            prefill_kv(torch, dec, c, device, ctx - 256, max(batches), 1, 0)
+            for b in batches:
+                ms = float(np.median(timed_steps(torch, None, tb, dec, device, 1, b, ctx - 256, K, W, args.repeats))) / K
+                by = step_weight_bytes(c) + b * kv_bytes_per_seq(c, ctx - 256 + W + K // 2)
+                r["decode"][f"int4_batch{b}"] = {"tokens_per_s": b * 1e3 / ms, "ms_per_step": ms, "launches_per_step": dec.launches_per_step(),
+                                                 "frac_of_hbm_peak": by / (ms * 1e-3) / 1e9 / peak}
+            ms = prompt_ms(lambda: dec.prefill_tokens(ids, 0))
+            r["prompt"]["int4_32_rows"] = {"tokens": ctx, "ms": ms, "tokens_per_s": ctx * 1e3 / ms,
+                                           "frac_of_bf16_peak": ctx * (2.0 * (body + head) + attn_flops) / (ms * 1e-3) / 1e12 / tflops}
+            dec.close()
+            del model
+            torch.cuda.empty_cache()
+            out.append(r)
+    _RESULT_LINE.append(json.dumps({"metric": "design_tokens_per_s", "design": args.design, "steps": K, "warmup": W, "data": "synthetic",
+                                    "peak_kind": f"of {kind}", "fault_flag": int(tb.lib().tb_device_fault_flag()), "clocks": clocks.summary(), "sizes": out}))
+
+
 def lib_stream(tb, dec):
     return tb.lib().tb_decoder_stream(dec.handle)
 
@@ -782,6 +889,8 @@ def main():
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--model", default="llama8b", choices=["llama8b", "qwen05b", "llama70b"],
                     help="qwen05b: workload configuration 3; llama70b: configuration 5 (8 GPUs, --batch 16); both with --quick")
+    ap.add_argument("--design", default=None, choices=["dabevik"],
+                    help="instead of the headline workload: decode and prompt throughput of a layered design beside the INT4 decoder of equal size")
     ap.add_argument("--repeats", type=int, default=5, help="timed regions of --steps steps each; the median is reported")
     ap.add_argument("--no-batch-sweep", dest="batch_sweep", action="store_false", help="skip the batch 2 / 4 / 8 / 32 measurements")
     ap.add_argument("--no-config3", dest="config3", action="store_false", help="skip the Qwen2.5-0.5B-shaped measurement")
@@ -799,7 +908,9 @@ def main():
     real_stdout = os.dup(1)
     os.dup2(2, 1)
     try:
-        if args.impl == "reference":
+        if args.design:
+            run_design(args)
+        elif args.impl == "reference":
             run_reference(args)
         else:
             run_gpu(args)

@@ -162,30 +162,42 @@ def test_window_edges_by_influence(tmp_path, size, keep, dtype):
                 assert (moved > 1e-4) if seen else (moved == 0.0), (i, j, split, moved)
 
 
-@pytest.mark.parametrize("dtype", DTYPES)
-def test_far_key_stands_out(tmp_path, dtype):
-    """Query and key projections agree and positions are silent, so a repeated token scores far above the
-    hundreds of others: losing that one key, or its first-token neighbours, shows at once."""
+def needle_model():
+    """Token 300 + n is the key that token n asks for: the key projection is the query projection on permuted
+    features, and the embedding of 300 + n is that of n under the permutation, so their score stands far above
+    the hundreds of others.  Returns the tokens with such pairs at the given places and the same without keys."""
     cfg = o.make_config(vocab=400, width=96, taps=2, max_positions=800, layers=[
-        o.make_layer(4, 4, 32, 24, size=500, keep_first=2, ff=None, scale=0.5), o.make_layer(4, 4, 32, 24, size=40, keep_first=4, ff=64, scale=0.5)])
+        o.make_layer(4, 4, 32, 24, size=500, keep_first=2, ff=None, scale=0.6), o.make_layer(4, 4, 32, 24, size=40, keep_first=4, ff=64, scale=0.6)])
     w = o.make_weights(cfg, 11, sharp=1.0)
     w["pos"][:] = 0
-    for l in (0, 1):
-        for n in ("", ".b"):
-            w[f"l{l}.mix.k{n}"] = w[f"l{l}.mix.q{n}"]
-        w[f"l{l}.mix.q.norm"][:] = 1.0
-        w[f"l{l}.mix.k.norm"][:] = 1.0
-        w[f"l{l}.canon1"] *= 0.25
     rng = np.random.default_rng(5)
-    toks = rng.integers(10, cfg["vocab"], 620).tolist()
-    pairs = [(1, 45), (2, 70), (63, 560), (64, 563), (101, 600), (119, 619)]     # (key, query): near, at the edge, far
-    for n, (j, i) in enumerate(pairs):
-        toks[j] = toks[i] = n
+    perm = rng.permutation(cfg["width"])
+    for n in range(8):
+        w["embed"][300 + n][perm] = w["embed"][n]
+    for l in (0, 1):
+        p = f"l{l}."
+        w[p + "mix.k"] = np.zeros_like(w[p + "mix.q"])
+        w[p + "mix.k"][:, perm] = w[p + "mix.q"]
+        w[p + "mix.q.b"] *= 0
+        w[p + "mix.k.b"] *= 0
+        w[p + "mix.q.norm"][:] = 1.0
+        w[p + "mix.k.norm"][:] = 1.0
+        w[p + "norm1"][:] = 1.0
+        w[p + "canon1"] *= 0.25
+    toks = rng.integers(10, 290, 620).tolist()
+    pairs = [(1, 550), (0, 610), (63, 560), (64, 563), (101, 600), (119, 618), (579, 619)]   # kept, at the edge, far, near
     without = list(toks)
-    for n, (j, _) in enumerate(pairs):
-        without[j] = 9
+    for n, (j, i) in enumerate(pairs):
+        toks[j], toks[i] = 300 + n, n
+        without[i] = n
+    return cfg, w, toks, without, pairs
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_far_key_stands_out(tmp_path, dtype):
+    cfg, w, toks, without, pairs = needle_model()
     want, lost = o.forward(cfg, w, toks), o.forward(cfg, w, without)
-    assert all(err(lost[[i]], want[[i]]) > 5 * TOL["bfloat16"] for j, i in pairs if i - j < 500 and j > 3)
+    assert all(err(lost[[i]], want[[i]]) > 5 * TOL["bfloat16"] for _, i in pairs)
     dec = load(o.save_model(str(tmp_path), cfg, w), dtype, prefill_rows=128)
     at = [i for _, i in pairs]
     assert err(dec.extend(toks, 0, at), want[at]) < TOL[dtype]

@@ -215,11 +215,13 @@ struct WindowAttnArgs {
   int64_t scratch_rows = 0;
   ActOperand out;                        // K = heads * vdim
   bool one_sequence = false;             // the rows are consecutive positions of one sequence
-  int max_pos_hint = 0;                  // highest position of the step when one_sequence (host's knowledge)
   bool pdl = false;
 };
 constexpr int kScoreSplitsMax = 64;
 size_t window_attn_score_stride(int64_t max_visible);
 tb_status launch_window_attention(Precision p, const WindowAttnArgs& a, cudaStream_t st, int* launches);
+// Tensor-core form for a portion of one sequence (window_attention_mma.cu); reads q16, not q.
+bool window_mma_supported(const WindowAttnArgs& a);
+tb_status launch_window_attention_mma(const WindowAttnArgs& a, cudaStream_t st, int* launches);
 
 }  // namespace tb

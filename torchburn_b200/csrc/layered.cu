@@ -408,17 +408,20 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
     qa.heads = w.heads; qa.kv_heads = w.kv_heads; qa.dim = w.dim; qa.vdim = w.vdim; qa.dpad = w.dpad; qa.vpad = w.vpad;
     qa.q_off = w.q_off; qa.k_off = w.k_off; qa.v_off = w.v_off; qa.eps = m->cfg.norm_eps;
     qa.k_cache = run.k_cache; qa.v_cache = run.v_cache; qa.geom = run.geom; qa.pdl = s.pdl;
-    qa.q = m->q;
-    TB_TRY(launch_qkv_prep(prec, qa, st));
-    ++n;
     WindowAttnArgs wa;
-    wa.r = r; wa.q = m->q; wa.q16 = m->q16; wa.k_cache = run.k_cache; wa.v_cache = run.v_cache; wa.geom = run.geom;
+    wa.r = r; wa.k_cache = run.k_cache; wa.v_cache = run.v_cache; wa.geom = run.geom;
     wa.heads = w.heads; wa.kv_heads = w.kv_heads; wa.dim = w.dim; wa.vdim = w.vdim; wa.dpad = w.dpad; wa.vpad = w.vpad;
     wa.scale = run.scale; wa.window = run.window; wa.keep_first = run.keep_first; wa.talk = w.talk; wa.max_visible = run.max_visible;
     wa.scores = m->scores; wa.part = m->part;
     wa.scratch_rows = m->score_floats / ((int64_t)w.heads * (int64_t)window_attn_score_stride(run.max_visible));
     wa.out = ActOperand{m->act_o, mp, (int)w.o.kp};
-    wa.one_sequence = s.one_sequence; wa.max_pos_hint = s.last_pos; wa.pdl = s.pdl;
+    wa.one_sequence = s.one_sequence; wa.pdl = s.pdl;
+    wa.q = m->q; wa.q16 = m->q16;
+    const bool mma = prec == Precision::kBf16 && window_mma_supported(wa);
+    qa.q = mma ? nullptr : m->q;
+    qa.q16 = mma ? m->q16 : nullptr;
+    TB_TRY(launch_qkv_prep(prec, qa, st));
+    ++n;
     TB_TRY(launch_window_attention(prec, wa, st, &n));
     TB_TRY(product(w.o, wa.out, &y));
     g.y = y; g.y_bias = w.o_b; g.post_w = w.norm1b;

@@ -12,7 +12,6 @@ struct LayeredModel;
 struct LayeredStep {
   StepRows r;                      // tokens / slots / offsets on the device
   bool one_sequence = false;       // the rows are consecutive positions of one sequence
-  int last_pos = 0;                // its last position (host's knowledge, one_sequence only)
   const int32_t* row_map = nullptr;  // row -> logits row or -1; null: every row in place
   int logit_rows = 0;
   float* logits = nullptr;         // [logit_rows, vocab]

@@ -291,11 +291,15 @@ tb_status launch_generic(const WindowAttnArgs& a, cudaStream_t st, int* launches
 
 }  // namespace
 
-size_t window_attn_score_stride(int64_t max_visible) { return (size_t)pad_to(max_visible, 4); }
+size_t window_attn_score_stride(int64_t max_visible) {
+  // the tensor-core form numbers keys per block of 64 queries: up to 63 more than one row sees
+  return (size_t)pad_to(max_visible + 64, 32);
+}
 
 tb_status launch_window_attention(Precision p, const WindowAttnArgs& a, cudaStream_t st, int* launches) {
   if (a.heads < 1 || a.kv_heads < 1 || a.heads % a.kv_heads || a.dpad % 16 || a.vpad % 16 || a.scratch_rows < 1)
     return fail(TB_ERR_SHAPE, "window attention: bad shape");
+  if (p == Precision::kBf16 && window_mma_supported(a)) return launch_window_attention_mma(a, st, launches);
   if (p == Precision::kBf16) return launch_generic<__nv_bfloat16, true>(a, st, launches);
   return launch_generic<float, false>(a, st, launches);
 }

@@ -204,7 +204,7 @@ __global__ void __launch_bounds__(256, 2) window_mix_mma_kernel(const WindowAttn
   }
   // tiles that hold a key one of these queries sees
   const VisibleRange first(pos0, a.window, a.keep_first);
-  const int kept_tiles = (min(keys.nk, pos1 + 1) + kKT - 1) / kKT;
+  const int kept_tiles = (min(a.keep_first, keys.count) + kKT - 1) / kKT;   // a kept position's number is the position itself
   const int win0 = (keys.nk + first.lo - keys.lo) / kKT, win1 = (keys.nk + pos1 - keys.lo) / kKT;
   const int pieces = nkv * a.vpad >> 3;
   const int upv = a.vpad >> 4, units = nh * upv;     // 16-column output units

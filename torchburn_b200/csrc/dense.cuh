@@ -93,7 +93,7 @@ tb_status dense_weight_alloc(DenseWeight* w, int64_t rows, int64_t k);
 // Rows [row0, row0 + n) of the image from a row-major bf16 matrix [n, k] (host or device).
 tb_status dense_weight_fill(DenseWeight* w, int64_t row0, const uint16_t* src, int64_t n, int64_t k, tb_space space);
 
-// Partial sums of a projection: y[s][row][ldy], s < splits; the consumer adds them in that order.
+// Partial sums of a projection: y[s][row][ldy], s < splits <= 8; the consumer adds them in that order.
 struct PartialSums {
   float* y = nullptr;
   int splits = 1;
@@ -154,6 +154,9 @@ struct GlueArgs {
   float eps = 0.f;
   int row0 = 0;                          // first row handled
   float* snapshot = nullptr;             // optional copy of x' [rows, xs]
+  float* rstd = nullptr;                 // [rows] scratch: 1 / rms of x'.  When given, the glue is two kernels
+                                         // (row sums, then everything per element), better for many rows;
+                                         // row0 > 0 then runs the second one alone
   bool pdl = false;
 };
 tb_status launch_glue(Precision p, const GlueArgs& a, cudaStream_t st);
@@ -213,6 +216,7 @@ struct WindowAttnArgs {
   float* scores = nullptr;               // scratch [rows of a pass][heads][score_stride]
   float* part = nullptr;                 // scratch [rows of a pass][heads][splits][2]
   int64_t scratch_rows = 0;
+  float* parts = nullptr;                // scratch of window_parts_floats(), tensor-core form only; null: never split
   ActOperand out;                        // K = heads * vdim
   bool one_sequence = false;             // the rows are consecutive positions of one sequence
   bool pdl = false;
@@ -221,6 +225,7 @@ constexpr int kScoreSplitsMax = 64;
 size_t window_attn_score_stride(int64_t max_visible);
 tb_status launch_window_attention(Precision p, const WindowAttnArgs& a, cudaStream_t st, int* launches);
 // Tensor-core form for a portion of one sequence (window_attention_mma.cu); reads q16, not q.
+size_t window_parts_floats(int rows, int64_t cols);
 bool window_mma_supported(const WindowAttnArgs& a);
 tb_status launch_window_attention_mma(const WindowAttnArgs& a, cudaStream_t st, int* launches);
 

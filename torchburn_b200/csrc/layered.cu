@@ -27,7 +27,8 @@ namespace {
 
 constexpr int kHistory = 128;      // positions a sequence can always be taken back
 constexpr int kMaxSplits = 8;
-constexpr size_t kScoreBudget = 256u << 20;
+constexpr size_t kScoreBudget = 1024u << 20;
+constexpr int kManyRows = 64;       // from here on the glue is two kernels
 
 struct LayerWeights {
   int heads = 0, kv_heads = 0, dim = 0, vdim = 0, dpad = 0, vpad = 0;
@@ -79,6 +80,7 @@ struct LayeredModel {
   float* final_norm = nullptr;
   float* x[2] = {nullptr, nullptr};
   int32_t* pos = nullptr;
+  float* rstd = nullptr;
   float* y = nullptr;              // partial sums of a product
   int64_t y_floats = 0;
   void *act_x = nullptr, *act_o = nullptr, *act_z = nullptr;
@@ -86,6 +88,7 @@ struct LayeredModel {
   __nv_bfloat16* q16 = nullptr;
   float *scores = nullptr, *part = nullptr;
   int64_t score_floats = 0, part_rows = 0;
+  float* parts = nullptr;          // attention sums of key splits
   float* snap = nullptr;
   int64_t rollback = 0;
   std::vector<void*> owned;        // every device allocation
@@ -266,6 +269,7 @@ tb_status create_impl(LayeredModel* m, const tb_layered_layer* layers, const uin
   const size_t rp = (size_t)dense_row_pad(R);
   for (auto& x : m->x) TB_TRY(dev_alloc(m, &x, (size_t)R * m->xs, true));
   TB_TRY(dev_alloc(m, &m->pos, (size_t)R, true));
+  TB_TRY(dev_alloc(m, &m->rstd, (size_t)R, true));
   const int64_t y_rows = R > kMaxSplits * 64 ? R : kMaxSplits * 64;
   m->y_floats = y_rows * max_cols;
   TB_TRY(dev_alloc(m, &m->y, (size_t)m->y_floats, true));
@@ -285,6 +289,7 @@ tb_status create_impl(LayeredModel* m, const tb_layered_layer* layers, const uin
   m->score_floats = srows * max_score_row;
   TB_TRY(dev_alloc(m, &m->scores, (size_t)m->score_floats, false));
   TB_TRY(dev_alloc(m, &m->part, (size_t)(R * max_heads * kScoreSplitsMax * 2), false));
+  if (m->prec == Precision::kBf16) TB_TRY(dev_alloc(m, &m->parts, window_parts_floats(R, max_o), false));
   if (snapshots) TB_TRY(dev_alloc(m, &m->snap, (size_t)m->L * R * m->xs, true));
   TB_CUDA_TRY(cudaDeviceSynchronize());
   return TB_OK;
@@ -370,6 +375,7 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
   auto reset_glue = [&] {
     g = GlueArgs();
     g.r = r; g.width = m->width; g.xs = m->xs; g.eps = m->cfg.norm_eps; g.taps = m->taps; g.ring = m->ring; g.pdl = s.pdl;
+    g.rstd = rows >= kManyRows ? m->rstd : nullptr;
   };
   auto glue = [&](const float* pre_w, const float* conv, float* state) -> tb_status {
     g.pre_w = pre_w; g.conv_w = conv; g.conv_state = state;
@@ -380,12 +386,11 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
     const bool direct = conv != nullptr && (rows <= room || !s.one_sequence);
     g.write_state = direct;
     TB_TRY(launch_glue(prec, g, st));
-    ++n;
+    n += g.rstd ? 2 : 1;
     cur ^= 1;
     if (conv != nullptr && !direct) {   // a long portion: its last inputs, once every row has been done
-      GlueArgs t;
-      t.r = r; t.width = m->width; t.xs = m->xs; t.eps = m->cfg.norm_eps; t.ring = m->ring; t.pdl = s.pdl;
-      t.x_in = m->x[cur]; t.pre_w = pre_w; t.conv_state = state; t.write_state = true;
+      GlueArgs t = g;
+      t.conv_w = nullptr; t.out.data = nullptr; t.write_state = true;
       t.row0 = rows - room;
       TB_TRY(launch_glue(prec, t, st));
       ++n;
@@ -412,7 +417,7 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
     wa.r = r; wa.k_cache = run.k_cache; wa.v_cache = run.v_cache; wa.geom = run.geom;
     wa.heads = w.heads; wa.kv_heads = w.kv_heads; wa.dim = w.dim; wa.vdim = w.vdim; wa.dpad = w.dpad; wa.vpad = w.vpad;
     wa.scale = run.scale; wa.window = run.window; wa.keep_first = run.keep_first; wa.talk = w.talk; wa.max_visible = run.max_visible;
-    wa.scores = m->scores; wa.part = m->part;
+    wa.scores = m->scores; wa.part = m->part; wa.parts = m->parts;
     wa.scratch_rows = m->score_floats / ((int64_t)w.heads * (int64_t)window_attn_score_stride(run.max_visible));
     wa.out = ActOperand{m->act_o, mp, (int)w.o.kp};
     wa.one_sequence = s.one_sequence; wa.pdl = s.pdl;
@@ -444,10 +449,11 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
     // the final norm, for the rows whose logits are wanted, and the tied output matrix
     const ActOperand af{m->act_x, dense_row_pad(s.logit_rows > 0 ? s.logit_rows : 1), m->xs};
     g.pre_w = m->final_norm;
+    g.x_out = m->x[cur ^ 1];
     if (s.logit_rows > 0) g.out = af;
     g.row_map = s.row_map;
     TB_TRY(launch_glue(prec, g, st));
-    ++n;
+    n += g.rstd ? 2 : 1;
     if (s.logit_rows > 0) {
       DenseGemmArgs a;
       a.w = &m->embed; a.x = af; a.rows = s.logit_rows; a.out = s.logits; a.ldo = m->cfg.vocab_size; a.n_valid = m->cfg.vocab_size;

@@ -74,11 +74,116 @@ __device__ __forceinline__ float4 scale4(float4 a, float s) { return make_float4
 __device__ __forceinline__ float4 fma4(float4 a, float4 b, float4 c) {
   return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w));
 }
+constexpr int kMaxParts = 8;
 __device__ __forceinline__ float4 sum_partials(const PartialSums& y, int row, int col) {
   const float* p = y.y + (size_t)row * y.ldy + col;
-  float4 v = ld4(p);
-  for (int s = 1; s < y.splits; ++s) v = add4(v, ld4(p + (size_t)s * y.split_stride));
+  float4 t[kMaxParts];   // every load in flight before the first sum
+#pragma unroll
+  for (int s = 0; s < kMaxParts; ++s)
+    if (s < y.splits) t[s] = ld4(p + (size_t)s * y.split_stride);
+  float4 v = t[0];
+#pragma unroll
+  for (int s = 1; s < kMaxParts; ++s)
+    if (s < y.splits) v = add4(v, t[s]);
   return v;
+}
+// Four features of the embedding of token `tok` at position `pos`, from k on: the tile images of the tied output
+// matrix, scaled, plus the position row.
+__device__ __forceinline__ float4 embed4(const GlueArgs& a, int tok, int pos, int k) {
+  const unsigned char* t = static_cast<const unsigned char*>(a.embed.img) + ((size_t)(tok >> 7) * (a.embed.kp >> 6) + (k >> 6)) * 16384 +
+                           (size_t)(tok & 127) * 128 + ((((k >> 3) & 7) ^ (tok & 7)) << 4) + ((k & 7) << 1);
+  const uint2 u = *reinterpret_cast<const uint2*>(t);
+  float4 v = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
+  v = scale4(v, a.embed_scale);
+  if (a.pos_table) {
+    const __nv_bfloat16* pr = a.pos_table + (size_t)pos * a.width;
+    if (k < a.width) v.x += __bfloat162float(pr[k]);
+    if (k + 1 < a.width) v.y += __bfloat162float(pr[k + 1]);
+    if (k + 2 < a.width) v.z += __bfloat162float(pr[k + 2]);
+    if (k + 3 < a.width) v.w += __bfloat162float(pr[k + 3]);
+  }
+  return v;
+}
+// Is row q of the step the position r - q in front of row r's, in the same sequence?
+__device__ __forceinline__ bool same_run(const int32_t* slots, const int32_t* posv, int q, int r) {
+  return q >= 0 && slots[q] == slots[r] && posv[q] >= 0 && posv[q] == posv[r] - (r - q);
+}
+
+// Many rows, first half of the glue: one CTA per row, x' and 1 / rms(x').
+__global__ void __launch_bounds__(kThreads) residual_norm_kernel(const GlueArgs a, const int e4) {
+  extern __shared__ float4 s_dyn[];   // [e4][kThreads]
+  __shared__ ClusterSum<1> s_sum;
+  const int tid = threadIdx.x, r = (int)blockIdx.x, xs4 = a.xs >> 2;
+  grid_dep_launch();
+  grid_dep_wait();
+  const bool emb = a.embed.img != nullptr;
+  int tok = 0, pos = 0;
+  if (emb) {
+    tok = a.r.tokens[r];
+    pos = a.r.offsets[r];
+    if (!(tok >= 0 && tok < a.vocab && pos >= 0 && pos < a.max_pos)) pos = -1;
+    if (tid == 0) a.r.pos[r] = pos;
+  }
+  float inv = 1.f;
+  float ss[1] = {0.f};
+  if (!emb) {
+    for (int e = 0, i = tid; i < xs4; ++e, i += kThreads) {
+      float4 v = sum_partials(a.y, r, i * 4);
+      if (a.y_bias) v = add4(v, ld4(a.y_bias + i * 4));
+      s_dyn[e * kThreads + tid] = v;
+      ss[0] += dot4(v);
+    }
+    if (a.post_w) {
+      cluster_sum<1>(s_sum, 0, 1, 0, ss);
+      inv = 1.0f / sqrtf(ss[0] / (float)a.width + a.eps);
+    }
+  }
+  ss[0] = 0.f;
+  for (int e = 0, i = tid; i < xs4; ++e, i += kThreads) {
+    float4 v = f4(0.f);
+    if (emb) {
+      if (pos >= 0) v = embed4(a, tok, pos, i * 4);
+    } else {
+      const float4 y = s_dyn[e * kThreads + tid];
+      v = ld4(a.x_in + (size_t)r * a.xs + i * 4);
+      v = a.post_w ? fma4(scale4(y, inv), ld4(a.post_w + i * 4), v) : add4(v, y);
+    }
+    ss[0] += dot4(v);
+    *reinterpret_cast<float4*>(a.x_out + (size_t)r * a.xs + i * 4) = v;
+    if (a.snapshot) *reinterpret_cast<float4*>(a.snapshot + (size_t)r * a.xs + i * 4) = v;
+  }
+  cluster_sum<1>(s_sum, 0, 1, 0, ss);
+  if (tid == 0) a.rstd[r] = 1.0f / sqrtf(ss[0] / (float)a.width + a.eps);
+}
+
+// Second half: h = x' * rstd * pre_w, the convolution, the operand, the convolution's state.  grid (rows, columns / 1024)
+template <bool BF16>
+__global__ void __launch_bounds__(kThreads) norm_conv_kernel(const GlueArgs a) {
+  const int r = a.row0 + (int)blockIdx.x, i = (int)blockIdx.y * kThreads + threadIdx.x;
+  grid_dep_launch();
+  grid_dep_wait();
+  if (i >= (a.xs >> 2)) return;
+  const int pos = a.r.pos[r];
+  const float4 pw = ld4(a.pre_w + i * 4);
+  auto input = [&](int q) { return mul4(scale4(ld4(a.x_out + (size_t)q * a.xs + i * 4), a.rstd[q]), pw); };
+  const float4 h = input(r);
+  if (a.write_state && pos >= 0)
+    *reinterpret_cast<float4*>(a.conv_state + ((size_t)a.r.slots[r] * a.ring + (pos & (a.ring - 1))) * a.xs + i * 4) = h;
+  const int orow = a.row_map != nullptr ? a.row_map[r] : r;
+  if (a.out.data == nullptr || orow < 0) return;
+  float4 o = h;
+  if (a.conv_w != nullptr && pos >= 0) {
+    for (int j = 0; j < a.taps && j <= pos; ++j) {
+      float4 hp = h;
+      if (j > 0) {
+        if (same_run(a.r.slots, a.r.pos, r - j, r)) hp = input(r - j);
+        else hp = ld4(a.conv_state + ((size_t)a.r.slots[r] * a.ring + ((pos - j) & (a.ring - 1))) * a.xs + i * 4);
+      }
+      o = fma4(ld4(a.conv_w + (size_t)(a.taps - 1 - j) * a.xs + i * 4), hp, o);
+    }
+  }
+  if (pos < 0) o = f4(0.f);
+  act_store4<BF16>(a.out, orow, i * 4, o);
 }
 
 // grid: (rows / rows_per * csize); rows_per consecutive rows per cluster, after up to taps - 1 rows of the same
@@ -103,10 +208,9 @@ __global__ void __launch_bounds__(kThreads) glue_kernel(const GlueArgs a, const 
   const bool emb = a.embed.img != nullptr;
   int slot = 0;
   const int32_t* posv = emb ? a.r.offsets : a.r.pos;   // the embedding kernel is the one that writes r.pos
-  auto same_run = [&](int q, int r) { return q >= 0 && a.r.slots[q] == a.r.slots[r] && posv[q] >= 0 && posv[q] == posv[r] - (r - q); };
 
   for (int r = max(0, r0 - (taps - 1)); r < r1; ++r) {
-    if (r < r0 && !same_run(r, r0)) continue;
+    if (r < r0 && !same_run(a.r.slots, posv, r, r0)) continue;
     // ---- x' ----
     int tok = 0, pos = posv[r];
     bool live = pos >= 0;
@@ -135,22 +239,7 @@ __global__ void __launch_bounds__(kThreads) glue_kernel(const GlueArgs a, const 
     for (int e = 0, i = lane4; i < xs4; ++e, i += step4) {
       float4 v = f4(0.f);
       if (emb) {
-        if (live) {
-          const int k = i * 4;
-          // embedding row from the tile images of the tied output matrix
-          const unsigned char* t = static_cast<const unsigned char*>(a.embed.img) + ((size_t)(tok >> 7) * (a.embed.kp >> 6) + (k >> 6)) * 16384 +
-                                   (size_t)(tok & 127) * 128 + ((((k >> 3) & 7) ^ (tok & 7)) << 4) + ((k & 7) << 1);
-          const uint2 u = *reinterpret_cast<const uint2*>(t);
-          v = make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
-          v = scale4(v, a.embed_scale);
-          if (a.pos_table) {
-            const __nv_bfloat16* pr = a.pos_table + (size_t)pos * a.width;
-            if (k < a.width) v.x += __bfloat162float(pr[k]);
-            if (k + 1 < a.width) v.y += __bfloat162float(pr[k + 1]);
-            if (k + 2 < a.width) v.z += __bfloat162float(pr[k + 2]);
-            if (k + 3 < a.width) v.w += __bfloat162float(pr[k + 3]);
-          }
-        }
+        if (live) v = embed4(a, tok, pos, i * 4);
       } else {
         v = ld4(a.x_in + (size_t)r * a.xs + i * 4);
         if (a.y.y != nullptr) {
@@ -169,7 +258,7 @@ __global__ void __launch_bounds__(kThreads) glue_kernel(const GlueArgs a, const 
     inv = 1.0f / sqrtf(ss[0] / (float)a.width + a.eps);
     const int orow = (a.row_map != nullptr && r >= r0) ? a.row_map[r] : r;
     uint32_t in_step = 0;   // bit j: the input j positions back is a row of this step (else it is in the state)
-    for (int j = 1; j < taps; ++j) in_step |= same_run(r - j, r) ? 1u << j : 0u;
+    for (int j = 1; j < taps; ++j) in_step |= same_run(a.r.slots, posv, r - j, r) ? 1u << j : 0u;
     float4* h_cur = s_h + (size_t)(r % taps) * hist;
     for (int e = 0, i = lane4; i < xs4; ++e, i += step4) {
       const float4 h = mul4(scale4(s_x[e * kThreads + tid], inv), ld4(a.pre_w + i * 4));
@@ -197,47 +286,57 @@ __global__ void __launch_bounds__(kThreads) glue_kernel(const GlueArgs a, const 
 
 // Query/key norm over the whole projection, biases, heads split and padded, k and v into the cache.
 template <typename T>
-__global__ void __launch_bounds__(kThreads) qkv_prep_kernel(const QkvPrepArgs a) {
+__global__ void __launch_bounds__(kThreads) qkv_prep_kernel(const QkvPrepArgs a, const int e4) {
+  extern __shared__ float4 s_val[];   // [e4][kThreads]: this thread's pieces of the row, summed
   __shared__ ClusterSum<2> s_sum;
   const int tid = threadIdx.x;
   const int csize = (int)cg::this_cluster().num_blocks();
   const int crank = (int)cg::this_cluster().block_rank();
   const int r = (int)blockIdx.x / csize;
   const int nq = a.heads * a.dim, nk = a.kv_heads * a.dim, nv = a.kv_heads * a.vdim;
+  const int cols4 = (a.v_off + nv + 3) >> 2, k4 = a.k_off >> 2, v4 = a.v_off >> 2;
   const int first = crank * kThreads + tid, step = csize * kThreads;
   if (csize > 1) cg::this_cluster().sync();
   grid_dep_launch();
   grid_dep_wait();
   const int pos = a.r.pos[r];
-  auto value = [&](int col) {
-    const float* p = a.y.y + (size_t)r * a.y.ldy + col;
-    float v = p[0];
-    for (int s = 1; s < a.y.splits; ++s) v += p[(size_t)s * a.y.split_stride];
-    return a.bias ? v + a.bias[col] : v;
-  };
   float ss[2] = {0.f, 0.f};
-  for (int i = first; i < nq; i += step) { const float v = value(a.q_off + i); ss[0] = fmaf(v, v, ss[0]); }
-  for (int i = first; i < nk; i += step) { const float v = value(a.k_off + i); ss[1] = fmaf(v, v, ss[1]); }
+  for (int e = 0, i = first; i < cols4; ++e, i += step) {   // padded columns are zero
+    float4 v = sum_partials(a.y, r, i * 4);
+    if (a.bias) v = add4(v, ld4(a.bias + i * 4));
+    s_val[e * kThreads + tid] = v;
+    if (i < k4) ss[0] += dot4(v);
+    else if (i < v4) ss[1] += dot4(v);
+  }
   cluster_sum<2>(s_sum, 0, csize, crank, ss);
   const float iq = a.q_norm ? 1.0f / sqrtf(ss[0] / (float)nq + a.eps) : 1.f;
   const float ik = a.k_norm ? 1.0f / sqrtf(ss[1] / (float)nk + a.eps) : 1.f;
-  for (int i = first; i < nq; i += step) {
-    float v = value(a.q_off + i) * iq;
-    if (a.q_norm) v *= a.q_norm[i];
-    const size_t o = (size_t)r * a.heads * a.dpad + (size_t)(i / a.dim) * a.dpad + i % a.dim;
-    if (a.q) a.q[o] = v;
-    if (a.q16) a.q16[o] = __float2bfloat16_rn(v);
-  }
-  if (pos < 0) return;
-  const size_t crow = (size_t)a.r.slots[r] * a.geom.rows + a.geom.row_of(pos);
+  const size_t crow = pos < 0 ? 0 : (size_t)a.r.slots[r] * a.geom.rows + a.geom.row_of(pos);
   T* kc = static_cast<T*>(a.k_cache) + crow * (size_t)(a.kv_heads * a.dpad);
   T* vc = static_cast<T*>(a.v_cache) + crow * (size_t)(a.kv_heads * a.vpad);
-  for (int i = first; i < nk; i += step) {
-    float v = value(a.k_off + i) * ik;
-    if (a.k_norm) v *= a.k_norm[i];
-    kc[(i / a.dim) * a.dpad + i % a.dim] = (T)v;
+  for (int e = 0, i = first; i < cols4; ++e, i += step) {
+    const float4 v4v = s_val[e * kThreads + tid];
+    const float v[4] = {v4v.x, v4v.y, v4v.z, v4v.w};
+    // segment of this piece: segments start at multiples of 4
+    const int seg = i < k4 ? 0 : (i < v4 ? 1 : 2);
+    const int base = i * 4 - (seg == 0 ? 0 : (seg == 1 ? a.k_off : a.v_off));
+    const int n = seg == 0 ? nq : (seg == 1 ? nk : nv), d = seg == 2 ? a.vdim : a.dim, dp = seg == 2 ? a.vpad : a.dpad;
+    int head = base / d, c = base - head * d;
+#pragma unroll
+    for (int j = 0; j < 4; ++j, ++c) {
+      if (base + j >= n) break;
+      if (c == d) { c = 0; ++head; }
+      const size_t o = (size_t)head * dp + c;
+      if (seg == 0) {
+        const float q = v[j] * iq * (a.q_norm ? a.q_norm[base + j] : 1.f);
+        if (a.q) a.q[(size_t)r * a.heads * a.dpad + o] = q;
+        if (a.q16) a.q16[(size_t)r * a.heads * a.dpad + o] = __float2bfloat16_rn(q);
+      } else if (pos >= 0) {
+        if (seg == 1) kc[o] = (T)(v[j] * ik * (a.k_norm ? a.k_norm[base + j] : 1.f));
+        else vc[o] = (T)v[j];
+      }
+    }
   }
-  for (int i = first; i < nv; i += step) vc[(i / a.vdim) * a.vpad + i % a.vdim] = (T)value(a.v_off + i);
 }
 
 template <bool BF16>
@@ -285,6 +384,15 @@ int row_cluster(int rows, int64_t n4) {
 tb_status launch_glue(Precision p, const GlueArgs& a, cudaStream_t st) {
   const int n = a.r.rows - a.row0;
   if (n < 1) return TB_OK;
+  if (a.rstd != nullptr) {   // many rows: two kernels, nothing computed twice
+    const int e4 = (a.xs / 4 + kThreads - 1) / kThreads;
+    if (a.taps > 32 || e4 > 50) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: hidden size %d with %d taps", a.width, a.taps);
+    if (a.row0 == 0)
+      TB_TRY(launch_kernel(residual_norm_kernel, dim3((unsigned)n), dim3(kThreads), (size_t)e4 * kThreads * sizeof(float4), st, a.pdl, 1, a, e4));
+    const dim3 grid((unsigned)n, (unsigned)e4);
+    return p == Precision::kBf16 ? launch_kernel(norm_conv_kernel<true>, grid, dim3(kThreads), 0, st, a.pdl, 1, a)
+                                 : launch_kernel(norm_conv_kernel<false>, grid, dim3(kThreads), 0, st, a.pdl, 1, a);
+  }
   const int c = row_cluster(n, a.xs / 4);
   int per = 1;
   if (c == 1)
@@ -299,10 +407,14 @@ tb_status launch_glue(Precision p, const GlueArgs& a, cudaStream_t st) {
 }
 
 tb_status launch_qkv_prep(Precision p, const QkvPrepArgs& a, cudaStream_t st) {
-  const int c = row_cluster(a.r.rows, (int64_t)(a.heads + 2 * a.kv_heads) * a.dim / 2);
+  const int cols4 = (a.v_off + a.kv_heads * a.vdim + 3) / 4;
+  const int c = row_cluster(a.r.rows, cols4);
+  const int e4 = (cols4 + c * kThreads - 1) / (c * kThreads);
+  const size_t smem = (size_t)e4 * kThreads * sizeof(float4);
+  if (smem > 200 * 1024) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: %d query and %d key heads", a.heads, a.kv_heads);
   const dim3 grid((unsigned)(a.r.rows * c));
-  if (p == Precision::kBf16) return launch_kernel(qkv_prep_kernel<__nv_bfloat16>, grid, dim3(kThreads), 0, st, a.pdl, c, a);
-  return launch_kernel(qkv_prep_kernel<float>, grid, dim3(kThreads), 0, st, a.pdl, c, a);
+  if (p == Precision::kBf16) return launch_kernel(qkv_prep_kernel<__nv_bfloat16>, grid, dim3(kThreads), smem, st, a.pdl, c, a, e4);
+  return launch_kernel(qkv_prep_kernel<float>, grid, dim3(kThreads), smem, st, a.pdl, c, a, e4);
 }
 
 tb_status launch_poly_norm(Precision p, const PolyNormArgs& a, cudaStream_t st) {

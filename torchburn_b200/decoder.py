@@ -61,7 +61,10 @@ class DecoderHandle:
         self._rng = C.c_uint64(0x9E3779B97F4A7C15)
 
     def __del__(self):
-        self.close()
+        try:
+            self.close()
+        except Exception:   # interpreter shutdown: the module's globals may be gone
+            pass
 
     def close(self) -> None:
         if getattr(self, "_h", None):

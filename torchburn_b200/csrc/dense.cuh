@@ -153,6 +153,7 @@ struct GlueArgs {
   int width = 0, xs = 0;
   float eps = 0.f;
   int row0 = 0;                          // first row handled
+  bool neighbours = true;                // false: no row of the step follows another one in its sequence
   float* snapshot = nullptr;             // optional copy of x' [rows, xs]
   float* rstd = nullptr;                 // [rows] scratch: 1 / rms of x'.  When given, the glue is two kernels
                                          // (row sums, then everything per element), better for many rows;

@@ -375,7 +375,8 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
   auto reset_glue = [&] {
     g = GlueArgs();
     g.r = r; g.width = m->width; g.xs = m->xs; g.eps = m->cfg.norm_eps; g.taps = m->taps; g.ring = m->ring; g.pdl = s.pdl;
-    g.rstd = rows >= kManyRows ? m->rstd : nullptr;
+    g.rstd = rows >= kManyRows && s.one_sequence ? m->rstd : nullptr;
+    g.neighbours = s.one_sequence && rows > 1;
   };
   auto glue = [&](const float* pre_w, const float* conv, float* state) -> tb_status {
     g.pre_w = pre_w; g.conv_w = conv; g.conv_state = state;

@@ -284,6 +284,77 @@ __global__ void __launch_bounds__(kThreads) glue_kernel(const GlueArgs a, const 
   }
 }
 
+// Decode rows: every row its own sequence, four features per thread.  The same arithmetic as glue_kernel; the
+// weights are read before the grid dependency wait, everything else as soon as its address is known.
+constexpr int kStepTaps = 8;
+template <bool BF16>
+__global__ void __launch_bounds__(kThreads) glue_step_kernel(const GlueArgs a) {
+  __shared__ ClusterSum<1> s_sum;
+  const int tid = threadIdx.x;
+  const int csize = (int)cg::this_cluster().num_blocks();
+  const int crank = (int)cg::this_cluster().block_rank();
+  const int r = a.row0 + (int)blockIdx.x / csize, i = crank * kThreads + tid;
+  const bool in = i < (a.xs >> 2), emb = a.embed.img != nullptr;
+  const int taps = a.conv_w != nullptr ? a.taps : 1;
+  const float4 zero = f4(0.f);
+  float4 pw = zero, ow = zero, bias = zero, cw[kStepTaps];
+  if (in) {
+    pw = ld4(a.pre_w + i * 4);
+    if (!emb && a.post_w) ow = ld4(a.post_w + i * 4);
+    if (!emb && a.y_bias) bias = ld4(a.y_bias + i * 4);
+#pragma unroll
+    for (int j = 0; j < kStepTaps; ++j)
+      if (a.conv_w != nullptr && j < taps) cw[j] = ld4(a.conv_w + (size_t)(taps - 1 - j) * a.xs + i * 4);
+  }
+  if (csize > 1) cg::this_cluster().sync();
+  grid_dep_launch();
+  grid_dep_wait();
+  int tok = 0, pos = emb ? a.r.offsets[r] : a.r.pos[r];
+  if (emb) {
+    tok = a.r.tokens[r];
+    if (!(tok >= 0 && tok < a.vocab && pos >= 0 && pos < a.max_pos)) pos = -1;
+    if (tid == 0 && crank == 0) a.r.pos[r] = pos;
+  }
+  float4 v = zero, x = zero, prev[kStepTaps];
+  if (in && !emb) {
+    x = ld4(a.x_in + (size_t)r * a.xs + i * 4);
+    v = add4(sum_partials(a.y, r, i * 4), bias);
+  }
+  float* state = a.conv_w != nullptr ? a.conv_state + (size_t)a.r.slots[r] * a.ring * a.xs + i * 4 : nullptr;
+  if (in && a.conv_w != nullptr) {
+#pragma unroll
+    for (int j = 1; j < kStepTaps; ++j)
+      if (j < taps && j <= pos) prev[j] = ld4(state + (size_t)((pos - j) & (a.ring - 1)) * a.xs);
+  }
+  float ss[1];
+  if (emb) {
+    if (in && pos >= 0) v = embed4(a, tok, pos, i * 4);
+  } else if (a.post_w) {
+    ss[0] = dot4(v);
+    cluster_sum<1>(s_sum, 0, csize, crank, ss);
+    v = fma4(scale4(v, 1.0f / sqrtf(ss[0] / (float)a.width + a.eps)), ow, x);
+  } else {
+    v = add4(x, v);
+  }
+  ss[0] = dot4(v);
+  cluster_sum<1>(s_sum, 1, csize, crank, ss);
+  if (!in) return;
+  if (a.x_out) *reinterpret_cast<float4*>(a.x_out + (size_t)r * a.xs + i * 4) = v;
+  if (a.snapshot) *reinterpret_cast<float4*>(a.snapshot + (size_t)r * a.xs + i * 4) = v;
+  const float4 h = mul4(scale4(v, 1.0f / sqrtf(ss[0] / (float)a.width + a.eps)), pw);
+  if (a.write_state && pos >= 0) *reinterpret_cast<float4*>(state + (size_t)(pos & (a.ring - 1)) * a.xs) = h;
+  const int orow = a.row_map != nullptr ? a.row_map[r] : r;
+  if (a.out.data == nullptr || orow < 0) return;
+  float4 o = h;
+  if (a.conv_w != nullptr) {
+#pragma unroll
+    for (int j = 0; j < kStepTaps; ++j)
+      if (j < taps && j <= pos) o = fma4(cw[j], j == 0 ? h : prev[j], o);
+  }
+  if (pos < 0) o = zero;
+  act_store4<BF16>(a.out, orow, i * 4, o);
+}
+
 // Query/key norm over the whole projection, biases, heads split and padded, k and v into the cache.
 template <typename T>
 __global__ void __launch_bounds__(kThreads) qkv_prep_kernel(const QkvPrepArgs a, const int e4) {
@@ -352,13 +423,26 @@ __global__ void __launch_bounds__(kThreads) poly_norm_kernel(const PolyNormArgs 
   grid_dep_launch();
   grid_dep_wait();
   float ss[3] = {0.f, 0.f, 0.f};
-  for (int e = 0, i = lane4; i < k4; ++e, i += step4) {
-    const float4 z = sum_partials(a.z, r, i * 4);
+  auto take = [&](int e, float4 z) {
     s_z[e * kThreads + tid] = z;
     const float4 z2 = mul4(z, z), z3 = mul4(z2, z);
     ss[0] += dot4(z);
     ss[1] += dot4(z2);
     ss[2] += dot4(z3);
+  };
+  if (a.z.splits == 1) {   // whole sums: several pieces in flight per thread
+    const float* z = a.z.y + (size_t)r * a.z.ldy;
+    int e = 0, i = lane4;
+    for (; i + 3 * step4 < k4; e += 4, i += 4 * step4) {
+      const float4 z0 = ld4(z + i * 4), z1 = ld4(z + (i + step4) * 4), z2 = ld4(z + (i + 2 * step4) * 4), z3 = ld4(z + (i + 3 * step4) * 4);
+      take(e, z0);
+      take(e + 1, z1);
+      take(e + 2, z2);
+      take(e + 3, z3);
+    }
+    for (; i < k4; ++e, i += step4) take(e, ld4(z + i * 4));
+  } else {
+    for (int e = 0, i = lane4; i < k4; ++e, i += step4) take(e, sum_partials(a.z, r, i * 4));
   }
   cluster_sum<3>(s_sum, 0, csize, crank, ss);
   const float n = (float)a.width;
@@ -400,6 +484,11 @@ tb_status launch_glue(Precision p, const GlueArgs& a, cudaStream_t st) {
   const int e4 = (a.xs / 4 + c * kThreads - 1) / (c * kThreads);
   const int taps = a.conv_w ? a.taps : 1;
   const size_t smem = (size_t)(1 + taps) * e4 * kThreads * sizeof(float4);
+  if (!a.neighbours && e4 == 1 && per == 1 && taps <= kStepTaps && (a.embed.img != nullptr || a.y.y != nullptr)) {
+    const dim3 grid((unsigned)(n * c));
+    return p == Precision::kBf16 ? launch_kernel(glue_step_kernel<true>, grid, dim3(kThreads), 0, st, a.pdl, c, a)
+                                 : launch_kernel(glue_step_kernel<false>, grid, dim3(kThreads), 0, st, a.pdl, c, a);
+  }
   if (smem > 200 * 1024 || taps > 32) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: hidden size %d with %d taps", a.width, a.taps);
   const dim3 grid((unsigned)((n + per - 1) / per * c));
   if (p == Precision::kBf16) return launch_kernel(glue_kernel<true>, grid, dim3(kThreads), smem, st, a.pdl, c, a, per, e4);

@@ -28,20 +28,6 @@ constexpr int kMixThreads = 512;  // one thread per position in the weight phase
 constexpr int kMixWarps = kMixThreads / 32;
 constexpr int kHeadChunk = 4;     // query heads that share a key's load
 
-template <typename T> __device__ __forceinline__ void load8(const T* p, float (&v)[8]);
-template <> __device__ __forceinline__ void load8<float>(const float* p, float (&v)[8]) {
-  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-template <> __device__ __forceinline__ void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) {
-  const uint4 u = *reinterpret_cast<const uint4*>(p);
-  const uint32_t w[4] = {u.x, u.y, u.z, u.w};
-#pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    v[2 * i] = __uint_as_float(w[i] << 16);
-    v[2 * i + 1] = __uint_as_float(w[i] & 0xFFFF0000u);
-  }
-}
 __device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
 __device__ __forceinline__ float2 load2(const __nv_bfloat16* p) {
   const uint32_t u = *reinterpret_cast<const uint32_t*>(p);
@@ -51,26 +37,45 @@ __device__ __forceinline__ void cp16(void* dst, const void* src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
 }
 
+__device__ __forceinline__ void ldm4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
+__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
 struct ScoreShape {
   int splits;       // CTAs that share a row's positions
   int64_t stride;   // floats per (row, head) of the score scratch
   int row0;
 };
 
-// grid (splits, kv heads, rows).  A warp takes 32 positions at a time: their keys by cp.async into the warp's own
-// tile, then one position per lane against every query head of the kv head.
+// Bytes of the queries of one kv head in shared memory.  fp32: [heads][dpad].  bf16: per four heads eight rows
+// [dpad + 8]: the heads rounded to bf16, then what the rounding left (together 16 mantissa bits).
+template <typename T>
+__host__ __device__ constexpr size_t query_bytes(int gq, int dpad) {
+  return sizeof(T) == 4 ? (size_t)gq * dpad * 4 : (size_t)((gq + 3) / 4) * 8 * (dpad + 8) * 2;
+}
+
+// grid (splits, kv heads, rows).  A warp takes 32 positions at a time, their keys by cp.async into the warp's own
+// tile.  fp32: one position per lane against every query head of the kv head.  bf16: the keys are the 16-row side
+// of mma.sync, the two pieces of four query heads its eight columns.
 template <typename T>
 __global__ void __launch_bounds__(256) window_scores_kernel(const WindowAttnArgs a, const ScoreShape sh) {
   extern __shared__ __align__(16) unsigned char s_raw[];
   constexpr int EP = 16 / (int)sizeof(T);
+  constexpr bool MMA = sizeof(T) == 2;
   const int gq = a.heads / a.kv_heads;
   const int kv = (int)blockIdx.y, h0 = kv * gq;
   const int lr = (int)blockIdx.z, r = sh.row0 + lr;
   const int stride = a.dpad + EP, pieces = a.dpad / EP;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = (int)blockDim.x >> 5;
-  float* s_q = reinterpret_cast<float*>(s_raw);        // [gq][dpad]
-  float2* s_ml = reinterpret_cast<float2*>(s_q + gq * a.dpad);   // [warps][gq] running (max, sum)
-  T* s_k = reinterpret_cast<T*>(s_raw + (((size_t)gq * a.dpad * 4 + (size_t)nw * gq * 8 + 15) & ~(size_t)15)) + (size_t)warp * kTileP * stride;
+  const size_t qb = query_bytes<T>(gq, a.dpad);
+  float2* s_ml = reinterpret_cast<float2*>(s_raw + qb);   // [warps][gq] running (max, sum)
+  T* s_k = reinterpret_cast<T*>(s_raw + ((qb + (size_t)nw * gq * 8 + 15) & ~(size_t)15)) + (size_t)warp * kTileP * stride;
   grid_dep_launch();
   grid_dep_wait();
   const int pos = a.r.pos[r];
@@ -95,49 +100,107 @@ __global__ void __launch_bounds__(256) window_scores_kernel(const WindowAttnArgs
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   if (t0 + warp < t1) stage(t0 + warp);
-  for (int i = tid; i < gq * a.dpad; i += (int)blockDim.x) s_q[i] = a.q[(size_t)r * a.heads * a.dpad + (size_t)h0 * a.dpad + i];
+  const float* qrow = a.q + (size_t)r * a.heads * a.dpad + (size_t)h0 * a.dpad;
+  if constexpr (MMA) {
+    __nv_bfloat16* s_q = reinterpret_cast<__nv_bfloat16*>(s_raw);
+    for (int i = tid; i < (gq + 3) / 4 * 4 * a.dpad; i += (int)blockDim.x) {
+      const int h = i / a.dpad, c = i - h * a.dpad;
+      const float q = h < gq ? qrow[i] : 0.f;
+      const __nv_bfloat16 hi = __float2bfloat16_rn(q);
+      __nv_bfloat16* d = s_q + (size_t)((h >> 2) * 8 + (h & 3)) * (a.dpad + 8) + c;
+      d[0] = hi;
+      d[4 * (a.dpad + 8)] = __float2bfloat16_rn(q - __bfloat162float(hi));
+    }
+  } else {
+    float* s_q = reinterpret_cast<float*>(s_raw);
+    for (int i = tid; i < gq * a.dpad; i += (int)blockDim.x) s_q[i] = qrow[i];
+  }
   for (int i = tid; i < nw * gq; i += (int)blockDim.x) s_ml[i] = make_float2(-INFINITY, 0.f);
   __syncthreads();
+  // running (max, sum) of head h with the maximum and sum of a tile
+  auto fold = [&](int h, float mx, float l) {
+    const float2 old = s_ml[warp * gq + h];
+    const float m1 = fmaxf(old.x, mx);
+    s_ml[warp * gq + h] = make_float2(m1, (old.x == -INFINITY ? 0.f : old.y * expf(old.x - m1)) + l * expf(mx - m1));
+  };
+  float* srow = a.scores + ((size_t)lr * a.heads + h0) * sh.stride;
   for (int t = t0 + warp; t < t1; t += nw) {
     if (t != t0 + warp) stage(t);
     asm volatile("cp.async.wait_all;" ::: "memory");
     __syncwarp();
-    const int v = t * kTileP + lane;
-    const T* kr = s_k + lane * stride;
     for (int hb = 0; hb < gq; hb += kHeadChunk) {
-      float acc[kHeadChunk];
+      if constexpr (MMA) {
+        const __nv_bfloat16* q = reinterpret_cast<const __nv_bfloat16*>(s_raw) + (size_t)((hb >> 2) * 8 + (lane >> 2)) * (a.dpad + 8) + (lane & 3) * 2;
+        float d[2][4];
 #pragma unroll
-      for (int j = 0; j < kHeadChunk; ++j) acc[j] = 0.f;
-      const float* q = s_q + hb * a.dpad;
-#pragma unroll 2
-      for (int c = 0; c < a.dpad; c += 8) {
-        float k8[8];
-        load8<T>(kr + c, k8);
+        for (int m = 0; m < 2; ++m)
 #pragma unroll
-        for (int j = 0; j < kHeadChunk; ++j) {
-          if (hb + j < gq) {
-            const float4 qa = *reinterpret_cast<const float4*>(q + j * a.dpad + c), qb = *reinterpret_cast<const float4*>(q + j * a.dpad + c + 4);
-            acc[j] = fmaf(qa.x, k8[0], fmaf(qa.y, k8[1], fmaf(qa.z, k8[2], fmaf(qa.w, k8[3], acc[j]))));
-            acc[j] = fmaf(qb.x, k8[4], fmaf(qb.y, k8[5], fmaf(qb.z, k8[6], fmaf(qb.w, k8[7], acc[j]))));
+          for (int i = 0; i < 4; ++i) d[m][i] = 0.f;
+#pragma unroll 4
+        for (int c = 0; c < a.dpad; c += 16) {
+          const uint32_t b0 = *reinterpret_cast<const uint32_t*>(q + c), b1 = *reinterpret_cast<const uint32_t*>(q + c + 8);
+#pragma unroll
+          for (int m = 0; m < 2; ++m) {
+            uint32_t ka[4];
+            ldm4(ka, s_k + (m * 16 + (lane & 15)) * stride + c + (lane >> 4) * 8);
+            mma16816(d[m], ka, b0, b1);
           }
         }
-      }
+        // d[m][2 x + y]: position 16 m + lane / 4 + 8 x, column 2 (lane & 3) + y = piece (lane & 3) / 2 of head 2 (lane & 1) + y
 #pragma unroll
-      for (int j = 0; j < kHeadChunk; ++j) {
-        if (hb + j >= gq) break;
-        const int h = hb + j;
-        const float s = v < nv ? acc[j] * a.scale : -INFINITY;
-        if (v < nv) a.scores[((size_t)lr * a.heads + h0 + h) * sh.stride + v] = s;
-        float mx = s;
+        for (int m = 0; m < 2; ++m)
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-        float l = v < nv ? expf(s - mx) : 0.f;
+          for (int i = 0; i < 4; ++i) d[m][i] += __shfl_xor_sync(0xffffffffu, d[m][i], 2);
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-        if (lane == 0) {
-          const float2 old = s_ml[warp * gq + h];
-          const float m1 = fmaxf(old.x, mx);
-          s_ml[warp * gq + h] = make_float2(m1, (old.x == -INFINITY ? 0.f : old.y * expf(old.x - m1)) + l * expf(mx - m1));
+        for (int y = 0; y < 2; ++y) {
+          const int h = hb + (lane & 1) * 2 + y;
+          float s[4], mx = -INFINITY;
+#pragma unroll
+          for (int x = 0; x < 4; ++x) {
+            const int v = t * kTileP + (x >> 1) * 16 + (lane >> 2) + (x & 1) * 8;
+            s[x] = v < nv ? d[x >> 1][(x & 1) * 2 + y] * a.scale : -INFINITY;
+            if (v < nv && (lane & 2) == 0 && h < gq) srow[(size_t)h * sh.stride + v] = s[x];
+            mx = fmaxf(mx, s[x]);
+          }
+#pragma unroll
+          for (int o = 16; o > 2; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+          float l = 0.f;
+#pragma unroll
+          for (int x = 0; x < 4; ++x) l += expf(s[x] - mx);
+#pragma unroll
+          for (int o = 16; o > 2; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+          if (lane < 2 && h < gq) fold(h, mx, l);
+        }
+      } else {
+        const int v = t * kTileP + lane;
+        const T* kr = s_k + lane * stride;
+        float acc[kHeadChunk];
+#pragma unroll
+        for (int j = 0; j < kHeadChunk; ++j) acc[j] = 0.f;
+        const float* q = reinterpret_cast<const float*>(s_raw) + hb * a.dpad;
+#pragma unroll 2
+        for (int c = 0; c < a.dpad; c += 4) {
+          const float4 k4 = *reinterpret_cast<const float4*>(kr + c);
+#pragma unroll
+          for (int j = 0; j < kHeadChunk; ++j) {
+            if (hb + j < gq) {
+              const float4 q4 = *reinterpret_cast<const float4*>(q + j * a.dpad + c);
+              acc[j] = fmaf(q4.x, k4.x, fmaf(q4.y, k4.y, fmaf(q4.z, k4.z, fmaf(q4.w, k4.w, acc[j]))));
+            }
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < kHeadChunk; ++j) {
+          if (hb + j >= gq) break;
+          const float s = v < nv ? acc[j] * a.scale : -INFINITY;
+          if (v < nv) srow[(size_t)(hb + j) * sh.stride + v] = s;
+          float mx = s;
+#pragma unroll
+          for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+          float l = v < nv ? expf(s - mx) : 0.f;
+#pragma unroll
+          for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+          if (lane == 0) fold(hb + j, mx, l);
         }
       }
     }
@@ -157,10 +220,44 @@ __global__ void __launch_bounds__(256) window_scores_kernel(const WindowAttnArgs
   }
 }
 
-// grid (cluster size, head groups, rows): HG query heads of one kv head per CTA.  512 positions at a time: a
-// thread takes one position through all heads (weights and mixing, in registers), then a warp takes 32 of the
-// positions, its lanes the value columns.
-template <typename T, bool BF16, int HG>
+// A warp's 32 positions times the values: lanes own CPL neighbouring columns; sums are added to `red` (the warp's own).
+template <typename T, int HG, int CPL>
+__device__ __forceinline__ void warp_values(const T* vals, const int* rows, int64_t row_elems, const float* w, int nj, int vpad, float* red) {
+  const int lane = threadIdx.x & 31;
+  for (int c = lane * CPL; c < vpad; c += 32 * CPL) {
+    float acc[HG][CPL];
+#pragma unroll
+    for (int h = 0; h < HG; ++h)
+#pragma unroll
+      for (int i = 0; i < CPL; ++i) acc[h][i] = 0.f;
+#pragma unroll 8
+    for (int j = 0; j < nj; ++j) {
+      const T* p = vals + (size_t)(rows ? rows[j] : j) * row_elems + c;
+      float x[CPL];
+#pragma unroll
+      for (int i = 0; i < CPL; i += 2) {
+        const float2 f = load2(p + i);
+        x[i] = f.x;
+        x[i + 1] = f.y;
+      }
+#pragma unroll
+      for (int h = 0; h < HG; ++h) {
+        const float wj = w[j * HG + h];
+#pragma unroll
+        for (int i = 0; i < CPL; ++i) acc[h][i] = fmaf(wj, x[i], acc[h][i]);
+      }
+    }
+#pragma unroll
+    for (int h = 0; h < HG; ++h)
+#pragma unroll
+      for (int i = 0; i < CPL; ++i) red[h * vpad + c + i] += acc[h][i];
+  }
+}
+
+// grid (cluster size, head groups, rows): HG query heads of one kv head per CTA.  A warp takes 32 positions at a
+// time and needs no other: their values by cp.async into the warp's tile (VSM) while a lane takes one position
+// through all heads (weights and mixing, in registers), then the lanes are the value columns.
+template <typename T, bool BF16, int HG, bool VSM>
 __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const WindowAttnArgs a, const ScoreShape sh) {
   extern __shared__ __align__(16) unsigned char s_raw[];
   const int gq = a.heads / a.kv_heads, per_kv = (gq + HG - 1) / HG;
@@ -174,6 +271,7 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const Window
   float* s_red = s_w + kMixThreads * HG;                                       // [warps][HG][vpad]
   float* s_acc = s_red + (size_t)kMixWarps * HG * a.vpad;                      // [HG][vpad]
   int* s_row = reinterpret_cast<int*>(s_acc + HG * a.vpad);                    // [512] cache rows
+  T* s_v = reinterpret_cast<T*>(s_row + kMixThreads) + (size_t)(threadIdx.x >> 5) * 32 * a.vpad;   // the warp's values when VSM
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int csize = (int)gridDim.x, crank = (int)blockIdx.x;
   grid_dep_launch();
@@ -201,16 +299,36 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const Window
     if (lane == 0) { s_m[g] = m; s_il[g] = l > 0.f ? 1.0f / l : 0.f; }
   }
   __syncthreads();
-  // this CTA's positions, in blocks of 512
+  // this CTA's positions, 32 per warp
   const int v_begin = (int)((int64_t)nv * crank / csize), v_end = (int)((int64_t)nv * (crank + 1) / csize);
-  for (int v0 = v_begin; v0 < v_end; v0 += kMixThreads) {
-    const int v = v0 + tid;
+  float* w_w = s_w + warp * 32 * HG;
+  int* w_row = s_row + warp * 32;
+  float* red = s_red + (size_t)warp * HG * a.vpad;
+  for (int v0 = v_begin + warp * 32; v0 < v_end; v0 += kMixThreads) {
+    const int v = v0 + lane;
     const bool live = v < v_end;
+    const int crow = a.geom.row_of(vr.position(live ? v : v0));
+    if (VSM) {
+      constexpr int EP = 16 / (int)sizeof(T);
+      const int pieces = a.vpad / EP;
+      int tr = lane / pieces, c = lane - tr * pieces;
+      const int rstep = 32 / pieces, cstep = 32 - rstep * pieces;
+      for (int i = 0; i < pieces; ++i) {
+        const int src = __shfl_sync(0xffffffffu, crow, tr);
+        cp16(s_v + tr * a.vpad + c * EP, vc + (size_t)src * crow_elems + c * EP);
+        tr += rstep;
+        c += cstep;
+        if (c >= pieces) { c -= pieces; ++tr; }
+      }
+      asm volatile("cp.async.commit_group;" ::: "memory");
+    } else {
+      w_row[lane] = crow;
+    }
     const float* sp = a.scores + (size_t)lr * a.heads * sh.stride + (live ? v : v0);
     float w[HG];
 #pragma unroll
     for (int h = 0; h < HG; ++h) w[h] = 0.f;
-    constexpr int GB = 8;
+    constexpr int GB = 16;
     for (int g0 = 0; g0 < a.heads; g0 += GB) {
       float s8[GB];
 #pragma unroll
@@ -225,36 +343,18 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const Window
         }
       }
     }
-    if (live) {
 #pragma unroll
-      for (int h = 0; h < HG; ++h) s_w[tid * HG + h] = w[h];
-      s_row[tid] = a.geom.row_of(vr.position(v));
+    for (int h = 0; h < HG; ++h) w_w[lane * HG + h] = w[h];
+    if (VSM) asm volatile("cp.async.wait_all;" ::: "memory");
+    __syncwarp();
+    const int nj = min(32, v_end - v0);
+    if (VSM) {
+      if (a.vpad > 64) warp_values<T, HG, 4>(s_v, nullptr, a.vpad, w_w, nj, a.vpad, red);
+      else warp_values<T, HG, 2>(s_v, nullptr, a.vpad, w_w, nj, a.vpad, red);
+    } else {
+      warp_values<T, HG, 2>(vc, w_row, crow_elems, w_w, nj, a.vpad, red);
     }
-    __syncthreads();
-    const int j0 = warp * 32, nj = min(32, v_end - v0 - j0);
-    if (nj > 0)
-      for (int c = lane * 2; c < a.vpad; c += 64) {
-        float2 acc[HG];
-#pragma unroll
-        for (int h = 0; h < HG; ++h) acc[h] = make_float2(0.f, 0.f);
-#pragma unroll 8
-        for (int j = 0; j < nj; ++j) {
-          const float2 x = load2(vc + (size_t)s_row[j0 + j] * crow_elems + c);
-#pragma unroll
-          for (int h = 0; h < HG; ++h) {
-            const float wj = s_w[(j0 + j) * HG + h];
-            acc[h].x = fmaf(wj, x.x, acc[h].x);
-            acc[h].y = fmaf(wj, x.y, acc[h].y);
-          }
-        }
-        float* d = s_red + (size_t)warp * HG * a.vpad + c;
-#pragma unroll
-        for (int h = 0; h < HG; ++h) {
-          d[h * a.vpad] += acc[h].x;
-          d[h * a.vpad + 1] += acc[h].y;
-        }
-      }
-    __syncthreads();
+    __syncwarp();
   }
   __syncthreads();
   for (int i = tid; i < HG * a.vpad; i += kMixThreads) {
@@ -294,7 +394,7 @@ tb_status launch_generic(const WindowAttnArgs& a, cudaStream_t st, int* launches
   const int64_t rows = pass;
   // scores: as many warps as their tiles fit
   auto sbytes = [&](int w) {
-    return (((size_t)gq * a.dpad * 4 + (size_t)w * gq * 8 + 15) & ~(size_t)15) + (size_t)w * kTileP * (a.dpad + 16 / sizeof(T)) * sizeof(T);
+    return ((query_bytes<T>(gq, a.dpad) + (size_t)w * gq * 8 + 15) & ~(size_t)15) + (size_t)w * kTileP * (a.dpad + 16 / sizeof(T)) * sizeof(T);
   };
   int warps = 8;
   while (warps > 1 && (sbytes(warps) > 112 * 1024 || warps / 2 >= tiles)) warps /= 2;
@@ -307,11 +407,15 @@ tb_status launch_generic(const WindowAttnArgs& a, cudaStream_t st, int* launches
   const int groups = a.kv_heads * ((gq + hg - 1) / hg);
   int cluster = 1;
   while (cluster < 8 && (int64_t)cluster * 64 < a.max_visible && rows * groups * cluster < sm_count()) cluster *= 2;
-  const size_t msm = (((size_t)a.heads * 8 + 15) & ~(size_t)15) +
-                     4 * ((((size_t)a.heads * hg + 3) & ~(size_t)3) + (size_t)kMixThreads * hg + (size_t)(kMixWarps + 1) * hg * a.vpad + kMixThreads);
-  if (sbytes(warps) > 200 * 1024 || msm > 200 * 1024)
+  size_t msm = (((size_t)a.heads * 8 + 15) & ~(size_t)15) +
+               4 * ((((size_t)a.heads * hg + 3) & ~(size_t)3) + (size_t)kMixThreads * hg + (size_t)(kMixWarps + 1) * hg * a.vpad + kMixThreads);
+  const size_t vsm = (size_t)kMixThreads * a.vpad * sizeof(T);
+  const bool staged = msm + vsm <= 220 * 1024;
+  if (staged) msm += vsm;
+  if (sbytes(warps) > 200 * 1024 || msm > 220 * 1024)
     return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: attention with %d heads of size %d/%d", a.heads, a.dim, a.vdim);
-  auto* mix = hg == 4 ? window_mix_kernel<T, BF16, 4> : (hg == 2 ? window_mix_kernel<T, BF16, 2> : window_mix_kernel<T, BF16, 1>);
+  auto* mix = staged ? (hg == 4 ? window_mix_kernel<T, BF16, 4, true> : (hg == 2 ? window_mix_kernel<T, BF16, 2, true> : window_mix_kernel<T, BF16, 1, true>))
+                     : (hg == 4 ? window_mix_kernel<T, BF16, 4, false> : (hg == 2 ? window_mix_kernel<T, BF16, 2, false> : window_mix_kernel<T, BF16, 1, false>));
   for (int64_t r0 = 0; r0 < a.r.rows; r0 += pass) {
     const int n = (int)(a.r.rows - r0 < pass ? a.r.rows - r0 : pass);
     sh.row0 = (int)r0;

@@ -24,8 +24,7 @@ namespace tb {
 namespace {
 
 constexpr int kTileP = 32;        // positions per tile: one per lane
-constexpr int kMixThreads = 512;  // one thread per position in the weight phase of the mix kernel
-constexpr int kMixWarps = kMixThreads / 32;
+constexpr int kMixThreads = 512;  // most threads of a mix CTA
 constexpr int kHeadChunk = 4;     // query heads that share a key's load
 
 __device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
@@ -267,15 +266,15 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const Window
   float* s_m = reinterpret_cast<float*>(s_raw);                                // [heads]
   float* s_il = s_m + a.heads;                                                 // [heads]
   float* s_t = reinterpret_cast<float*>(s_raw + (((size_t)a.heads * 8 + 15) & ~(size_t)15));   // [heads][HG]
-  float* s_w = s_t + (((size_t)a.heads * HG + 3) & ~(size_t)3);                // [512][HG]
-  float* s_red = s_w + kMixThreads * HG;                                       // [warps][HG][vpad]
-  float* s_acc = s_red + (size_t)kMixWarps * HG * a.vpad;                      // [HG][vpad]
-  int* s_row = reinterpret_cast<int*>(s_acc + HG * a.vpad);                    // [512] cache rows
-  T* s_v = reinterpret_cast<T*>(s_row + kMixThreads) + (size_t)(threadIdx.x >> 5) * 32 * a.vpad;   // the warp's values when VSM
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  float* s_w = s_t + (((size_t)a.heads * HG + 3) & ~(size_t)3);                // [32 warps][HG]
+  float* s_red = s_w + blockDim.x * HG;                                       // [warps][HG][vpad]
+  float* s_acc = s_red + (size_t)(blockDim.x >> 5) * HG * a.vpad;                      // [HG][vpad]
+  int* s_row = reinterpret_cast<int*>(s_acc + HG * a.vpad);                    // [32 warps] cache rows
+  T* s_v = reinterpret_cast<T*>(s_row + blockDim.x) + (size_t)(threadIdx.x >> 5) * 32 * a.vpad;   // the warp's values when VSM
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nthr = (int)blockDim.x, nw = nthr >> 5;
   const int csize = (int)gridDim.x, crank = (int)blockIdx.x;
   grid_dep_launch();
-  for (int i = tid; i < a.heads * HG; i += kMixThreads) {
+  for (int i = tid; i < a.heads * HG; i += nthr) {
     const int g = i / HG, h = i - g * HG;
     s_t[i] = h < nh ? a.talk[(size_t)(h0 + h) * a.heads + g] : 0.f;
   }
@@ -286,7 +285,27 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const Window
   const int nv = vr.count();
   const int64_t crow_elems = (int64_t)a.kv_heads * a.vpad;
   const T* vc = static_cast<const T*>(a.v_cache) + (pos < 0 ? 0 : (size_t)a.r.slots[r] * a.geom.rows * crow_elems) + kv * a.vpad;
-  for (int g = warp; g < a.heads; g += kMixWarps) {   // softmax statistics from the parts, in a fixed order
+  // this CTA's positions, 32 per warp at a time
+  const int v_begin = (int)((int64_t)nv * crank / csize), v_end = (int)((int64_t)nv * (crank + 1) / csize);
+  auto stage = [&](int crow) {
+    constexpr int EP = 16 / (int)sizeof(T);
+    const int pieces = a.vpad / EP;
+    int tr = lane / pieces, c = lane - tr * pieces;
+    const int rstep = 32 / pieces, cstep = 32 - rstep * pieces;
+    for (int i = 0; i < pieces; ++i) {
+      const int src = __shfl_sync(0xffffffffu, crow, tr);
+      cp16(s_v + tr * a.vpad + c * EP, vc + (size_t)src * crow_elems + c * EP);
+      tr += rstep;
+      c += cstep;
+      if (c >= pieces) { c -= pieces; ++tr; }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (VSM && v_begin + warp * 32 < v_end) {   // the first values travel while the statistics are put together
+    const int v = v_begin + warp * 32 + lane;
+    stage(a.geom.row_of(vr.position(v < v_end ? v : v_begin + warp * 32)));
+  }
+  for (int g = warp; g < a.heads; g += nw) {   // softmax statistics from the parts, in a fixed order
     const float2* p = reinterpret_cast<const float2*>(a.part) + ((size_t)lr * a.heads + g) * sh.splits;
     const float2 p0 = lane < sh.splits ? p[lane] : make_float2(-INFINITY, 0.f);
     const float2 p1 = lane + 32 < sh.splits ? p[lane + 32] : make_float2(-INFINITY, 0.f);
@@ -299,28 +318,15 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const Window
     if (lane == 0) { s_m[g] = m; s_il[g] = l > 0.f ? 1.0f / l : 0.f; }
   }
   __syncthreads();
-  // this CTA's positions, 32 per warp
-  const int v_begin = (int)((int64_t)nv * crank / csize), v_end = (int)((int64_t)nv * (crank + 1) / csize);
   float* w_w = s_w + warp * 32 * HG;
   int* w_row = s_row + warp * 32;
   float* red = s_red + (size_t)warp * HG * a.vpad;
-  for (int v0 = v_begin + warp * 32; v0 < v_end; v0 += kMixThreads) {
+  for (int v0 = v_begin + warp * 32; v0 < v_end; v0 += nthr) {
     const int v = v0 + lane;
     const bool live = v < v_end;
     const int crow = a.geom.row_of(vr.position(live ? v : v0));
     if (VSM) {
-      constexpr int EP = 16 / (int)sizeof(T);
-      const int pieces = a.vpad / EP;
-      int tr = lane / pieces, c = lane - tr * pieces;
-      const int rstep = 32 / pieces, cstep = 32 - rstep * pieces;
-      for (int i = 0; i < pieces; ++i) {
-        const int src = __shfl_sync(0xffffffffu, crow, tr);
-        cp16(s_v + tr * a.vpad + c * EP, vc + (size_t)src * crow_elems + c * EP);
-        tr += rstep;
-        c += cstep;
-        if (c >= pieces) { c -= pieces; ++tr; }
-      }
-      asm volatile("cp.async.commit_group;" ::: "memory");
+      if (v0 != v_begin + warp * 32) stage(crow);
     } else {
       w_row[lane] = crow;
     }
@@ -357,10 +363,10 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const Window
     __syncwarp();
   }
   __syncthreads();
-  for (int i = tid; i < HG * a.vpad; i += kMixThreads) {
+  for (int i = tid; i < HG * a.vpad; i += nthr) {
     float v = 0.f;
-#pragma unroll
-    for (int q = 0; q < kMixWarps; ++q) v += s_red[(size_t)q * HG * a.vpad + i];
+#pragma unroll 4
+    for (int q = 0; q < nw; ++q) v += s_red[(size_t)q * HG * a.vpad + i];
     s_acc[i] = v;
   }
   // sum over the cluster in rank order; every CTA finishes a slice of the columns
@@ -368,7 +374,7 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const Window
   if (csize > 1) cl.sync();
   else __syncthreads();
   const int total = nh * a.vdim, per = (total + csize - 1) / csize;
-  for (int i = crank * per + tid; i < min(total, (crank + 1) * per); i += kMixThreads) {
+  for (int i = crank * per + tid; i < min(total, (crank + 1) * per); i += nthr) {
     const int h = i / a.vdim, c = i - h * a.vdim;
     float v = 0.f;
     if (csize > 1) {
@@ -379,7 +385,7 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const Window
     act_store1<BF16>(a.out, r, (h0 + h) * a.vdim + c, pos < 0 ? 0.f : v);
   }
   if (h0 + nh == a.heads && crank == 0)
-    for (int k = a.heads * a.vdim + tid; k < a.out.kp; k += kMixThreads) act_store1<BF16>(a.out, r, k, 0.f);
+    for (int k = a.heads * a.vdim + tid; k < a.out.kp; k += nthr) act_store1<BF16>(a.out, r, k, 0.f);
   if (csize > 1) cl.sync();   // nobody leaves while its sums may still be read
 }
 
@@ -402,14 +408,17 @@ tb_status launch_generic(const WindowAttnArgs& a, cudaStream_t st, int* launches
   if (splits > (tiles + warps - 1) / warps) splits = (tiles + warps - 1) / warps;
   if (splits > kScoreSplitsMax) splits = kScoreSplitsMax;
   sh.splits = (int)splits;
-  // mix: query heads of one kv head per CTA, a cluster over the positions
-  const int hg = gq >= 4 ? 4 : (gq >= 2 ? 2 : 1);
-  const int groups = a.kv_heads * ((gq + hg - 1) / hg);
+  // mix: query heads of one kv head per CTA, a cluster over the positions; two smaller CTAs per SM when there are many
+  auto groups_of = [&](int n) { return (int64_t)a.kv_heads * ((gq + n - 1) / n); };
+  int hg = gq >= 4 ? 4 : (gq >= 2 ? 2 : 1);
+  if (hg == 4 && rows * groups_of(4) * 16 <= sm_count()) hg = 2;
+  const int groups = (int)groups_of(hg);
   int cluster = 1;
   while (cluster < 8 && (int64_t)cluster * 64 < a.max_visible && rows * groups * cluster < sm_count()) cluster *= 2;
+  const int mix_threads = rows * groups * cluster > sm_count() || a.max_visible <= 256 * cluster ? 256 : kMixThreads;
   size_t msm = (((size_t)a.heads * 8 + 15) & ~(size_t)15) +
-               4 * ((((size_t)a.heads * hg + 3) & ~(size_t)3) + (size_t)kMixThreads * hg + (size_t)(kMixWarps + 1) * hg * a.vpad + kMixThreads);
-  const size_t vsm = (size_t)kMixThreads * a.vpad * sizeof(T);
+               4 * ((((size_t)a.heads * hg + 3) & ~(size_t)3) + (size_t)mix_threads * hg + (size_t)(mix_threads / 32 + 1) * hg * a.vpad + mix_threads);
+  const size_t vsm = (size_t)mix_threads * a.vpad * sizeof(T);
   const bool staged = msm + vsm <= 220 * 1024;
   if (staged) msm += vsm;
   if (sbytes(warps) > 200 * 1024 || msm > 220 * 1024)
@@ -421,7 +430,7 @@ tb_status launch_generic(const WindowAttnArgs& a, cudaStream_t st, int* launches
     sh.row0 = (int)r0;
     TB_TRY(launch_kernel(window_scores_kernel<T>, dim3((unsigned)sh.splits, (unsigned)a.kv_heads, (unsigned)n), dim3((unsigned)warps * 32),
                          sbytes(warps), st, a.pdl, 1, a, sh));
-    TB_TRY(launch_kernel(mix, dim3((unsigned)cluster, (unsigned)groups, (unsigned)n), dim3(kMixThreads), msm, st, a.pdl, cluster, a, sh));
+    TB_TRY(launch_kernel(mix, dim3((unsigned)cluster, (unsigned)groups, (unsigned)n), dim3((unsigned)mix_threads), msm, st, a.pdl, cluster, a, sh));
     *launches += 2;
   }
   return TB_OK;

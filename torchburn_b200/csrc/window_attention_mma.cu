@@ -80,11 +80,12 @@ struct MmaShape {
   int64_t stride;   // floats per (row, head) of the score scratch
   int row0, rows;   // rows of this pass
   int hg, kvs;      // mix: heads per group, most kv heads a group touches
+  int score_splits; // scores: CTAs that share a query block's keys
   int key_splits;   // mix: CTAs that share a query block's keys
   float* parts;     // [key_splits][rows][heads * vdim] when key_splits > 1
 };
 
-// grid (heads, blocks of 64 queries), 128 threads
+// grid (heads, blocks of 64 queries, score splits), 128 threads
 __global__ void __launch_bounds__(128) window_scores_mma_kernel(const WindowAttnArgs a, const MmaShape sh) {
   extern __shared__ __align__(16) unsigned char s_raw[];
   const int ld = a.dpad + 8;   // row stride in elements: 16 bytes past a multiple of 32 bytes
@@ -122,12 +123,13 @@ __global__ void __launch_bounds__(128) window_scores_mma_kernel(const WindowAttn
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   const int tiles = (keys.count + kKeys - 1) / kKeys;
-  fetch(0);
+  const int t0 = (int)((int64_t)tiles * blockIdx.z / sh.score_splits), t1 = (int)((int64_t)tiles * (blockIdx.z + 1) / sh.score_splits);
+  if (t0 < t1) fetch(t0);
   // the warp's 16 queries: this thread holds rows lane / 4 and lane / 4 + 8, key columns 2 (lane & 3) and the next
   const int qr[2] = {warp * 16 + (lane >> 2), warp * 16 + (lane >> 2) + 8};
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
-  for (int t = 0; t < tiles; ++t) {
-    if (t + 1 < tiles) {
+  for (int t = t0; t < t1; ++t) {
+    if (t + 1 < t1) {
       fetch(t + 1);
       asm volatile("cp.async.wait_group 1;" ::: "memory");
     } else {
@@ -194,7 +196,7 @@ __global__ void __launch_bounds__(128) window_scores_mma_kernel(const WindowAttn
     l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
     l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
     if ((lane & 3) == 0 && qr[e] < nrows) {
-      float* p = a.part + ((size_t)(b0 + qr[e]) * a.heads + h) * 2;
+      float* p = a.part + (((size_t)(b0 + qr[e]) * a.heads + h) * sh.score_splits + blockIdx.z) * 2;
       p[0] = m[e];
       p[1] = l[e];
     }
@@ -233,8 +235,14 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_mma_kernel(const Wi
     const int g = i / kQM, q = i - g * kQM;
     float2 v = make_float2(INFINITY, 0.f);           // a dead row's weights are exp(-inf) = 0
     if (q < nrows && g < a.heads) {
-      const float* p = a.part + ((size_t)(q0 + q) * a.heads + g) * 2;
-      v = make_float2(p[0], 1.0f / p[1]);
+      const float* p = a.part + ((size_t)(q0 + q) * a.heads + g) * sh.score_splits * 2;
+      float m = p[0], l = p[1];
+      for (int z = 1; z < sh.score_splits; ++z) {      // in order
+        const float m2 = p[2 * z], l2 = p[2 * z + 1], m1 = fmaxf(m, m2);
+        l = (m == -INFINITY ? 0.f : l * expf(m - m1)) + (m2 == -INFINITY ? 0.f : l2 * expf(m2 - m1));
+        m = m1;
+      }
+      v = make_float2(m, 1.0f / l);
     }
     s_ml[i] = v;
   }
@@ -431,7 +439,10 @@ tb_status launch_window_attention_mma(const WindowAttnArgs& a, cudaStream_t st, 
   for (int64_t r0 = 0; r0 < a.r.rows; r0 += pass) {
     sh.row0 = (int)r0;
     sh.rows = (int)(a.r.rows - r0 < pass ? a.r.rows - r0 : pass);
-    TB_TRY(launch_kernel(window_scores_mma_kernel, dim3((unsigned)a.heads, (unsigned)((sh.rows + kQB - 1) / kQB)), dim3(128), ssm, st, a.pdl, 1, a, sh));
+    const int64_t qb = (sh.rows + kQB - 1) / kQB;
+    sh.score_splits = 1;
+    while (sh.score_splits < 8 && a.heads * qb * sh.score_splits < 4 * sm_count() && a.max_visible >= (int64_t)kKeys * 4 * sh.score_splits) sh.score_splits *= 2;
+    TB_TRY(launch_kernel(window_scores_mma_kernel, dim3((unsigned)a.heads, (unsigned)qb, (unsigned)sh.score_splits), dim3(128), ssm, st, a.pdl, 1, a, sh));
     const int qblocks = (sh.rows + kQM - 1) / kQM;
     sh.key_splits = 1;
     while (a.parts != nullptr && sh.key_splits < kMaxKeySplits && groups * qblocks * sh.key_splits * 3 / 2 < sm_count() &&

@@ -217,7 +217,8 @@ struct WindowAttnArgs {
   float* scores = nullptr;               // scratch [rows of a pass][heads][score_stride]
   float* part = nullptr;                 // scratch [rows of a pass][heads][splits][2]
   int64_t scratch_rows = 0;
-  float* parts = nullptr;                // scratch of window_parts_floats(), tensor-core form only; null: never split
+  float* parts = nullptr;                // scratch [parts_rows][heads * vdim]: sums of CTAs that share a row's positions
+  int64_t parts_rows = 0;                // rows x splits it holds
   ActOperand out;                        // K = heads * vdim
   bool one_sequence = false;             // the rows are consecutive positions of one sequence
   bool pdl = false;
@@ -225,8 +226,8 @@ struct WindowAttnArgs {
 constexpr int kScoreSplitsMax = 64;
 size_t window_attn_score_stride(int64_t max_visible);
 tb_status launch_window_attention(Precision p, const WindowAttnArgs& a, cudaStream_t st, int* launches);
+tb_status launch_window_parts(Precision p, const WindowAttnArgs& a, int splits, int row0, int rows, cudaStream_t st);
 // Tensor-core form for a portion of one sequence (window_attention_mma.cu); reads q16, not q.
-size_t window_parts_floats(int rows, int64_t cols);
 bool window_mma_supported(const WindowAttnArgs& a);
 tb_status launch_window_attention_mma(const WindowAttnArgs& a, cudaStream_t st, int* launches);
 

@@ -87,8 +87,9 @@ struct LayeredModel {
   float* q = nullptr;
   __nv_bfloat16* q16 = nullptr;
   float *scores = nullptr, *part = nullptr;
-  int64_t score_floats = 0, part_rows = 0;
-  float* parts = nullptr;          // attention sums of key splits
+  int64_t score_floats = 0;
+  float* parts = nullptr;          // attention sums of CTAs that share a row's positions
+  int64_t parts_rows = 0;
   float* snap = nullptr;
   int64_t rollback = 0;
   std::vector<void*> owned;        // every device allocation
@@ -285,11 +286,12 @@ tb_status create_impl(LayeredModel* m, const tb_layered_layer* layers, const uin
   int64_t srows = (int64_t)(kScoreBudget / 4) / max_score_row;
   if (srows < 1) srows = 1;
   if (srows > R) srows = R;
-  m->part_rows = R;
+  
   m->score_floats = srows * max_score_row;
   TB_TRY(dev_alloc(m, &m->scores, (size_t)m->score_floats, false));
   TB_TRY(dev_alloc(m, &m->part, (size_t)(R * max_heads * kScoreSplitsMax * 2), false));
-  if (m->prec == Precision::kBf16) TB_TRY(dev_alloc(m, &m->parts, window_parts_floats(R, max_o), false));
+  m->parts_rows = 4 * R > 4 * kScoreSplitsMax ? 4 * R : 4 * kScoreSplitsMax;
+  TB_TRY(dev_alloc(m, &m->parts, (size_t)m->parts_rows * max_o, false));
   if (snapshots) TB_TRY(dev_alloc(m, &m->snap, (size_t)m->L * R * m->xs, true));
   TB_CUDA_TRY(cudaDeviceSynchronize());
   return TB_OK;
@@ -418,7 +420,7 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
     wa.r = r; wa.k_cache = run.k_cache; wa.v_cache = run.v_cache; wa.geom = run.geom;
     wa.heads = w.heads; wa.kv_heads = w.kv_heads; wa.dim = w.dim; wa.vdim = w.vdim; wa.dpad = w.dpad; wa.vpad = w.vpad;
     wa.scale = run.scale; wa.window = run.window; wa.keep_first = run.keep_first; wa.talk = w.talk; wa.max_visible = run.max_visible;
-    wa.scores = m->scores; wa.part = m->part; wa.parts = m->parts;
+    wa.scores = m->scores; wa.part = m->part; wa.parts = m->parts; wa.parts_rows = m->parts_rows;
     wa.scratch_rows = m->score_floats / ((int64_t)w.heads * (int64_t)window_attn_score_stride(run.max_visible));
     wa.out = ActOperand{m->act_o, mp, (int)w.o.kp};
     wa.one_sequence = s.one_sequence; wa.pdl = s.pdl;

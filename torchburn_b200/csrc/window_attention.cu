@@ -7,24 +7,20 @@
 //
 //   scores   raw scores of every (row, head, visible position) -> scratch, with the running (max, sum) of
 //            each CTA's share of the positions
-//   mix      weights = exp(score - max) / sum, mixed over the heads, times the values; a cluster of CTAs
-//            shares a row's positions and adds its parts through distributed shared memory in rank order
+//   mix      weights = exp(score - max) / sum, mixed over the heads, times the values.  The weights are
+//            normalised, so CTAs that share a row's positions leave plain sums, added in order by a last kernel
 //
-// Both read the cache once.  These two serve decode steps (any number of sequences) in both precisions and
+// Each half of the cache is read once.  These two serve decode steps (any number of sequences) in both precisions and
 // whole portions in fp32; portions in bf16 take the tensor-core kernels in window_attention_mma.cu.
-#include <cooperative_groups.h>
-
 #include "dense.cuh"
 #include "window_attention.cuh"
-
-namespace cg = cooperative_groups;
 
 namespace tb {
 
 namespace {
 
 constexpr int kTileP = 32;        // positions per tile: one per lane
-constexpr int kMixThreads = 512;  // most threads of a mix CTA
+constexpr int kMixThreads = 256;
 constexpr int kHeadChunk = 4;     // query heads that share a key's load
 
 __device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
@@ -49,7 +45,7 @@ __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], 
 struct ScoreShape {
   int splits;       // CTAs that share a row's positions
   int64_t stride;   // floats per (row, head) of the score scratch
-  int row0;
+  int row0, rows;   // rows of this pass
 };
 
 // Bytes of the queries of one kv head in shared memory.  fp32: [heads][dpad].  bf16: per four heads eight rows
@@ -253,11 +249,11 @@ __device__ __forceinline__ void warp_values(const T* vals, const int* rows, int6
   }
 }
 
-// grid (cluster size, head groups, rows): HG query heads of one kv head per CTA.  A warp takes 32 positions at a
+// grid (position splits, head groups, rows): HG query heads of one kv head per CTA.  A warp takes 32 positions at a
 // time and needs no other: their values by cp.async into the warp's tile (VSM) while a lane takes one position
 // through all heads (weights and mixing, in registers), then the lanes are the value columns.
 template <typename T, bool BF16, int HG, bool VSM>
-__global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const WindowAttnArgs a, const ScoreShape sh) {
+__global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const WindowAttnArgs a, const ScoreShape sh) {
   extern __shared__ __align__(16) unsigned char s_raw[];
   const int gq = a.heads / a.kv_heads, per_kv = (gq + HG - 1) / HG;
   const int kv = (int)blockIdx.y / per_kv, sub = (int)blockIdx.y - kv * per_kv;
@@ -272,7 +268,7 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const Window
   int* s_row = reinterpret_cast<int*>(s_acc + HG * a.vpad);                    // [32 warps] cache rows
   T* s_v = reinterpret_cast<T*>(s_row + blockDim.x) + (size_t)(threadIdx.x >> 5) * 32 * a.vpad;   // the warp's values when VSM
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nthr = (int)blockDim.x, nw = nthr >> 5;
-  const int csize = (int)gridDim.x, crank = (int)blockIdx.x;
+  const int csize = (int)gridDim.x, crank = (int)blockIdx.x;   // CTAs that share the row's positions
   grid_dep_launch();
   for (int i = tid; i < a.heads * HG; i += nthr) {
     const int g = i / HG, h = i - g * HG;
@@ -369,24 +365,17 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_kernel(const Window
     for (int q = 0; q < nw; ++q) v += s_red[(size_t)q * HG * a.vpad + i];
     s_acc[i] = v;
   }
-  // sum over the cluster in rank order; every CTA finishes a slice of the columns
-  cg::cluster_group cl = cg::this_cluster();
-  if (csize > 1) cl.sync();
-  else __syncthreads();
-  const int total = nh * a.vdim, per = (total + csize - 1) / csize;
-  for (int i = crank * per + tid; i < min(total, (crank + 1) * per); i += nthr) {
+  __syncthreads();
+  const int total = nh * a.vdim;
+  for (int i = tid; i < total; i += nthr) {
     const int h = i / a.vdim, c = i - h * a.vdim;
-    float v = 0.f;
-    if (csize > 1) {
-      for (int q = 0; q < csize; ++q) v += *cl.map_shared_rank(&s_acc[h * a.vpad + c], q);
-    } else {
-      v = s_acc[h * a.vpad + c];
-    }
-    act_store1<BF16>(a.out, r, (h0 + h) * a.vdim + c, pos < 0 ? 0.f : v);
+    const float v = pos < 0 ? 0.f : s_acc[h * a.vpad + c];
+    const int k = (h0 + h) * a.vdim + c;
+    if (csize > 1) a.parts[((size_t)crank * sh.rows + lr) * ((size_t)a.heads * a.vdim) + k] = v;
+    else act_store1<BF16>(a.out, r, k, v);
   }
-  if (h0 + nh == a.heads && crank == 0)
+  if (csize == 1 && h0 + nh == a.heads)
     for (int k = a.heads * a.vdim + tid; k < a.out.kp; k += nthr) act_store1<BF16>(a.out, r, k, 0.f);
-  if (csize > 1) cl.sync();   // nobody leaves while its sums may still be read
 }
 
 template <typename T, bool BF16>
@@ -408,17 +397,16 @@ tb_status launch_generic(const WindowAttnArgs& a, cudaStream_t st, int* launches
   if (splits > (tiles + warps - 1) / warps) splits = (tiles + warps - 1) / warps;
   if (splits > kScoreSplitsMax) splits = kScoreSplitsMax;
   sh.splits = (int)splits;
-  // mix: query heads of one kv head per CTA, a cluster over the positions; two smaller CTAs per SM when there are many
-  auto groups_of = [&](int n) { return (int64_t)a.kv_heads * ((gq + n - 1) / n); };
-  int hg = gq >= 4 ? 4 : (gq >= 2 ? 2 : 1);
-  if (hg == 4 && rows * groups_of(4) * 16 <= sm_count()) hg = 2;
-  const int groups = (int)groups_of(hg);
-  int cluster = 1;
-  while (cluster < 8 && (int64_t)cluster * 64 < a.max_visible && rows * groups * cluster < sm_count()) cluster *= 2;
-  const int mix_threads = rows * groups * cluster > sm_count() || a.max_visible <= 256 * cluster ? 256 : kMixThreads;
+  // mix: query heads of one kv head per CTA; up to two CTAs per SM share a row's positions
+  const int hg = gq >= 4 ? 4 : (gq >= 2 ? 2 : 1);
+  const int groups = a.kv_heads * ((gq + hg - 1) / hg);
+  int64_t mix_splits = 2 * sm_count() / (rows * groups);
+  if (mix_splits > (a.max_visible + kMixThreads - 1) / kMixThreads) mix_splits = (a.max_visible + kMixThreads - 1) / kMixThreads;
+  if (mix_splits > a.parts_rows / rows) mix_splits = a.parts_rows / rows;
+  if (mix_splits < 1) mix_splits = 1;
   size_t msm = (((size_t)a.heads * 8 + 15) & ~(size_t)15) +
-               4 * ((((size_t)a.heads * hg + 3) & ~(size_t)3) + (size_t)mix_threads * hg + (size_t)(mix_threads / 32 + 1) * hg * a.vpad + mix_threads);
-  const size_t vsm = (size_t)mix_threads * a.vpad * sizeof(T);
+               4 * ((((size_t)a.heads * hg + 3) & ~(size_t)3) + (size_t)kMixThreads * hg + (size_t)(kMixThreads / 32 + 1) * hg * a.vpad + kMixThreads);
+  const size_t vsm = (size_t)kMixThreads * a.vpad * sizeof(T);
   const bool staged = msm + vsm <= 220 * 1024;
   if (staged) msm += vsm;
   if (sbytes(warps) > 200 * 1024 || msm > 220 * 1024)
@@ -428,15 +416,41 @@ tb_status launch_generic(const WindowAttnArgs& a, cudaStream_t st, int* launches
   for (int64_t r0 = 0; r0 < a.r.rows; r0 += pass) {
     const int n = (int)(a.r.rows - r0 < pass ? a.r.rows - r0 : pass);
     sh.row0 = (int)r0;
+    sh.rows = n;
     TB_TRY(launch_kernel(window_scores_kernel<T>, dim3((unsigned)sh.splits, (unsigned)a.kv_heads, (unsigned)n), dim3((unsigned)warps * 32),
                          sbytes(warps), st, a.pdl, 1, a, sh));
-    TB_TRY(launch_kernel(mix, dim3((unsigned)cluster, (unsigned)groups, (unsigned)n), dim3((unsigned)mix_threads), msm, st, a.pdl, cluster, a, sh));
+    TB_TRY(launch_kernel(mix, dim3((unsigned)mix_splits, (unsigned)groups, (unsigned)n), dim3(kMixThreads), msm, st, a.pdl, 1, a, sh));
     *launches += 2;
+    if (mix_splits > 1) {
+      TB_TRY(launch_window_parts(BF16 ? Precision::kBf16 : Precision::kF32, a, (int)mix_splits, (int)r0, n, st));
+      ++*launches;
+    }
   }
   return TB_OK;
 }
 
+// Sums over the splits of a row's positions, in order, as the next projection's operand.  grid (rows, columns / 256)
+template <bool BF16>
+__global__ void __launch_bounds__(256) window_parts_kernel(const WindowAttnArgs a, const int splits, const int row0, const int rows) {
+  grid_dep_launch();
+  grid_dep_wait();
+  const int q = (int)blockIdx.x, k = (int)blockIdx.y * 256 + threadIdx.x, cols = a.heads * a.vdim;
+  if (k >= a.out.kp) return;
+  float v = 0.f;
+  if (k < cols) {
+#pragma unroll 8
+    for (int z = 0; z < splits; ++z) v += a.parts[((size_t)z * rows + q) * cols + k];
+  }
+  act_store1<BF16>(a.out, row0 + q, k, v);
+}
+
 }  // namespace
+
+tb_status launch_window_parts(Precision p, const WindowAttnArgs& a, int splits, int row0, int rows, cudaStream_t st) {
+  const dim3 grid((unsigned)rows, (unsigned)((a.out.kp + 255) / 256));
+  return p == Precision::kBf16 ? launch_kernel(window_parts_kernel<true>, grid, dim3(256), 0, st, a.pdl, 1, a, splits, row0, rows)
+                               : launch_kernel(window_parts_kernel<false>, grid, dim3(256), 0, st, a.pdl, 1, a, splits, row0, rows);
+}
 
 size_t window_attn_score_stride(int64_t max_visible) {
   // the tensor-core form numbers keys per block of 64 queries: up to 63 more than one row sees

@@ -82,7 +82,6 @@ struct MmaShape {
   int hg, kvs;      // mix: heads per group, most kv heads a group touches
   int score_splits; // scores: CTAs that share a query block's keys
   int key_splits;   // mix: CTAs that share a query block's keys
-  float* parts;     // [key_splits][rows][heads * vdim] when key_splits > 1
 };
 
 // grid (heads, blocks of 64 queries, score splits), 128 threads
@@ -377,25 +376,13 @@ __global__ void __launch_bounds__(kMixThreads, 1) window_mix_mma_kernel(const Wi
         const int q = (lane >> 2) + (i >> 1) * 8, col = c + j * 8 + (lane & 3) * 2 + (i & 1);
         if (q >= nrows || col >= a.vdim) continue;
         const int k = (h0 + h) * a.vdim + col;
-        if (sh.key_splits > 1) sh.parts[((size_t)blockIdx.z * sh.rows + q0 + q) * cols + k] = acc[u][j][i];
+        if (sh.key_splits > 1) a.parts[((size_t)blockIdx.z * sh.rows + q0 + q) * cols + k] = acc[u][j][i];
         else act_store1<true>(a.out, sh.row0 + q0 + q, k, acc[u][j][i]);
       }
   }
   if (sh.key_splits == 1 && h0 + nh == a.heads)
     for (int q = 0; q < nrows; ++q)
       for (int k = cols + tid; k < a.out.kp; k += kMixThreads) act_store1<true>(a.out, sh.row0 + q0 + q, k, 0.f);
-}
-
-// The key splits' parts, added in order.  grid (rows, columns / 256)
-__global__ void __launch_bounds__(256) window_parts_kernel(const WindowAttnArgs a, const MmaShape sh) {
-  grid_dep_launch();
-  grid_dep_wait();
-  const int q = (int)blockIdx.x, k = (int)blockIdx.y * 256 + threadIdx.x, cols = a.heads * a.vdim;
-  if (k >= a.out.kp) return;
-  float v = 0.f;
-  if (k < cols)
-    for (int z = 0; z < sh.key_splits; ++z) v += sh.parts[((size_t)z * sh.rows + q) * cols + k];
-  act_store1<true>(a.out, sh.row0 + q, k, v);
 }
 
 size_t mix_bytes(const WindowAttnArgs& a, int hg, int kvs, bool staged) {
@@ -417,9 +404,6 @@ bool window_mma_supported(const WindowAttnArgs& a) {
          mix_bytes(a, 1, 1, false) <= kSmemMax;
 }
 
-// Floats of WindowAttnArgs::parts for steps of up to `rows` rows.
-size_t window_parts_floats(int rows, int64_t cols) { return (size_t)kMaxKeySplits * rows * cols; }
-
 tb_status launch_window_attention_mma(const WindowAttnArgs& a, cudaStream_t st, int* launches) {
   // heads per group: as many as one MMA holds and accumulators and shared memory allow
   int hg = 16;
@@ -428,7 +412,6 @@ tb_status launch_window_attention_mma(const WindowAttnArgs& a, cudaStream_t st, 
   sh.hg = hg;
   sh.kvs = group_kv_heads(a, hg);
   sh.stride = (int64_t)window_attn_score_stride(a.max_visible);
-  sh.parts = a.parts;
   const bool staged = mix_bytes(a, hg, sh.kvs, true) <= kSmemMax;
   // passes of equal size, in whole query blocks, as many rows as the score scratch holds
   const int64_t blocks = (a.r.rows + kQB - 1) / kQB, fit = a.scratch_rows / kQB;
@@ -445,14 +428,14 @@ tb_status launch_window_attention_mma(const WindowAttnArgs& a, cudaStream_t st, 
     TB_TRY(launch_kernel(window_scores_mma_kernel, dim3((unsigned)a.heads, (unsigned)qb, (unsigned)sh.score_splits), dim3(128), ssm, st, a.pdl, 1, a, sh));
     const int qblocks = (sh.rows + kQM - 1) / kQM;
     sh.key_splits = 1;
-    while (a.parts != nullptr && sh.key_splits < kMaxKeySplits && groups * qblocks * sh.key_splits * 3 / 2 < sm_count() &&
+    while (sh.key_splits < kMaxKeySplits && a.parts_rows >= 2 * (int64_t)sh.rows * sh.key_splits && groups * qblocks * sh.key_splits * 3 / 2 < sm_count() &&
            a.max_visible >= (int64_t)kKT * 8 * sh.key_splits)
       sh.key_splits *= 2;
     auto* kern = staged ? window_mix_mma_kernel<true> : window_mix_mma_kernel<false>;
     TB_TRY(launch_kernel(kern, dim3((unsigned)groups, (unsigned)qblocks, (unsigned)sh.key_splits), dim3(kMixThreads), msm, st, a.pdl, 1, a, sh));
     *launches += 2;
     if (sh.key_splits > 1) {
-      TB_TRY(launch_kernel(window_parts_kernel, dim3((unsigned)sh.rows, (unsigned)((a.out.kp + 255) / 256)), dim3(256), 0, st, a.pdl, 1, a, sh));
+      TB_TRY(launch_window_parts(Precision::kBf16, a, sh.key_splits, sh.row0, sh.rows, st));
       ++*launches;
     }
   }

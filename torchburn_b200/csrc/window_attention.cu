@@ -36,6 +36,10 @@ __device__ __forceinline__ void ldm4(uint32_t (&r)[4], const void* p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
 }
+__device__ __forceinline__ void ldm4t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"((uint32_t)__cvta_generic_to_shared(p)));
+}
 __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
@@ -252,7 +256,8 @@ __device__ __forceinline__ void warp_values(const T* vals, const int* rows, int6
 // grid (position splits, head groups, rows): HG query heads of one kv head per CTA.  A warp takes 32 positions at a
 // time and needs no other: their values by cp.async into the warp's tile (VSM) while a lane takes one position
 // through all heads (weights and mixing, in registers), then the lanes are the value columns.
-template <typename T, bool BF16, int HG, bool VSM>
+// VSM: 0 values from global memory, 1 staged, fp32 products, 2 staged, mma.sync (bf16, at most 128 columns).
+template <typename T, bool BF16, int HG, int VSM>
 __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const WindowAttnArgs a, const ScoreShape sh) {
   extern __shared__ __align__(16) unsigned char s_raw[];
   const int gq = a.heads / a.kv_heads, per_kv = (gq + HG - 1) / HG;
@@ -266,7 +271,8 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
   float* s_red = s_w + blockDim.x * HG;                                       // [warps][HG][vpad]
   float* s_acc = s_red + (size_t)(blockDim.x >> 5) * HG * a.vpad;                      // [HG][vpad]
   int* s_row = reinterpret_cast<int*>(s_acc + HG * a.vpad);                    // [32 warps] cache rows
-  T* s_v = reinterpret_cast<T*>(s_row + blockDim.x) + (size_t)(threadIdx.x >> 5) * 32 * a.vpad;   // the warp's values when VSM
+  const int vld = a.vpad + (VSM == 2 ? 8 : 0);
+  T* s_v = reinterpret_cast<T*>(s_row + blockDim.x) + (size_t)(threadIdx.x >> 5) * 32 * vld;   // the warp's values when VSM
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nthr = (int)blockDim.x, nw = nthr >> 5;
   const int csize = (int)gridDim.x, crank = (int)blockIdx.x;   // CTAs that share the row's positions
   grid_dep_launch();
@@ -290,7 +296,7 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
     const int rstep = 32 / pieces, cstep = 32 - rstep * pieces;
     for (int i = 0; i < pieces; ++i) {
       const int src = __shfl_sync(0xffffffffu, crow, tr);
-      cp16(s_v + tr * a.vpad + c * EP, vc + (size_t)src * crow_elems + c * EP);
+      cp16(s_v + tr * vld + c * EP, vc + (size_t)src * crow_elems + c * EP);
       tr += rstep;
       c += cstep;
       if (c >= pieces) { c -= pieces; ++tr; }
@@ -301,22 +307,53 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
     const int v = v_begin + warp * 32 + lane;
     stage(a.geom.row_of(vr.position(v < v_end ? v : v_begin + warp * 32)));
   }
-  for (int g = warp; g < a.heads; g += nw) {   // softmax statistics from the parts, in a fixed order
-    const float2* p = reinterpret_cast<const float2*>(a.part) + ((size_t)lr * a.heads + g) * sh.splits;
-    const float2 p0 = lane < sh.splits ? p[lane] : make_float2(-INFINITY, 0.f);
-    const float2 p1 = lane + 32 < sh.splits ? p[lane + 32] : make_float2(-INFINITY, 0.f);
-    float m = fmaxf(p0.x, p1.x);
+  constexpr int GB = 16;                      // heads whose scores are requested together
+  float pre[GB];                              // the first ones of the first positions
+  const float* score_row = a.scores + (size_t)lr * a.heads * sh.stride;
+  {
+    const int v = v_begin + warp * 32 + lane;
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-    float l = (p0.x == -INFINITY ? 0.f : p0.y * expf(p0.x - m)) + (p1.x == -INFINITY ? 0.f : p1.y * expf(p1.x - m));
+    for (int j = 0; j < GB; ++j) pre[j] = j < a.heads && v < v_end ? score_row[(size_t)j * sh.stride + v] : 0.f;
+  }
+  constexpr int SB = 4;                       // softmax statistics from the parts, in a fixed order; SB heads in flight
+  for (int g0 = warp * SB; g0 < a.heads; g0 += nw * SB) {
+    float2 p0[SB], p1[SB];
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-    if (lane == 0) { s_m[g] = m; s_il[g] = l > 0.f ? 1.0f / l : 0.f; }
+    for (int j = 0; j < SB; ++j) {
+      const float2* p = reinterpret_cast<const float2*>(a.part) + ((size_t)lr * a.heads + g0 + j) * sh.splits;
+      p0[j] = p1[j] = make_float2(-INFINITY, 0.f);
+      if (g0 + j < a.heads && lane < sh.splits) p0[j] = p[lane];
+      if (g0 + j < a.heads && lane + 32 < sh.splits) p1[j] = p[lane + 32];
+    }
+    float m[SB], l[SB];
+#pragma unroll
+    for (int j = 0; j < SB; ++j) m[j] = fmaxf(p0[j].x, p1[j].x);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+      for (int j = 0; j < SB; ++j) m[j] = fmaxf(m[j], __shfl_xor_sync(0xffffffffu, m[j], o));
+#pragma unroll
+    for (int j = 0; j < SB; ++j)
+      l[j] = (p0[j].x == -INFINITY ? 0.f : p0[j].y * expf(p0[j].x - m[j])) + (p1[j].x == -INFINITY ? 0.f : p1[j].y * expf(p1[j].x - m[j]));
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+      for (int j = 0; j < SB; ++j) l[j] += __shfl_xor_sync(0xffffffffu, l[j], o);
+    if (lane == 0)
+#pragma unroll
+      for (int j = 0; j < SB; ++j)
+        if (g0 + j < a.heads) { s_m[g0 + j] = m[j]; s_il[g0 + j] = l[j] > 0.f ? 1.0f / l[j] : 0.f; }
   }
   __syncthreads();
   float* w_w = s_w + warp * 32 * HG;
   int* w_row = s_row + warp * 32;
   float* red = s_red + (size_t)warp * HG * a.vpad;
+  constexpr int NT = VSM == 2 ? 16 : 1;       // 8-column tiles
+  float acc[NT][4];
+#pragma unroll
+  for (int n = 0; n < NT; ++n)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[n][i] = 0.f;
   for (int v0 = v_begin + warp * 32; v0 < v_end; v0 += nthr) {
     const int v = v0 + lane;
     const bool live = v < v_end;
@@ -326,15 +363,15 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
     } else {
       w_row[lane] = crow;
     }
-    const float* sp = a.scores + (size_t)lr * a.heads * sh.stride + (live ? v : v0);
+    const float* sp = score_row + (live ? v : v0);
+    const bool first = v0 == v_begin + warp * 32;
     float w[HG];
 #pragma unroll
     for (int h = 0; h < HG; ++h) w[h] = 0.f;
-    constexpr int GB = 16;
     for (int g0 = 0; g0 < a.heads; g0 += GB) {
       float s8[GB];
 #pragma unroll
-      for (int j = 0; j < GB; ++j) s8[j] = g0 + j < a.heads ? sp[(size_t)(g0 + j) * sh.stride] : 0.f;
+      for (int j = 0; j < GB; ++j) s8[j] = first && g0 == 0 ? pre[j] : (g0 + j < a.heads ? sp[(size_t)(g0 + j) * sh.stride] : 0.f);
 #pragma unroll
       for (int j = 0; j < GB; ++j) {
         const int g = g0 + j;
@@ -350,13 +387,47 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
     if (VSM) asm volatile("cp.async.wait_all;" ::: "memory");
     __syncwarp();
     const int nj = min(32, v_end - v0);
-    if (VSM) {
+    if constexpr (VSM == 2) {
+      // rows 0-3 of A: the weights of the heads rounded to bf16, rows 4-7: what the rounding left
+      const int hr = (lane >> 2) & 3;
+      const bool rest = lane >= 16;
+#pragma unroll
+      for (int kk = 0; kk < 32; kk += 16) {
+        uint32_t wa[4] = {0u, 0u, 0u, 0u};
+#pragma unroll
+        for (int x = 0; x < 2; ++x) {
+          const int key = kk + x * 8 + (lane & 3) * 2;
+          const float w0 = hr < HG && key < nj ? w_w[key * HG + hr] : 0.f, w1 = hr < HG && key + 1 < nj ? w_w[(key + 1) * HG + hr] : 0.f;
+          const __nv_bfloat162 hi = __floats2bfloat162_rn(w0, w1);
+          const float2 hf = __bfloat1622float2(hi);
+          const __nv_bfloat162 lo = __floats2bfloat162_rn(w0 - hf.x, w1 - hf.y);
+          wa[2 * x] = rest ? *reinterpret_cast<const uint32_t*>(&lo) : *reinterpret_cast<const uint32_t*>(&hi);
+        }
+#pragma unroll
+        for (int n = 0; n < NT; n += 2) {
+          if (n * 8 >= a.vpad) break;
+          uint32_t vb[4];
+          ldm4t(vb, s_v + (kk + (lane & 15)) * vld + n * 8 + (lane >> 4) * 8);
+          mma16816(acc[n], wa, vb[0], vb[1]);
+          mma16816(acc[n + 1 < NT ? n + 1 : n], wa, vb[2], vb[3]);
+        }
+      }
+    } else if (VSM) {
       if (a.vpad > 64) warp_values<T, HG, 4>(s_v, nullptr, a.vpad, w_w, nj, a.vpad, red);
       else warp_values<T, HG, 2>(s_v, nullptr, a.vpad, w_w, nj, a.vpad, red);
     } else {
       warp_values<T, HG, 2>(vc, w_row, crow_elems, w_w, nj, a.vpad, red);
     }
     __syncwarp();
+  }
+  if constexpr (VSM == 2) {   // the two pieces' sums, into the warp's row sums
+#pragma unroll
+    for (int n = 0; n < NT; ++n)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const float v = acc[n][i] + __shfl_xor_sync(0xffffffffu, acc[n][i], 16);
+        if (lane < 16 && (lane >> 2) < HG && n * 8 < a.vpad) red[(lane >> 2) * a.vpad + n * 8 + (lane & 3) * 2 + i] = v;
+      }
   }
   __syncthreads();
   for (int i = tid; i < HG * a.vpad; i += nthr) {
@@ -406,13 +477,17 @@ tb_status launch_generic(const WindowAttnArgs& a, cudaStream_t st, int* launches
   if (mix_splits < 1) mix_splits = 1;
   size_t msm = (((size_t)a.heads * 8 + 15) & ~(size_t)15) +
                4 * ((((size_t)a.heads * hg + 3) & ~(size_t)3) + (size_t)kMixThreads * hg + (size_t)(kMixThreads / 32 + 1) * hg * a.vpad + kMixThreads);
-  const size_t vsm = (size_t)kMixThreads * a.vpad * sizeof(T);
+  const bool tensor = sizeof(T) == 2 && a.vpad <= 128;
+  const size_t vsm = (size_t)kMixThreads * (a.vpad + (tensor ? 8 : 0)) * sizeof(T);
   const bool staged = msm + vsm <= 220 * 1024;
   if (staged) msm += vsm;
   if (sbytes(warps) > 200 * 1024 || msm > 220 * 1024)
     return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: attention with %d heads of size %d/%d", a.heads, a.dim, a.vdim);
-  auto* mix = staged ? (hg == 4 ? window_mix_kernel<T, BF16, 4, true> : (hg == 2 ? window_mix_kernel<T, BF16, 2, true> : window_mix_kernel<T, BF16, 1, true>))
-                     : (hg == 4 ? window_mix_kernel<T, BF16, 4, false> : (hg == 2 ? window_mix_kernel<T, BF16, 2, false> : window_mix_kernel<T, BF16, 1, false>));
+  void (*mix)(WindowAttnArgs, ScoreShape) =
+      staged ? (hg == 4 ? window_mix_kernel<T, BF16, 4, 1> : (hg == 2 ? window_mix_kernel<T, BF16, 2, 1> : window_mix_kernel<T, BF16, 1, 1>))
+             : (hg == 4 ? window_mix_kernel<T, BF16, 4, 0> : (hg == 2 ? window_mix_kernel<T, BF16, 2, 0> : window_mix_kernel<T, BF16, 1, 0>));
+  if constexpr (sizeof(T) == 2)
+    if (staged && tensor) mix = hg == 4 ? window_mix_kernel<T, BF16, 4, 2> : (hg == 2 ? window_mix_kernel<T, BF16, 2, 2> : window_mix_kernel<T, BF16, 1, 2>);
   for (int64_t r0 = 0; r0 < a.r.rows; r0 += pass) {
     const int n = (int)(a.r.rows - r0 < pass ? a.r.rows - r0 : pass);
     sh.row0 = (int)r0;

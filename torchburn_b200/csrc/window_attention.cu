@@ -21,6 +21,7 @@ namespace {
 
 constexpr int kTileP = 32;        // positions per tile: one per lane
 constexpr int kMixThreads = 256;
+constexpr float kLog2E = 1.44269504f;
 constexpr int kHeadChunk = 4;     // query heads that share a key's load
 
 __device__ __forceinline__ float2 load2(const float* p) { return *reinterpret_cast<const float2*>(p); }
@@ -91,7 +92,7 @@ __global__ void __launch_bounds__(256) window_scores_kernel(const WindowAttnArgs
     const int rstep = 32 / pieces, cstep = 32 - rstep * pieces;
     for (int i = 0; i < pieces; ++i) {   // 32 * pieces copies, 32 at a time
       const int src = __shfl_sync(0xffffffffu, crow, tr);
-      cp16(s_k + tr * stride + c * EP, kc + (size_t)src * crow_elems + c * EP);
+      cp16(s_k + tr * stride + c * EP, kc + (size_t)(uint32_t)src * (uint32_t)crow_elems + c * EP);
       tr += rstep;
       c += cstep;
       if (c >= pieces) { c -= pieces; ++tr; }
@@ -296,7 +297,7 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
     const int rstep = 32 / pieces, cstep = 32 - rstep * pieces;
     for (int i = 0; i < pieces; ++i) {
       const int src = __shfl_sync(0xffffffffu, crow, tr);
-      cp16(s_v + tr * vld + c * EP, vc + (size_t)src * crow_elems + c * EP);
+      cp16(s_v + tr * vld + c * EP, vc + (size_t)(uint32_t)src * (uint32_t)crow_elems + c * EP);
       tr += rstep;
       c += cstep;
       if (c >= pieces) { c -= pieces; ++tr; }
@@ -342,7 +343,11 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
     if (lane == 0)
 #pragma unroll
       for (int j = 0; j < SB; ++j)
-        if (g0 + j < a.heads) { s_m[g0 + j] = m[j]; s_il[g0 + j] = l[j] > 0.f ? 1.0f / l[j] : 0.f; }
+        if (g0 + j < a.heads) {
+          // bf16: exp(s - m) / l as one exponential, 2^(s log2 e - (m log2 e + log2 l)); a row that sees nothing: 2^-inf
+          s_m[g0 + j] = BF16 ? (l[j] > 0.f ? fmaf(m[j], kLog2E, log2f(l[j])) : INFINITY) : m[j];
+          s_il[g0 + j] = l[j] > 0.f ? 1.0f / l[j] : 0.f;
+        }
   }
   __syncthreads();
   float* w_w = s_w + warp * 32 * HG;
@@ -371,12 +376,12 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
     for (int g0 = 0; g0 < a.heads; g0 += GB) {
       float s8[GB];
 #pragma unroll
-      for (int j = 0; j < GB; ++j) s8[j] = first && g0 == 0 ? pre[j] : (g0 + j < a.heads ? sp[(size_t)(g0 + j) * sh.stride] : 0.f);
+      for (int j = 0; j < GB; ++j, sp += sh.stride) s8[j] = first && g0 == 0 ? pre[j] : (g0 + j < a.heads ? *sp : 0.f);
 #pragma unroll
       for (int j = 0; j < GB; ++j) {
         const int g = g0 + j;
         if (g < a.heads) {
-          const float p = expf(s8[j] - s_m[g]) * s_il[g];
+          const float p = BF16 ? exp2f(fmaf(s8[j], kLog2E, -s_m[g])) : expf(s8[j] - s_m[g]) * s_il[g];
 #pragma unroll
           for (int h = 0; h < HG; ++h) w[h] = fmaf(s_t[g * HG + h], p, w[h]);
         }

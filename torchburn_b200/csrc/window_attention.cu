@@ -220,6 +220,19 @@ __global__ void __launch_bounds__(256) window_scores_kernel(const WindowAttnArgs
   }
 }
 
+template <int N>
+__device__ __forceinline__ void load_row(const float* p, float (&v)[N]) {   // p aligned to the row
+  if constexpr (N == 4) {
+    const float4 x = *reinterpret_cast<const float4*>(p);
+    v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w;
+  } else if constexpr (N == 2) {
+    const float2 x = *reinterpret_cast<const float2*>(p);
+    v[0] = x.x; v[1] = x.y;
+  } else {
+    v[0] = *p;
+  }
+}
+
 // A warp's 32 positions times the values: lanes own CPL neighbouring columns; sums are added to `red` (the warp's own).
 template <typename T, int HG, int CPL>
 __device__ __forceinline__ void warp_values(const T* vals, const int* rows, int64_t row_elems, const float* w, int nj, int vpad, float* red) {
@@ -240,12 +253,12 @@ __device__ __forceinline__ void warp_values(const T* vals, const int* rows, int6
         x[i] = f.x;
         x[i + 1] = f.y;
       }
+      float wj[HG];
+      load_row<HG>(w + j * HG, wj);
 #pragma unroll
-      for (int h = 0; h < HG; ++h) {
-        const float wj = w[j * HG + h];
+      for (int h = 0; h < HG; ++h)
 #pragma unroll
-        for (int i = 0; i < CPL; ++i) acc[h][i] = fmaf(wj, x[i], acc[h][i]);
-      }
+        for (int i = 0; i < CPL; ++i) acc[h][i] = fmaf(wj[h], x[i], acc[h][i]);
     }
 #pragma unroll
     for (int h = 0; h < HG; ++h)
@@ -265,10 +278,11 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
   const int kv = (int)blockIdx.y / per_kv, sub = (int)blockIdx.y - kv * per_kv;
   const int h0 = kv * gq + sub * HG, nh = min(HG, gq - sub * HG);
   const int lr = (int)blockIdx.z, r = sh.row0 + lr;
-  float* s_m = reinterpret_cast<float*>(s_raw);                                // [heads]
-  float* s_il = s_m + a.heads;                                                 // [heads]
-  float* s_t = reinterpret_cast<float*>(s_raw + (((size_t)a.heads * 8 + 15) & ~(size_t)15));   // [heads][HG]
-  float* s_w = s_t + (((size_t)a.heads * HG + 3) & ~(size_t)3);                // [32 warps][HG]
+  const int hp = (a.heads + 15) & ~15;                                         // heads in whole blocks; the rest weigh nothing
+  float* s_m = reinterpret_cast<float*>(s_raw);                                // [hp]
+  float* s_il = s_m + hp;                                                      // [hp]
+  float* s_t = s_il + hp;                                                      // [hp][HG], T transposed
+  float* s_w = s_t + hp * HG;                                                  // [32 warps][HG]
   float* s_red = s_w + blockDim.x * HG;                                       // [warps][HG][vpad]
   float* s_acc = s_red + (size_t)(blockDim.x >> 5) * HG * a.vpad;                      // [HG][vpad]
   int* s_row = reinterpret_cast<int*>(s_acc + HG * a.vpad);                    // [32 warps] cache rows
@@ -277,9 +291,9 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nthr = (int)blockDim.x, nw = nthr >> 5;
   const int csize = (int)gridDim.x, crank = (int)blockIdx.x;   // CTAs that share the row's positions
   grid_dep_launch();
-  for (int i = tid; i < a.heads * HG; i += nthr) {
+  for (int i = tid; i < hp * HG; i += nthr) {
     const int g = i / HG, h = i - g * HG;
-    s_t[i] = h < nh ? a.talk[(size_t)(h0 + h) * a.heads + g] : 0.f;
+    s_t[i] = h < nh && g < a.heads ? a.talk[(size_t)(h0 + h) * a.heads + g] : 0.f;
   }
   for (int i = lane; i < HG * a.vpad; i += 32) s_red[(size_t)warp * HG * a.vpad + i] = 0.f;
   grid_dep_wait();
@@ -317,7 +331,7 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
     for (int j = 0; j < GB; ++j) pre[j] = j < a.heads && v < v_end ? score_row[(size_t)j * sh.stride + v] : 0.f;
   }
   constexpr int SB = 4;                       // softmax statistics from the parts, in a fixed order; SB heads in flight
-  for (int g0 = warp * SB; g0 < a.heads; g0 += nw * SB) {
+  for (int g0 = warp * SB; g0 < hp; g0 += nw * SB) {
     float2 p0[SB], p1[SB];
 #pragma unroll
     for (int j = 0; j < SB; ++j) {
@@ -343,9 +357,10 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
     if (lane == 0)
 #pragma unroll
       for (int j = 0; j < SB; ++j)
-        if (g0 + j < a.heads) {
-          // bf16: exp(s - m) / l as one exponential, 2^(s log2 e - (m log2 e + log2 l)); a row that sees nothing: 2^-inf
-          s_m[g0 + j] = BF16 ? (l[j] > 0.f ? fmaf(m[j], kLog2E, log2f(l[j])) : INFINITY) : m[j];
+        if (g0 + j < hp) {
+          // bf16: exp(s - m) / l as one exponential, 2^(s log2 e - (m log2 e + log2 l)).  A head that is only padding,
+          // or a row that sees nothing: exp(-inf)
+          s_m[g0 + j] = l[j] > 0.f ? (BF16 ? fmaf(m[j], kLog2E, log2f(l[j])) : m[j]) : INFINITY;
           s_il[g0 + j] = l[j] > 0.f ? 1.0f / l[j] : 0.f;
         }
   }
@@ -380,11 +395,11 @@ __global__ void __launch_bounds__(kMixThreads, 2) window_mix_kernel(const Window
 #pragma unroll
       for (int j = 0; j < GB; ++j) {
         const int g = g0 + j;
-        if (g < a.heads) {
-          const float p = BF16 ? exp2f(fmaf(s8[j], kLog2E, -s_m[g])) : expf(s8[j] - s_m[g]) * s_il[g];
+        const float p = BF16 ? exp2f(fmaf(s8[j], kLog2E, -s_m[g])) : expf(s8[j] - s_m[g]) * s_il[g];
+        float t[HG];
+        load_row<HG>(s_t + g * HG, t);
 #pragma unroll
-          for (int h = 0; h < HG; ++h) w[h] = fmaf(s_t[g * HG + h], p, w[h]);
-        }
+        for (int h = 0; h < HG; ++h) w[h] = fmaf(t[h], p, w[h]);
       }
     }
 #pragma unroll
@@ -480,8 +495,8 @@ tb_status launch_generic(const WindowAttnArgs& a, cudaStream_t st, int* launches
   if (mix_splits > (a.max_visible + kMixThreads - 1) / kMixThreads) mix_splits = (a.max_visible + kMixThreads - 1) / kMixThreads;
   if (mix_splits > a.parts_rows / rows) mix_splits = a.parts_rows / rows;
   if (mix_splits < 1) mix_splits = 1;
-  size_t msm = (((size_t)a.heads * 8 + 15) & ~(size_t)15) +
-               4 * ((((size_t)a.heads * hg + 3) & ~(size_t)3) + (size_t)kMixThreads * hg + (size_t)(kMixThreads / 32 + 1) * hg * a.vpad + kMixThreads);
+  const size_t hp = ((size_t)a.heads + 15) & ~(size_t)15;
+  size_t msm = 4 * (hp * (2 + hg) + (size_t)kMixThreads * hg + (size_t)(kMixThreads / 32 + 1) * hg * a.vpad + kMixThreads);
   const bool tensor = sizeof(T) == 2 && a.vpad <= 128;
   const size_t vsm = (size_t)kMixThreads * (a.vpad + (tensor ? 8 : 0)) * sizeof(T);
   const bool staged = msm + vsm <= 220 * 1024;

@@ -387,29 +387,49 @@ void tb_decoder_destroy(tb_decoder* dec);
  * its comment says otherwise.  Weights are bfloat16 (the raw 16 bits) in the
  * layout [out, in]; NULL leaves an optional part out.
  *
- *   x = embed[token] * embed_scale (+ pos_table[position])
+ *   x = embed_norm(embed[token] * embed_scale (+ pos_table[position]))
  *   per layer:  x += norm1_after(mixer(c(norm1(x))));  x += norm2_after(mlp(c(norm2(x))))
- *   logits = embed final_norm(x)
+ *   logits = head final_norm(x)
  *
- * norms are RMS norms with norm_eps inside the root (a missing *_after norm
- * adds the sublayer's output as it is); c(h) = h + causal convolution of h over
- * conv_taps positions per channel (conv weights [hidden, conv_taps], the last
- * tap meets the current position).
- * Attention: q/k norm over the whole projection, score_scale, no rotation;
- * position i sees j <= i with i - j < mask_window or j < mask_keep_first;
- * softmax; the heads' weights are mixed by talk [heads, heads].
- * Feed-forward: down(a N(z) + b N(z^2) + c N(z^3) + e), z = up h, N dividing by
- * the root mean square over the features, act = {a, b, c, e}.
+ * norms are RMS norms with norm_eps inside the root; the weights of embed_norm,
+ * norm1, norm2 and final_norm are norm_offset + the tensor.  A missing
+ * embed_norm or *_after norm passes its input as it is; a missing head is embed.
+ * c(h) = h + causal convolution of h over conv_taps positions per channel (conv
+ * weights [hidden, conv_taps], the last tap meets the current position).
  *
- * State.  Per layer a KV cache (behind a window a ring of about window +
- * prefill_rows positions, the kept first positions apart) and per sublayer the
- * last inputs of the convolution.  A sequence must be fed gap-free; it may be
+ * TB_MIXER_ATTENTION: no rotation; q and k normed either over the whole
+ * projection (q_norm, k_norm) or per head without a weight (qk_unit_norm);
+ *   score(i, j) = cap(score_scale q_i . k_j) - slope_h (i - j)
+ * with cap(s) = score_softcap tanh(s / score_softcap) and slope_h =
+ * 2^(-distance_bias (h + 1) / heads) where these are not 0; position i sees
+ * j <= i with i - j < mask_window and, when mask_chunk > 0, i and j in the same
+ * mask_chunk positions counted from 0, or j < mask_keep_first; softmax.  talk
+ * [heads, heads] mixes the heads' weights (not together with a cap, a bias,
+ * chunks, qk_unit_norm, value mixing or a gate).  value_mix: in every such layer
+ * but the first, v <- (1 - vmix) v + vmix v of the first one, same token.
+ * gate_w [heads, hidden]: a head's output times sigmoid(gate_w h)_h.
+ *
+ * TB_MIXER_LATENT (num_kv_heads 1): c_q = rms(dq_w h) dq_norm [q_rank]; per head
+ * q = uq_w c_q, head_dim plain and rot_dim rotated dimensions; dkv_w h is
+ * [kv_rank | rot_dim]: the latent c = rms(.) dkv_norm and one rotated key part
+ * for all heads.  Per head k = uk_w c, v = uv_w c [value_dim]; score =
+ * score_scale (q . k + rotated q . rotated k).  Rotation: dimensions 2i and
+ * 2i + 1 turn by position * rot_base^(-2i / rot_dims) for 2i < rot_dims.  Cached
+ * are c and the rotated key part.  Masks as above.
+ *
+ * Feed-forward: down(act(up h)).  TB_MLP_POLYNORM: act(z) = a N(z) + b N(z^2) +
+ * c N(z^3) + e, N dividing by the root mean square over the features, act =
+ * {a, b, c, e}.  TB_MLP_RELU2: act(z) = max(z, 0)^2.
+ *
+ * State.  Per layer a cache of keys and values or of latents (behind a window or
+ * in chunks a ring of about that + prefill_rows positions, the kept first
+ * positions apart) and per sublayer the last inputs of the convolution.  A sequence must be fed gap-free; it may be
  * continued from an earlier position than its last one (speculation) by up to
  * a little over 100 positions, or from position 0; anything else fails with
  * TB_ERR_ARG. */
 enum { TB_PRECISION_BF16 = 0, TB_PRECISION_F32 = 1 };
-enum { TB_MIXER_ATTENTION = 0 };
-enum { TB_MLP_NONE = 0, TB_MLP_POLYNORM = 1 };
+enum { TB_MIXER_ATTENTION = 0, TB_MIXER_LATENT = 1 };
+enum { TB_MLP_NONE = 0, TB_MLP_POLYNORM = 1, TB_MLP_RELU2 = 2 };
 typedef struct tb_layered_config {
   int64_t vocab_size;
   int64_t hidden_size;
@@ -422,6 +442,7 @@ typedef struct tb_layered_config {
   int32_t prefill_rows;  /* positions of one sequence per step; 0 means 512 */
   int32_t precision;     /* TB_PRECISION_*: products in bf16 with fp32 sums, or everything in fp32 */
   int32_t flags;         /* TB_DECODER_NO_GRAPH, TB_DECODER_NO_PDL */
+  float norm_offset;     /* 1: norm weights are stored around zero */
 } tb_layered_config;
 typedef struct tb_layered_layer {
   int32_t mixer;
@@ -435,6 +456,16 @@ typedef struct tb_layered_layer {
   int32_t mask_keep_first;
   float score_scale;
   int64_t ff;
+  int32_t mask_chunk;    /* 0: none */
+  int32_t qk_unit_norm;
+  float score_softcap;   /* 0: none */
+  float distance_bias;   /* 0: none */
+  int32_t value_mix;
+  int32_t q_rank;
+  int32_t kv_rank;
+  int32_t rot_dim;
+  int32_t rot_dims;      /* of rot_dim, how many turn (even) */
+  double rot_base;
   const uint16_t* norm1;
   const uint16_t* norm1_after;
   const uint16_t* norm2;
@@ -455,11 +486,21 @@ typedef struct tb_layered_layer {
   const uint16_t* up_w;
   const uint16_t* down_w;
   const uint16_t* act;
+  const uint16_t* vmix;  /* one number */
+  const uint16_t* gate_w;
+  const uint16_t* dq_w;
+  const uint16_t* dq_norm;
+  const uint16_t* uq_w;
+  const uint16_t* dkv_w;
+  const uint16_t* dkv_norm;
+  const uint16_t* uk_w;
+  const uint16_t* uv_w;
 } tb_layered_layer;
-/* embed [vocab, hidden], pos_table [max_seq_len, hidden] or NULL, final_norm [hidden]. */
+/* embed [vocab, hidden], embed_norm [hidden] or NULL, pos_table [max_seq_len, hidden] or NULL, final_norm [hidden],
+ * head [vocab, hidden] or NULL (embed). */
 tb_status tb_decoder_create_layered(tb_decoder** out, const tb_layered_config* cfg, const tb_layered_layer* layers,
-                                    const uint16_t* embed, const uint16_t* pos_table, const uint16_t* final_norm,
-                                    tb_space weight_space);
+                                    const uint16_t* embed, const uint16_t* embed_norm, const uint16_t* pos_table,
+                                    const uint16_t* final_norm, const uint16_t* head, tb_space weight_space);
 /* The next n tokens of sequence `seq` at positions start_offset.. in as few steps as the decoder's rows
  * allow; logits_host [n_want, vocab] receives the logits at the places want[i] (indices into tokens, any
  * order).  With an INT4 decoder seq must be 0. */

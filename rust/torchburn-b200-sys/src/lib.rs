@@ -95,6 +95,7 @@ pub struct tb_layered_config {
     pub prefill_rows: i32,
     pub precision: i32,
     pub flags: i32,
+    pub norm_offset: f32,
 }
 
 /// One of its layers; null pointers leave optional parts out.
@@ -112,6 +113,16 @@ pub struct tb_layered_layer {
     pub mask_keep_first: i32,
     pub score_scale: f32,
     pub ff: i64,
+    pub mask_chunk: i32,
+    pub qk_unit_norm: i32,
+    pub score_softcap: f32,
+    pub distance_bias: f32,
+    pub value_mix: i32,
+    pub q_rank: i32,
+    pub kv_rank: i32,
+    pub rot_dim: i32,
+    pub rot_dims: i32,
+    pub rot_base: f64,
     pub norm1: *const u16,
     pub norm1_after: *const u16,
     pub norm2: *const u16,
@@ -132,6 +143,15 @@ pub struct tb_layered_layer {
     pub up_w: *const u16,
     pub down_w: *const u16,
     pub act: *const u16,
+    pub vmix: *const u16,
+    pub gate_w: *const u16,
+    pub dq_w: *const u16,
+    pub dq_norm: *const u16,
+    pub uq_w: *const u16,
+    pub dkv_w: *const u16,
+    pub dkv_norm: *const u16,
+    pub uk_w: *const u16,
+    pub uv_w: *const u16,
 }
 
 /// Per-layer weights in the capsule order of `create_rust_qwen_decoder`.
@@ -219,7 +239,7 @@ extern "C" {
     pub fn tb_fused_attention_step(qkv: *mut tb_linear, o: *mut tb_linear, x: *const f32, k_cache: *mut f32, v_cache: *mut f32, cos_p: *const f32, sin_p: *const f32, offset: i64, num_heads: i32, num_kv_heads: i32, head_dim: i32, max_seq_len: i64, out: *mut f32, io_space: tb_space, stream: *mut c_void) -> tb_status;
     pub fn tb_fused_transformer_layer_step(x: *mut f32, w: *const tb_layer_step_weights, k_cache: *mut f32, v_cache: *mut f32, cos_p: *const f32, sin_p: *const f32, offset: i64, hidden_size: i64, intermediate_size: i64, num_heads: i32, num_kv_heads: i32, head_dim: i32, max_seq_len: i64, group_size: i32, eps: f32, io_space: tb_space, stream: *mut c_void) -> tb_status;
     pub fn tb_decoder_create(out: *mut *mut tb_decoder, cfg: *const tb_model_config, embed_tokens: *const f32, layers: *const tb_layer_weights, final_norm_w: *const f32, lm_head_w: *const u8, lm_head_s: *const f32, weight_space: tb_space) -> tb_status;
-    pub fn tb_decoder_create_layered(out: *mut *mut tb_decoder, cfg: *const tb_layered_config, layers: *const tb_layered_layer, embed: *const u16, pos_table: *const u16, final_norm: *const u16, weight_space: tb_space) -> tb_status;
+    pub fn tb_decoder_create_layered(out: *mut *mut tb_decoder, cfg: *const tb_layered_config, layers: *const tb_layered_layer, embed: *const u16, embed_norm: *const u16, pos_table: *const u16, final_norm: *const u16, head: *const u16, weight_space: tb_space) -> tb_status;
     pub fn tb_decoder_extend(dec: *mut tb_decoder, seq: i32, start_offset: i64, tokens: *const i64, n: i64, want: *const i64, n_want: i64, logits_host: *mut f32) -> tb_status;
     pub fn tb_decoder_reset_sequence(dec: *mut tb_decoder, seq: i32) -> tb_status;
     pub fn tb_decoder_destroy(dec: *mut tb_decoder);

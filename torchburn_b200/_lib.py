@@ -40,8 +40,8 @@ class LayerWeights(C.Structure):
 
 
 TB_PRECISION = {"bfloat16": 0, "float32": 1}
-TB_MIXER_ATTENTION = 0
-TB_MLP_NONE, TB_MLP_POLYNORM = 0, 1
+TB_MIXER_ATTENTION, TB_MIXER_LATENT = 0, 1
+TB_MLP_NONE, TB_MLP_POLYNORM, TB_MLP_RELU2 = 0, 1, 2
 
 
 class LayeredConfig(C.Structure):
@@ -49,11 +49,13 @@ class LayeredConfig(C.Structure):
         ("vocab_size", C.c_int64), ("hidden_size", C.c_int64), ("num_layers", C.c_int32), ("conv_taps", C.c_int32),
         ("norm_eps", C.c_float), ("embed_scale", C.c_float), ("max_seq_len", C.c_int64), ("max_batch", C.c_int32),
         ("prefill_rows", C.c_int32), ("precision", C.c_int32), ("flags", C.c_int32),
+        ("norm_offset", C.c_float),
     ]
 
 
 LAYERED_TENSORS = ("norm1", "norm1_after", "norm2", "norm2_after", "conv1", "conv2", "q_w", "q_b", "k_w", "k_b", "v_w", "v_b",
-                   "q_norm", "k_norm", "talk", "o_w", "o_b", "up_w", "down_w", "act")
+                   "q_norm", "k_norm", "talk", "o_w", "o_b", "up_w", "down_w", "act", "vmix", "gate_w", "dq_w", "dq_norm", "uq_w", "dkv_w", "dkv_norm",
+                   "uk_w", "uv_w")
 
 
 class LayeredLayer(C.Structure):
@@ -61,6 +63,9 @@ class LayeredLayer(C.Structure):
         ("mixer", C.c_int32), ("mlp", C.c_int32), ("weights_of", C.c_int32), ("num_heads", C.c_int32), ("num_kv_heads", C.c_int32),
         ("head_dim", C.c_int32), ("value_dim", C.c_int32), ("mask_window", C.c_int32), ("mask_keep_first", C.c_int32),
         ("score_scale", C.c_float), ("ff", C.c_int64),
+        ("mask_chunk", C.c_int32), ("qk_unit_norm", C.c_int32), ("score_softcap", C.c_float), ("distance_bias", C.c_float),
+        ("value_mix", C.c_int32), ("q_rank", C.c_int32), ("kv_rank", C.c_int32), ("rot_dim", C.c_int32), ("rot_dims", C.c_int32),
+        ("rot_base", C.c_double),
     ] + [(k, C.c_void_p) for k in LAYERED_TENSORS]
 
 
@@ -114,7 +119,7 @@ SIGNATURES = {
     "tb_fused_attention_step": (_i32, [_p, _p, _p, _p, _p, _p, _p, _i64, _i32, _i32, _i32, _i64, _p, _i32, _p]),
     "tb_fused_transformer_layer_step": (_i32, [_p, _p, _p, _p, _p, _p, _i64, _i64, _i64, _i32, _i32, _i32, _i64, _i32, _f32, _i32, _p]),
     "tb_decoder_create": (_i32, [_PP, C.POINTER(ModelConfig), _p, _p, _p, _p, _p, _i32]),
-    "tb_decoder_create_layered": (_i32, [_PP, C.POINTER(LayeredConfig), _p, _p, _p, _p, _i32]),
+    "tb_decoder_create_layered": (_i32, [_PP, C.POINTER(LayeredConfig), _p, _p, _p, _p, _p, _p, _i32]),
     "tb_decoder_extend": (_i32, [_p, _i32, _i64, _p, _i64, _p, _i64, _p]),
     "tb_decoder_reset_sequence": (_i32, [_p, _i32]),
     "tb_decoder_destroy": (None, [_p]),

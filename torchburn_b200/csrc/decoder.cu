@@ -795,7 +795,8 @@ tb_status tb_decoder_create(tb_decoder** out, const tb_model_config* cfg,
 }
 
 tb_status tb_decoder_create_layered(tb_decoder** out, const tb_layered_config* cfg, const tb_layered_layer* layers,
-                                    const uint16_t* embed, const uint16_t* pos_table, const uint16_t* final_norm, tb_space ws) {
+                                    const uint16_t* embed, const uint16_t* embed_norm, const uint16_t* pos_table,
+                                    const uint16_t* final_norm, const uint16_t* head, tb_space ws) {
   if (!out) return fail(TB_ERR_ARG, "tb_decoder_create_layered: null out");
   *out = nullptr;
   if (!cfg || !layers || !embed || !final_norm) return fail(TB_ERR_ARG, "tb_decoder_create_layered: null argument");
@@ -818,7 +819,7 @@ tb_status tb_decoder_create_layered(tb_decoder** out, const tb_layered_config* c
   };
 #define CR(expr) do { const tb_status _st = (expr); if (_st != TB_OK) return fin(_st); } while (0)
 #define CRC(expr) do { cudaError_t _e = (expr); if (_e != cudaSuccess) return fin(fail(_e == cudaErrorMemoryAllocation ? TB_ERR_OOM : TB_ERR_CUDA, "%s failed: %s", #expr, cudaGetErrorString(_e))); } while (0)
-  CR(layered_create(&d->lay, c, layers, embed, pos_table, final_norm, ws, (c.flags & TB_DECODER_NO_GRAPH) != 0));
+  CR(layered_create(&d->lay, c, layers, LayeredTables{embed, embed_norm, pos_table, final_norm, head}, ws, (c.flags & TB_DECODER_NO_GRAPH) != 0));
   cudaGetDevice(&d->device);
   CRC(cudaStreamCreateWithFlags(&d->stream, cudaStreamNonBlocking));
   d->seq_len.assign((size_t)d->B, 0);

@@ -1,5 +1,5 @@
-// Kernels of the layered decoder (layered.cu): unquantized projections, the row kernels between them and
-// windowed attention with mixed heads.  Everything is a parameter: sizes, windows, taps, constants.
+// Kernels of the layered decoder (layered.cu): unquantized projections, the row kernels between them, flash
+// attention and windowed attention with mixed heads.  Everything is a parameter: sizes, windows, taps, constants.
 //
 // Precision.  With 16-bit products (Precision::kBf16) the operands of a projection are bf16 and the sums
 // fp32; the residual stream, norms, scores, attention weights and the convolution history are fp32, the KV
@@ -83,15 +83,18 @@ tb_status launch_kernel(void (*kern)(KArgs...), dim3 grid, dim3 block, size_t sm
 
 // ---- projections (dense_gemm.cu) ---------------------------------------------------------------
 // A weight matrix [n, k] as tiles of 128 rows x 64 columns, each a contiguous 16 KB image like
-// ActOperand's: tile (n / 128, k / 64) at ((n / 128) * (kp / 64) + k / 64) * 16384 bytes.
+// ActOperand's: tile (n / 128, k / 64) at ((n / 128) * (kp / 64) + k / 64) * 16384 bytes.  `batch` matrices of
+// one size (one per head, say) lie one after the other.
 struct DenseWeight {
   void* img = nullptr;
   int64_t rows = 0;   // padded rows (multiple of 128)
   int64_t kp = 0;     // padded K (multiple of 64)
+  int batch = 1;
 };
-tb_status dense_weight_alloc(DenseWeight* w, int64_t rows, int64_t k);
-// Rows [row0, row0 + n) of the image from a row-major bf16 matrix [n, k] (host or device).
-tb_status dense_weight_fill(DenseWeight* w, int64_t row0, const uint16_t* src, int64_t n, int64_t k, tb_space space);
+tb_status dense_weight_alloc(DenseWeight* w, int64_t rows, int64_t k, int batch = 1);
+// Rows [row0, row0 + n) of every matrix of the batch from bf16 matrices [batch][n, k] (host or device);
+// `transposed`: each is stored as [k, n].
+tb_status dense_weight_fill(DenseWeight* w, int64_t row0, const uint16_t* src, int64_t n, int64_t k, tb_space space, bool transposed = false);
 
 // Partial sums of a projection: y[s][row][ldy], s < splits <= 8; the consumer adds them in that order.
 struct PartialSums {
@@ -100,21 +103,31 @@ struct PartialSums {
   size_t split_stride = 0;   // floats
   int64_t ldy = 0;
 };
+// Where a product's sums go: fp32 partial sums for a row kernel, rows of the activation type (bf16 or fp32), or,
+// after an elementwise activation, the operand of the next product.
+enum class DenseSink { kPartials = 0, kRows = 1, kOperand = 2 };
+enum class DenseAct { kNone = 0, kRelu2 = 1 };   // kRelu2: the square of max(z, 0)
 struct DenseGemmArgs {
   const DenseWeight* w = nullptr;
-  ActOperand x;
+  ActOperand x;              // a batch: the operands of the matrices one after the other, each mp x kp
   int rows = 0;
-  float* out = nullptr;      // [splits][rows][ldo]
+  DenseSink sink = DenseSink::kPartials;
+  void* out = nullptr;       // kPartials: float [splits][rows][ldo]; kRows: [rows][ldo]
   int64_t ldo = 0;
-  int64_t n_valid = 0;       // output features stored (the rest of the last tile is dropped)
-  int splits = 1;
+  ActOperand operand;        // kOperand
+  DenseAct act = DenseAct::kNone;
+  int64_t batch_cols = 0;    // column of matrix b's first feature: b * batch_cols
+  int64_t n_valid = 0;       // output features stored per matrix (the rest of the last tile is dropped)
+  int splits = 1;            // 1 unless kPartials
   size_t split_stride = 0;
   bool pdl = false;
 };
 // Rows padded the way the product's row tile wants them.
 int dense_row_pad(int rows);
 // How many CTAs share an output tile by splitting K (deterministic: partial sums, no atomics).
-int dense_splits(Precision p, int64_t n_rows, int64_t kp, int rows, int max_splits);
+// Of two equally fast ways the one with fewer partial sums; `gain` (optional): what the split saves, in stages of
+// the K loop.
+int dense_splits(Precision p, int64_t n_rows, int64_t kp, int rows, int max_splits, double* gain = nullptr);
 tb_status launch_dense_gemm(Precision p, const DenseGemmArgs& a, cudaStream_t st);
 int dense_fault_flag();
 
@@ -128,7 +141,7 @@ struct StepRows {
   int rows = 0;
 };
 // x' = source; h = norm(x') * pre_w; operand = h + causal convolution of h over time.
-// Source: the embedding (scaled table row + position row), or x + [norm](y + bias) * post_w.
+// Source: [norm] of the embedding (scaled table row + position row) * post_w, or x + [norm](y + bias) * post_w.
 struct GlueArgs {
   StepRows r;
   // source
@@ -188,6 +201,60 @@ struct QkvPrepArgs {
 };
 tb_status launch_qkv_prep(Precision p, const QkvPrepArgs& a, cudaStream_t st);
 
+// Heads of a combined product [q | k | v | gates]: per-head norm of q and k without a weight, value mixing, the
+// cache append, gates = sigmoid.
+struct HeadsPrepArgs {
+  StepRows r;
+  PartialSums y;
+  int heads = 0, kv_heads = 0, dim = 0, vdim = 0, dpad = 0, vpad = 0;
+  int q_off = 0, k_off = 0, v_off = 0, g_off = 0;   // columns of y
+  bool unit_norm = false;
+  float eps = 0.f;
+  float* v_first = nullptr;              // [rows, kv_heads * vdim] or null: v <- (1 - mix) v + mix v_first,
+  bool keep_first_values = false;        // or this layer's values are the ones that later layers mix in
+  float mix = 0.f;
+  float* gate = nullptr;                 // [rows, heads] or null
+  void* q = nullptr;                     // [rows, heads * dpad] of the activation type
+  void* k_cache = nullptr;
+  void* v_cache = nullptr;
+  CacheGeom geom;
+  bool pdl = false;
+};
+tb_status launch_heads_prep(Precision p, const HeadsPrepArgs& a, cudaStream_t st);
+
+// Latent attention.  A position's cache row is [normed latent kv_rank | rotated key part rot_dim], padded to dpad; the
+// query of a head lives in the same space: its unrotated part times the head's key matrix, then its rotated part.
+// (q . W c = (W^T q) . c, so the keys of the heads are never written out.)
+struct LatentPrepArgs {
+  StepRows r;
+  PartialSums y;                         // [query latent | at kv_off: key/value latent, rotated key part]
+  int q_rank = 0, kv_rank = 0, rot_dim = 0, rot_dims = 0, kv_off = 0, dpad = 0;
+  const float* q_norm = nullptr;         // [q_rank]
+  const float* kv_norm = nullptr;        // [kv_rank]
+  const float2* table = nullptr;         // [positions][rot_dims / 2] cos, sin
+  float eps = 0.f;
+  ActOperand out;                        // the query latent
+  void* cache = nullptr;                 // [slots][cache rows][dpad]
+  CacheGeom geom;
+  bool pdl = false;
+};
+tb_status launch_latent_prep(Precision p, const LatentPrepArgs& a, cudaStream_t st);
+struct LatentQueryArgs {
+  StepRows r;
+  PartialSums y;                         // [heads][dim | rot_dim]
+  int heads = 0, dim = 0, rot_dim = 0, rot_dims = 0, kv_rank = 0, dpad = 0;
+  const float2* table = nullptr;
+  ActOperand out;                        // one operand of K = dim per head, one after the other
+  void* q = nullptr;                     // [rows, heads * dpad] of the activation type
+  bool pdl = false;
+};
+tb_status launch_latent_query(Precision p, const LatentQueryArgs& a, cudaStream_t st);
+// cos and sin of position * base^(-2i / dims).
+tb_status fill_rotation_table(float2* table, int64_t positions, int dims, double base);
+
+// operand = max(z, 0)^2 (the products write it themselves when they have no partial sums)
+tb_status launch_relu2(Precision p, int rows, const PartialSums& z, const ActOperand& out, bool pdl, cudaStream_t st);
+
 // operand = a N(z) + b N(z^2) + c N(z^3) + e, N dividing a row by its root mean square (PolyNorm).
 struct PolyNormArgs {
   int rows = 0;
@@ -199,6 +266,34 @@ struct PolyNormArgs {
   bool pdl = false;
 };
 tb_status launch_poly_norm(Precision p, const PolyNormArgs& a, cudaStream_t st);
+
+// ---- attention with an online softmax (flash_attention.cu) ----------------------------------------
+struct FlashArgs {
+  StepRows r;
+  const void* q = nullptr;               // [rows, heads * dpad] of the activation type
+  const void* k_cache = nullptr;
+  const void* v_cache = nullptr;
+  bool values_in_keys = false;           // one key/value head whose values are the first vdim elements of its keys
+  CacheGeom geom;
+  int heads = 0, kv_heads = 0, dim = 0, vdim = 0, dpad = 0, vpad = 0;
+  float scale = 1.f;
+  float softcap = 0.f;                   // 0: none
+  const float* slopes = nullptr;         // [heads], taken off per position between query and key; null: none
+  int window = 0;                        // position i sees j when i - j < window and i / chunk = j / chunk (chunk > 0),
+  int keep_first = 0;                    // or j < keep_first
+  int chunk = 0;
+  const float* gate = nullptr;           // [rows, heads] factors of the heads' outputs, or null
+  int64_t max_visible = 0;               // most positions one row can see
+  float* parts = nullptr;                // scratch [part_slots][vdim]
+  float2* part_ml = nullptr;             // scratch [part_slots]
+  int64_t part_slots = 0;
+  ActOperand out;                        // K = heads * vdim
+  bool out_per_head = false;             // or one operand of K = vdim per head, one after the other
+  bool one_sequence = false;             // the rows are consecutive positions of one sequence
+  bool pdl = false;
+};
+int64_t flash_part_slots(int64_t rows, int64_t heads);   // what the splits a step can use need
+tb_status launch_flash_attention(Precision p, const FlashArgs& a, cudaStream_t st, int* launches);
 
 // ---- windowed attention with mixed heads (window_attention.cu) -----------------------------------
 struct WindowAttnArgs {

@@ -1,0 +1,534 @@
+// Attention with an online softmax: grouped heads, a window with kept first positions or chunks of the sequence, a
+// soft cap on the scores, a distance bias per head, an output gate per head; or one latent shared by all heads, whose
+// first elements are also the values.
+//
+//   score(i, j) = cap(scale q_i . k_j) - slope_h (i - j),   cap(s) = softcap tanh(s / softcap)
+//
+// bf16 (flash_mma_kernel): a CTA takes up to 64 (query, head) pairs of one key/value head - the heads of one row in
+// a decode step, several queries times the heads in a portion - so that heads that share keys share their loads.
+// Per tile of 32 or 64 keys: scores by mma.sync with the warps side by side over the keys, softmax weights to shared
+// memory as two bf16 pieces (the second one what the rounding of the first left: 16 mantissa bits), then the values
+// with the warps side by side over the value columns.  CTAs that share a block's keys leave (max, sum, unnormalised
+// output) and a last kernel merges them in a fixed order.
+// fp32, and sizes beyond the tiles (flash_simple_kernel): a CTA per row and up to four heads, fp32 products.
+#include "dense.cuh"
+#include "window_attention.cuh"
+
+namespace tb {
+
+namespace {
+
+constexpr int kThreads = 256;
+constexpr float kLog2E = 1.44269504f;
+constexpr int kMaxSplits = 512;
+
+struct FlashShape {
+  int run_rows;   // rows that share a sequence: the whole step, or one
+  int tiles;      // CTAs' shares of a run's (query, head) pairs
+  int splits;     // CTAs that share a tile's keys
+  int pair_tile;  // kernel's pairs per tile
+};
+
+__device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
+__device__ __forceinline__ void cp16z(void* dst, const void* src, bool live) {   // zeros when not live
+  const int n = live ? 16 : 0;
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(n) : "memory");
+}
+__device__ __forceinline__ void ldm4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)));
+}
+__device__ __forceinline__ void ldm2(uint32_t (&r)[2], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_addr(p)));
+}
+__device__ __forceinline__ void ldm4t(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_addr(p)));
+}
+__device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+
+// Elements behind a head's output that the next product's padded K covers: column c of head h for c in [vdim, limit).
+__host__ __device__ __forceinline__ int column_limit(const FlashArgs& a, int h) {
+  if (a.out_per_head) return a.out.kp;
+  return h == a.heads - 1 ? a.out.kp - h * a.vdim : a.vdim;
+}
+template <bool BF16>
+__device__ __forceinline__ void store_column(const FlashArgs& a, int row, int h, int c, float v) {
+  if (!a.out_per_head) {
+    act_store1<BF16>(a.out, row, h * a.vdim + c, v);
+    return;
+  }
+  ActOperand o = a.out;
+  o.data = static_cast<unsigned char*>(o.data) + (size_t)h * o.mp * o.kp * (BF16 ? 2 : 4);
+  act_store1<BF16>(o, row, c, v);
+}
+
+// First positions that a row sees in its own run.
+__device__ __forceinline__ int run_start(const FlashArgs& a, int pos) { return VisibleRange(pos, a.window, 0, a.chunk).lo; }
+
+// grid (tiles * splits, kv heads, runs)
+template <int MG, int NV, int KT>
+__global__ void __launch_bounds__(kThreads, NV <= 8 ? 2 : 1) flash_mma_kernel(const FlashArgs a, const FlashShape sh) {
+  extern __shared__ __align__(16) unsigned char s_raw[];
+  constexpr int M = 16 * MG, WN = 8 / MG, KW = KT / WN, NS = KW / 8, PLD = KT + 8;
+  static_assert(NS >= 1, "a warp takes at least eight keys");
+  const int gq = a.heads / a.kv_heads, kv = (int)blockIdx.y;
+  const int split = (int)blockIdx.x % sh.splits, tile = sh.tiles - 1 - (int)blockIdx.x / sh.splits;   // the longest tiles first
+  const int row0 = (int)blockIdx.z * sh.run_rows, pairs = sh.run_rows * gq;
+  const int p0 = tile * M, np = min(M, pairs - p0);
+  const int ld = a.dpad + 8, vld = a.values_in_keys ? ld : a.vpad + 8;
+  __nv_bfloat16* s_q = reinterpret_cast<__nv_bfloat16*>(s_raw);             // [M][ld]
+  __nv_bfloat16* s_k = s_q + M * ld;                                        // [2][KT][ld]
+  __nv_bfloat16* s_v = a.values_in_keys ? s_k : s_k + 2 * KT * ld;          // [2][KT][vld]
+  __nv_bfloat16* s_p = a.values_in_keys ? s_k + 2 * KT * ld : s_v + 2 * KT * vld;   // [2 pieces][M][PLD]
+  float* s_max = reinterpret_cast<float*>(s_p + 2 * M * PLD);               // [WN][M]
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, wr = warp % MG, wc = warp / MG;
+  grid_dep_launch();
+  grid_dep_wait();
+  const int pos_r = a.r.pos[row0];
+  const int first = pos_r + p0 / gq;
+  int last = pos_r + (p0 + np - 1) / gq;
+  if (a.geom.ring == 0) last = min(last, (int)a.geom.rows - 1);
+  const BlockKeys keys(first, pos_r < 0 ? -1 : last, a.window, a.keep_first, a.chunk);
+  const size_t slot = pos_r < 0 ? 0 : (size_t)a.r.slots[row0];
+  const int krow = a.kv_heads * a.dpad, vrow = a.kv_heads * a.vpad;
+  const __nv_bfloat16* kc = static_cast<const __nv_bfloat16*>(a.k_cache) + slot * a.geom.rows * (size_t)krow + (size_t)kv * a.dpad;
+  const __nv_bfloat16* vc = static_cast<const __nv_bfloat16*>(a.v_cache) + (a.values_in_keys ? 0 : slot * a.geom.rows * (size_t)vrow + (size_t)kv * a.vpad);
+  // 2^lsh threads per row of 16-byte pieces
+  auto log_threads = [](int pieces) {
+    int l = 1;
+    while ((1 << l) < pieces) ++l;
+    return l;
+  };
+  const int kpieces = a.dpad >> 3, vpieces = a.vpad >> 3, klsh = log_threads(kpieces), vlsh = log_threads(vpieces);
+  auto fetch = [&](int t) {
+    const RunRows rows(keys, a.geom, t * KT);
+    {
+      const int c = tid & ((1 << klsh) - 1);
+      __nv_bfloat16* dst = s_k + (t & 1) * KT * ld + c * 8;
+      if (c < kpieces)
+        for (int r = tid >> klsh; r < KT; r += kThreads >> klsh) {
+          const int v = t * KT + r;
+          const bool live = v < keys.count;
+          cp16z(dst + r * ld, kc + (size_t)(live ? rows.row(v) : 0) * krow + c * 8, live);
+        }
+    }
+    if (!a.values_in_keys) {
+      const int c = tid & ((1 << vlsh) - 1);
+      __nv_bfloat16* dst = s_v + (t & 1) * KT * vld + c * 8;
+      if (c < vpieces)
+        for (int r = tid >> vlsh; r < KT; r += kThreads >> vlsh) {
+          const int v = t * KT + r;
+          const bool live = v < keys.count;
+          cp16z(dst + r * vld, vc + (size_t)(live ? rows.row(v) : 0) * vrow + c * 8, live);
+        }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  const int tiles = (keys.count + KT - 1) / KT;
+  const int t0 = (int)((int64_t)tiles * split / sh.splits), t1 = (int)((int64_t)tiles * (split + 1) / sh.splits);
+  {
+    const int c = tid & ((1 << klsh) - 1);
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q);
+    if (c < kpieces)
+      for (int i = tid >> klsh; i < M; i += kThreads >> klsh) {
+        const bool live = i < np;
+        const int p = p0 + (live ? i : 0), qi = p / gq;
+        cp16z(s_q + i * ld + c * 8, q + ((size_t)(row0 + qi) * a.heads + kv * gq + p - qi * gq) * a.dpad + c * 8, live);
+      }
+  }
+  if (t0 < t1) fetch(t0);
+  else asm volatile("cp.async.commit_group;" ::: "memory");
+  // this thread's two rows of the warp's sixteen
+  int qpos[2], lo[2], head[2], qrow[2];
+  float slope[2];
+  bool live[2];
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    const int i = wr * 16 + (lane >> 2) + 8 * e, p = p0 + i, qi = p / gq;
+    live[e] = i < np;
+    qrow[e] = row0 + qi;
+    head[e] = kv * gq + p - qi * gq;
+    qpos[e] = pos_r + qi;
+    lo[e] = run_start(a, qpos[e]);
+    slope[e] = live[e] && a.slopes ? a.slopes[head[e]] * kLog2E : 0.f;
+  }
+  const int lo_last = run_start(a, last);
+  const float scale2 = a.softcap > 0.f ? 0.f : a.scale * kLog2E;
+  const float cap_in = a.softcap > 0.f ? 2.f * kLog2E * a.scale / a.softcap : 0.f, cap_out = a.softcap * kLog2E;
+  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+  float acc[NV][4];
+#pragma unroll
+  for (int n = 0; n < NV; ++n)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[n][i] = 0.f;
+  const int cw = ((a.vpad + WN - 1) / WN + 15) & ~15, col0 = wc * cw, ncol = min(cw, a.vpad - col0);   // the warp's value columns
+
+  for (int t = t0; t < t1; ++t) {
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    __syncthreads();                       // tile t is here, nobody reads tile t - 1 or its weights any more
+    if (t + 1 < t1) fetch(t + 1);
+    const __nv_bfloat16* k = s_k + (t & 1) * KT * ld + wc * KW * ld;
+    float s[NS][4];
+#pragma unroll
+    for (int j = 0; j < NS; ++j)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) s[j][i] = 0.f;
+#pragma unroll 4
+    for (int c = 0; c < a.dpad; c += 16) {
+      uint32_t qa[4];
+      ldm4(qa, s_q + (wr * 16 + (lane & 15)) * ld + c + (lane >> 4) * 8);
+      if constexpr (NS == 1) {
+        uint32_t kb[2];
+        ldm2(kb, k + (lane & 7) * ld + c + ((lane >> 3) & 1) * 8);
+        mma16816(s[0], qa, kb[0], kb[1]);
+      } else {
+#pragma unroll
+        for (int j = 0; j < NS; j += 2) {
+          uint32_t kb[4];
+          ldm4(kb, k + (j * 8 + (lane & 7) + ((lane >> 4) << 3)) * ld + c + ((lane >> 3) & 1) * 8);
+          mma16816(s[j], qa, kb[0], kb[1]);
+          mma16816(s[j + 1], qa, kb[2], kb[3]);
+        }
+      }
+    }
+    // s[j][2 e + i]: row e, key 8 j + 2 (lane & 3) + i of the warp's
+    const int v0 = t * KT;
+    const bool all_seen = v0 >= keys.nk && v0 + KT <= keys.count && keys.position(v0 + KT - 1) <= first && keys.position(v0) >= lo_last;
+    float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+    for (int j = 0; j < NS; ++j)
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int v = v0 + wc * KW + j * 8 + (lane & 3) * 2 + i, p = keys.position(v);
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          float x = s[j][2 * e + i];
+          if (a.softcap > 0.f) x = fmaf(-2.f * cap_out, __fdividef(1.f, exp2f(x * cap_in) + 1.f), cap_out);   // tanh z = 1 - 2 / (e^2z + 1)
+          else x *= scale2;
+          x = fmaf(-slope[e], (float)(qpos[e] - p), x);
+          if (!all_seen && !(v < keys.count && p <= qpos[e] && (p >= lo[e] || p < a.keep_first))) x = -INFINITY;
+          s[j][2 * e + i] = x;
+          mx[e] = fmaxf(mx[e], x);
+        }
+      }
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
+      mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
+      if ((lane & 3) == 0) s_max[wc * M + wr * 16 + (lane >> 2) + 8 * e] = mx[e];
+    }
+    __syncthreads();
+    float alpha[2];
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      float mn = m[e];
+#pragma unroll
+      for (int w = 0; w < WN; ++w) mn = fmaxf(mn, s_max[w * M + wr * 16 + (lane >> 2) + 8 * e]);
+      const float base = mn == -INFINITY ? 0.f : mn;   // nothing seen yet: weights exp(-inf) = 0
+      alpha[e] = exp2f(m[e] - base);
+      m[e] = mn;
+      float sum = 0.f;
+      __nv_bfloat16* pr = s_p + (wr * 16 + (lane >> 2) + 8 * e) * PLD + wc * KW + (lane & 3) * 2;
+#pragma unroll
+      for (int j = 0; j < NS; ++j) {
+        const float w0 = exp2f(s[j][2 * e] - base), w1 = exp2f(s[j][2 * e + 1] - base);
+        sum += w0 + w1;
+        const __nv_bfloat162 hi = __floats2bfloat162_rn(w0, w1);
+        const float2 hf = __bfloat1622float2(hi);
+        *reinterpret_cast<__nv_bfloat162*>(pr + j * 8) = hi;
+        *reinterpret_cast<__nv_bfloat162*>(pr + M * PLD + j * 8) = __floats2bfloat162_rn(w0 - hf.x, w1 - hf.y);
+      }
+      l[e] = fmaf(l[e], alpha[e], sum);
+    }
+    __syncthreads();
+    if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
+#pragma unroll
+      for (int n = 0; n < NV; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[n][i] *= alpha[i >> 1];
+    }
+    const __nv_bfloat16* vt = s_v + (t & 1) * KT * vld + col0;
+#pragma unroll
+    for (int kk = 0; kk < KT; kk += 16) {
+      uint32_t hi[4], rest[4];
+      const __nv_bfloat16* pp = s_p + (wr * 16 + (lane & 15)) * PLD + kk + (lane >> 4) * 8;
+      ldm4(hi, pp);
+      ldm4(rest, pp + M * PLD);
+#pragma unroll
+      for (int n = 0; n < NV; n += 2) {
+        if (n * 8 >= ncol) break;
+        uint32_t vb[4];   // V is [key][column]: (keys 0-7, cols 0-7) (keys 8-15, cols 0-7) (keys 0-7, cols 8-15) ...
+        ldm4t(vb, vt + (kk + (lane & 15)) * vld + n * 8 + (lane >> 4) * 8);
+        mma16816(acc[n], hi, vb[0], vb[1]);
+        mma16816(acc[n + 1], hi, vb[2], vb[3]);
+        mma16816(acc[n], rest, vb[0], vb[1]);
+        mma16816(acc[n + 1], rest, vb[2], vb[3]);
+      }
+    }
+  }
+  asm volatile("cp.async.wait_all;" ::: "memory");
+  __syncthreads();
+  // the rows' sums over the warps side by side
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
+    l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
+    if ((lane & 3) == 0) s_max[wc * M + wr * 16 + (lane >> 2) + 8 * e] = l[e];
+  }
+  __syncthreads();
+  const bool whole = sh.splits == 1;
+#pragma unroll
+  for (int e = 0; e < 2; ++e) {
+    if (!live[e]) continue;
+    float sum = 0.f;
+#pragma unroll
+    for (int w = 0; w < WN; ++w) sum += s_max[w * M + wr * 16 + (lane >> 2) + 8 * e];
+    float f = 1.f;
+    if (whole) {
+      f = sum > 0.f ? 1.f / sum : 0.f;
+      if (a.gate) f *= a.gate[(size_t)qrow[e] * a.heads + head[e]];
+    }
+    const size_t part = ((size_t)split * a.r.rows + qrow[e]) * a.heads + head[e];
+    if (!whole && wc == 0 && (lane & 3) == 0) a.part_ml[part] = make_float2(m[e], sum);
+    float* dst = a.parts + part * a.vdim;
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      if (n * 8 >= ncol) break;
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const int c = col0 + n * 8 + (lane & 3) * 2 + i;
+        if (c >= a.vdim) continue;
+        if (whole) store_column<true>(a, qrow[e], head[e], c, acc[n][2 * e + i] * f);
+        else dst[c] = acc[n][2 * e + i];
+      }
+    }
+    if (whole && wc == 0)
+      for (int c = a.vdim + (lane & 3); c < column_limit(a, head[e]); c += 4) store_column<true>(a, qrow[e], head[e], c, 0.f);
+  }
+}
+
+// Merges the shares of a row's keys.  grid (heads, rows, columns / 128)
+__global__ void __launch_bounds__(128) flash_merge_kernel(const FlashArgs a, const int splits) {
+  __shared__ float s_w[kMaxSplits], s_red[4], s_sum[4];
+  const int tid = threadIdx.x, h = (int)blockIdx.x, r = (int)blockIdx.y, c = (int)blockIdx.z * 128 + tid;
+  grid_dep_launch();
+  grid_dep_wait();
+  const size_t stride = (size_t)a.r.rows * a.heads, at = (size_t)r * a.heads + h;
+  float m = -INFINITY;
+  for (int z = tid; z < splits; z += 128) m = fmaxf(m, a.part_ml[z * stride + at].x);
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+  if ((tid & 31) == 0) s_red[tid >> 5] = m;
+  __syncthreads();
+  m = fmaxf(fmaxf(s_red[0], s_red[1]), fmaxf(s_red[2], s_red[3]));
+  float l = 0.f;
+  for (int z = tid; z < splits; z += 128) {
+    const float2 p = a.part_ml[z * stride + at];
+    const float w = p.x == -INFINITY ? 0.f : exp2f(p.x - m);
+    s_w[z] = w;
+    l = fmaf(w, p.y, l);
+  }
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+  if ((tid & 31) == 0) s_sum[tid >> 5] = l;
+  __syncthreads();
+  l = (s_sum[0] + s_sum[1]) + (s_sum[2] + s_sum[3]);
+  if (c >= column_limit(a, h)) return;
+  float v = 0.f;
+  if (c < a.vdim) {
+    const float* p = a.parts + at * a.vdim + c;
+#pragma unroll 8
+    for (int z = 0; z < splits; ++z)
+      if (s_w[z] > 0.f) v = fmaf(s_w[z], p[(size_t)z * stride * a.vdim], v);   // a share that saw nothing left zeros or nothing
+    float f = l > 0.f ? 1.f / l : 0.f;
+    if (a.gate) f *= a.gate[at];
+    v *= f;
+  }
+  store_column<true>(a, r, h, c, v);
+}
+
+__device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 load4(const __nv_bfloat16* p) {
+  const uint2 u = *reinterpret_cast<const uint2*>(p);
+  return make_float4(__uint_as_float(u.x << 16), __uint_as_float(u.x & 0xFFFF0000u), __uint_as_float(u.y << 16), __uint_as_float(u.y & 0xFFFF0000u));
+}
+
+// grid (kv heads * groups of four of their query heads, rows)
+template <typename T>
+__global__ void __launch_bounds__(kThreads) flash_simple_kernel(const FlashArgs a) {
+  extern __shared__ __align__(16) float s_f[];
+  constexpr int HG = 4, KT = 32;
+  __shared__ float s_s[HG][KT], s_alpha[HG], s_l[HG];
+  __shared__ int s_row[KT];
+  const int gq = a.heads / a.kv_heads, groups = (gq + HG - 1) / HG;
+  const int kv = (int)blockIdx.x / groups, h0 = kv * gq + ((int)blockIdx.x - kv * groups) * HG, nh = min(HG, (kv + 1) * gq - h0);
+  const int r = (int)blockIdx.y, tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  float* s_q = s_f;                    // [HG][dpad]
+  float* s_o = s_q + HG * a.dpad;      // [HG][vdim]
+  grid_dep_launch();
+  grid_dep_wait();
+  const int pos = a.r.pos[r];
+  const VisibleRange vr(pos, a.window, a.keep_first, a.chunk);
+  const int nv = vr.count();
+  const size_t slot = pos < 0 ? 0 : (size_t)a.r.slots[r];
+  const int krow = a.kv_heads * a.dpad, vrow = a.values_in_keys ? krow : a.kv_heads * a.vpad;
+  const T* kc = static_cast<const T*>(a.k_cache) + slot * a.geom.rows * (size_t)krow + (size_t)kv * a.dpad;
+  const T* vc = a.values_in_keys ? kc : static_cast<const T*>(a.v_cache) + slot * a.geom.rows * (size_t)vrow + (size_t)kv * a.vpad;
+  const T* q = static_cast<const T*>(a.q) + ((size_t)r * a.heads + h0) * a.dpad;
+  for (int i = tid; i < nh * a.dpad; i += kThreads) s_q[i] = (float)q[i];
+  for (int i = tid; i < nh * a.vdim; i += kThreads) s_o[i] = 0.f;
+  float m = -INFINITY, l = 0.f;        // of head `warp`, in warps 0..nh-1
+  for (int t = 0; t < nv; t += KT) {
+    const int nj = min(KT, nv - t);
+    if (tid < KT) s_row[tid] = a.geom.row_of(vr.position(min(t + tid, nv - 1)));
+    __syncthreads();
+    {
+      const int j = tid >> 3, part = tid & 7;
+      const T* k = kc + (size_t)s_row[j] * krow;
+      float d[HG] = {0.f, 0.f, 0.f, 0.f};
+      for (int c = part * 4; c < a.dpad; c += 32) {
+        const float4 x = load4(k + c);
+#pragma unroll
+        for (int h = 0; h < HG; ++h)
+          if (h < nh) {
+            const float4 y = load4(s_q + h * a.dpad + c);
+            d[h] = fmaf(x.x, y.x, fmaf(x.y, y.y, fmaf(x.z, y.z, fmaf(x.w, y.w, d[h]))));
+          }
+      }
+#pragma unroll
+      for (int h = 0; h < HG; ++h) {
+#pragma unroll
+        for (int o = 4; o > 0; o >>= 1) d[h] += __shfl_xor_sync(0xffffffffu, d[h], o);
+        if (part == 0 && h < nh) {
+          float x = d[h] * a.scale;
+          if (a.softcap > 0.f) x = a.softcap * tanhf(x / a.softcap);
+          if (a.slopes) x -= a.slopes[h0 + h] * (float)(pos - vr.position(t + j));
+          s_s[h][j] = j < nj ? x : -INFINITY;
+        }
+      }
+    }
+    __syncthreads();
+    if (warp < nh) {
+      const float x = s_s[warp][lane];
+      float mx = x;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+      const float mn = fmaxf(m, mx), alpha = expf(m - mn), w = expf(x - mn);   // a tile holds at least one visible key
+      float sum = w;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+      l = fmaf(l, alpha, sum);
+      m = mn;
+      s_s[warp][lane] = w;
+      if (lane == 0) s_alpha[warp] = alpha;
+    }
+    __syncthreads();
+    for (int c = tid; c < a.vdim; c += kThreads) {
+      float o[HG];
+#pragma unroll
+      for (int h = 0; h < HG; ++h) o[h] = h < nh ? s_o[h * a.vdim + c] * s_alpha[h] : 0.f;
+      for (int j = 0; j < nj; ++j) {
+        const float v = (float)vc[(size_t)s_row[j] * vrow + c];
+#pragma unroll
+        for (int h = 0; h < HG; ++h) o[h] = h < nh ? fmaf(s_s[h][j], v, o[h]) : 0.f;
+      }
+#pragma unroll
+      for (int h = 0; h < HG; ++h)
+        if (h < nh) s_o[h * a.vdim + c] = o[h];
+    }
+    __syncthreads();
+  }
+  if (warp < nh && lane == 0) s_l[warp] = l;
+  __syncthreads();
+  for (int h = 0; h < nh; ++h) {
+    float f = s_l[h] > 0.f ? 1.f / s_l[h] : 0.f;
+    if (a.gate) f *= a.gate[(size_t)r * a.heads + h0 + h];
+    for (int c = tid; c < column_limit(a, h0 + h); c += kThreads)
+      store_column<sizeof(T) == 2>(a, r, h0 + h, c, c < a.vdim ? s_o[h * a.vdim + c] * f : 0.f);
+  }
+}
+
+template <typename T>
+tb_status launch_simple(const FlashArgs& a, cudaStream_t st, int* launches) {
+  const int gq = a.heads / a.kv_heads;
+  const size_t smem = 4 * (size_t)(a.dpad + a.vdim) * sizeof(float);
+  if (smem > 200 * 1024) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: attention with heads of size %d/%d", a.dim, a.vdim);
+  ++*launches;
+  return launch_kernel(flash_simple_kernel<T>, dim3((unsigned)(a.kv_heads * ((gq + 3) / 4)), (unsigned)a.r.rows), dim3(kThreads), smem, st, a.pdl, 1, a);
+}
+
+size_t mma_bytes(const FlashArgs& a, int mg, int kt) {
+  const size_t m = 16 * (size_t)mg, ld = (size_t)a.dpad + 8, vld = a.values_in_keys ? 0 : (size_t)a.vpad + 8;
+  return 2 * (m * ld + 2 * kt * ld + 2 * kt * vld + 2 * m * (kt + 8)) + 4 * (8 / mg) * m;
+}
+constexpr size_t kSmemMax = 226 * 1024;
+
+using FlashKernel = void (*)(FlashArgs, FlashShape);
+// The kernel with at least nv 8-column tiles per warp; null: none.
+FlashKernel pick_kernel(int mg, int nv, int kt) {
+  if (mg == 1 && kt == 64) return nv <= 2 ? flash_mma_kernel<1, 2, 64> : nv <= 4 ? flash_mma_kernel<1, 4, 64> : nv <= 8 ? flash_mma_kernel<1, 8, 64> : nullptr;
+  if (mg == 2 && kt == 64)
+    return nv <= 4 ? flash_mma_kernel<2, 4, 64> : nv <= 8 ? flash_mma_kernel<2, 8, 64> : nv <= 16 ? flash_mma_kernel<2, 16, 64> : nullptr;
+  if (mg == 2 && kt == 32) return nv <= 8 ? flash_mma_kernel<2, 8, 32> : nv <= 16 ? flash_mma_kernel<2, 16, 32> : nullptr;
+  if (mg == 4 && kt == 64)
+    return nv <= 4 ? flash_mma_kernel<4, 4, 64> : nv <= 8 ? flash_mma_kernel<4, 8, 64> : nv <= 16 ? flash_mma_kernel<4, 16, 64> : nullptr;
+  if (mg == 4 && kt == 32) return nv <= 16 ? flash_mma_kernel<4, 16, 32> : nv <= 32 ? flash_mma_kernel<4, 32, 32> : nullptr;
+  return nullptr;
+}
+
+}  // namespace
+
+tb_status launch_flash_attention(Precision p, const FlashArgs& a, cudaStream_t st, int* launches) {
+  if (a.heads < 1 || a.kv_heads < 1 || a.heads % a.kv_heads || a.dpad % 16 || a.vpad % 16 || (a.values_in_keys && (a.kv_heads != 1 || a.vpad > a.dpad)))
+    return fail(TB_ERR_SHAPE, "flash attention: bad shape");
+  if (p == Precision::kF32) return launch_simple<float>(a, st, launches);
+  const int gq = a.heads / a.kv_heads, rows = a.r.rows;
+  FlashShape sh;
+  sh.run_rows = a.one_sequence ? rows : 1;
+  const int runs = a.one_sequence ? 1 : rows;
+  const int64_t pairs = (int64_t)sh.run_rows * gq;
+  FlashKernel kern = nullptr;
+  int mg = pairs <= 16 ? 1 : (pairs <= 32 ? 2 : 4), kt = 0;
+  for (; mg <= 4 && kern == nullptr; mg *= 2) {
+    const int wn = 8 / mg, nv = (((a.vpad + wn - 1) / wn + 15) & ~15) / 8;
+    const int64_t ctas = (pairs + 16 * mg - 1) / (16 * mg) * a.kv_heads * runs;
+    // tiles of 32 keys where they alone fit, or where those of 64 are too few for the SMs
+    const bool small = mg > 1 && ctas * ((a.max_visible + 63) / 64) < sm_count();
+    for (const int k : {small ? 32 : 64, small ? 64 : 32}) {
+      if (kern == nullptr && mma_bytes(a, mg, k) <= kSmemMax) {
+        kern = pick_kernel(mg, nv, k);
+        kt = k;
+      }
+    }
+    if (kern) break;
+  }
+  if (kern == nullptr) return launch_simple<__nv_bfloat16>(a, st, launches);
+  sh.pair_tile = 16 * mg;
+  sh.tiles = (int)((pairs + sh.pair_tile - 1) / sh.pair_tile);
+  const size_t smem = mma_bytes(a, mg, kt);
+  const int64_t ctas = (int64_t)sh.tiles * a.kv_heads * runs, slots = (int64_t)sm_count() * (smem <= 112 * 1024 ? 2 : 1);
+  int64_t splits = slots / ctas;
+  const int64_t ktiles = (a.max_visible + (a.one_sequence ? sh.pair_tile / gq : 0) + kt - 1) / kt;
+  if (splits > ktiles) splits = ktiles;
+  if (splits > kMaxSplits) splits = kMaxSplits;
+  if (splits > a.part_slots / ((int64_t)rows * a.heads)) splits = a.part_slots / ((int64_t)rows * a.heads);
+  if (splits < 1) splits = 1;
+  sh.splits = (int)splits;
+  TB_TRY(launch_kernel(kern, dim3((unsigned)(sh.tiles * sh.splits), (unsigned)a.kv_heads, (unsigned)runs), dim3(kThreads), smem, st, a.pdl, 1, a, sh));
+  ++*launches;
+  if (sh.splits == 1) return TB_OK;
+  ++*launches;
+  const int cols = a.out_per_head ? a.out.kp : a.out.kp - (a.heads - 1) * a.vdim;
+  return launch_kernel(flash_merge_kernel, dim3((unsigned)a.heads, (unsigned)rows, (unsigned)((cols + 127) / 128)), dim3(128), 0, st, a.pdl, 1, a, sh.splits);
+}
+
+int64_t flash_part_slots(int64_t rows, int64_t heads) {
+  // every CTA of a wave leaves at most 64 (row, head) pairs, and a step that fills the wave is not split
+  const int64_t wave = 2 * (int64_t)sm_count() * 64, step = 2 * rows * heads;
+  return wave > step ? wave : step;
+}
+
+}  // namespace tb

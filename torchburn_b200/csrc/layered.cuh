@@ -20,8 +20,15 @@ struct LayeredStep {
   cudaEvent_t before_lm_head = nullptr;
 };
 
-tb_status layered_create(LayeredModel** out, const tb_layered_config& c, const tb_layered_layer* layers, const uint16_t* embed,
-                         const uint16_t* pos_table, const uint16_t* final_norm, tb_space space, bool snapshots);
+struct LayeredTables {
+  const uint16_t* embed = nullptr;
+  const uint16_t* embed_norm = nullptr;   // or null
+  const uint16_t* pos_table = nullptr;    // or null
+  const uint16_t* final_norm = nullptr;
+  const uint16_t* head = nullptr;         // null: embed
+};
+tb_status layered_create(LayeredModel** out, const tb_layered_config& c, const tb_layered_layer* layers, const LayeredTables& tables,
+                         tb_space space, bool snapshots);
 void layered_destroy(LayeredModel* m);
 int layered_max_rows(const LayeredModel* m);      // rows of one step
 // How far back of the furthest position written a sequence may be continued (its rings hold that much).

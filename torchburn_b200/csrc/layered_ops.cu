@@ -1,6 +1,7 @@
 // Row kernels of the layered decoder, between the projections: residual + norms + the causal convolution
-// in front of a sublayer (glue), query/key norm with the cache append, and PolyNorm.  All arithmetic is
-// fp32; the results are written as the next projection's operand.
+// in front of a sublayer (glue), query/key norm with the cache append (over the whole projection or per head),
+// the latent's norm and rotation, PolyNorm and the squared relu.  All arithmetic is fp32; the results are
+// written as the next projection's operand.
 //
 // A row is handled by a cluster of 1..8 CTAs (few rows: more CTAs, so that a decode row of several thousand
 // features is not one SM's work); block sums meet through distributed shared memory and are added in rank
@@ -126,28 +127,26 @@ __global__ void __launch_bounds__(kThreads) residual_norm_kernel(const GlueArgs 
   }
   float inv = 1.f;
   float ss[1] = {0.f};
-  if (!emb) {
-    for (int e = 0, i = tid; i < xs4; ++e, i += kThreads) {
-      float4 v = sum_partials(a.y, r, i * 4);
+  for (int e = 0, i = tid; i < xs4; ++e, i += kThreads) {
+    float4 v = f4(0.f);
+    if (!emb) {
+      v = sum_partials(a.y, r, i * 4);
       if (a.y_bias) v = add4(v, ld4(a.y_bias + i * 4));
-      s_dyn[e * kThreads + tid] = v;
-      ss[0] += dot4(v);
+    } else if (pos >= 0) {
+      v = embed4(a, tok, pos, i * 4);
     }
-    if (a.post_w) {
-      cluster_sum<1>(s_sum, 0, 1, 0, ss);
-      inv = 1.0f / sqrtf(ss[0] / (float)a.width + a.eps);
-    }
+    s_dyn[e * kThreads + tid] = v;
+    ss[0] += dot4(v);
+  }
+  if (a.post_w) {
+    cluster_sum<1>(s_sum, 0, 1, 0, ss);
+    inv = 1.0f / sqrtf(ss[0] / (float)a.width + a.eps);
   }
   ss[0] = 0.f;
   for (int e = 0, i = tid; i < xs4; ++e, i += kThreads) {
-    float4 v = f4(0.f);
-    if (emb) {
-      if (pos >= 0) v = embed4(a, tok, pos, i * 4);
-    } else {
-      const float4 y = s_dyn[e * kThreads + tid];
-      v = ld4(a.x_in + (size_t)r * a.xs + i * 4);
-      v = a.post_w ? fma4(scale4(y, inv), ld4(a.post_w + i * 4), v) : add4(v, y);
-    }
+    const float4 y = s_dyn[e * kThreads + tid];
+    float4 v = emb ? f4(0.f) : ld4(a.x_in + (size_t)r * a.xs + i * 4);
+    v = a.post_w ? fma4(scale4(y, inv), ld4(a.post_w + i * 4), v) : add4(v, y);
     ss[0] += dot4(v);
     *reinterpret_cast<float4*>(a.x_out + (size_t)r * a.xs + i * 4) = v;
     if (a.snapshot) *reinterpret_cast<float4*>(a.snapshot + (size_t)r * a.xs + i * 4) = v;
@@ -221,11 +220,17 @@ __global__ void __launch_bounds__(kThreads) glue_kernel(const GlueArgs a, const 
       if (r >= r0 && tid == 0 && crank == 0) a.r.pos[r] = pos;
     }
     float inv = 1.f;
-    if (!emb && a.y.y != nullptr) {
+    const bool source = emb || a.y.y != nullptr;
+    if (source) {
       float ss[1] = {0.f};
       for (int e = 0, i = lane4; i < xs4; ++e, i += step4) {
-        float4 v = sum_partials(a.y, r, i * 4);
-        if (a.y_bias) v = add4(v, ld4(a.y_bias + i * 4));
+        float4 v = f4(0.f);
+        if (!emb) {
+          v = sum_partials(a.y, r, i * 4);
+          if (a.y_bias) v = add4(v, ld4(a.y_bias + i * 4));
+        } else if (live) {
+          v = embed4(a, tok, pos, i * 4);
+        }
         s_x[e * kThreads + tid] = v;
         ss[0] += dot4(v);
       }
@@ -237,15 +242,10 @@ __global__ void __launch_bounds__(kThreads) glue_kernel(const GlueArgs a, const 
     }
     float ss[1] = {0.f};
     for (int e = 0, i = lane4; i < xs4; ++e, i += step4) {
-      float4 v = f4(0.f);
-      if (emb) {
-        if (live) v = embed4(a, tok, pos, i * 4);
-      } else {
-        v = ld4(a.x_in + (size_t)r * a.xs + i * 4);
-        if (a.y.y != nullptr) {
-          const float4 y = s_x[e * kThreads + tid];
-          v = a.post_w ? fma4(scale4(y, inv), ld4(a.post_w + i * 4), v) : add4(v, y);
-        }
+      float4 v = emb ? f4(0.f) : ld4(a.x_in + (size_t)r * a.xs + i * 4);
+      if (source) {
+        const float4 y = s_x[e * kThreads + tid];
+        v = a.post_w ? fma4(scale4(y, inv), ld4(a.post_w + i * 4), v) : add4(v, y);
       }
       s_x[e * kThreads + tid] = v;
       ss[0] += dot4(v);
@@ -300,7 +300,7 @@ __global__ void __launch_bounds__(kThreads) glue_step_kernel(const GlueArgs a) {
   float4 pw = zero, ow = zero, bias = zero, cw[kStepTaps];
   if (in) {
     pw = ld4(a.pre_w + i * 4);
-    if (!emb && a.post_w) ow = ld4(a.post_w + i * 4);
+    if (a.post_w) ow = ld4(a.post_w + i * 4);
     if (!emb && a.y_bias) bias = ld4(a.y_bias + i * 4);
 #pragma unroll
     for (int j = 0; j < kStepTaps; ++j)
@@ -327,9 +327,8 @@ __global__ void __launch_bounds__(kThreads) glue_step_kernel(const GlueArgs a) {
       if (j < taps && j <= pos) prev[j] = ld4(state + (size_t)((pos - j) & (a.ring - 1)) * a.xs);
   }
   float ss[1];
-  if (emb) {
-    if (in && pos >= 0) v = embed4(a, tok, pos, i * 4);
-  } else if (a.post_w) {
+  if (emb && in && pos >= 0) v = embed4(a, tok, pos, i * 4);
+  if (a.post_w) {
     ss[0] = dot4(v);
     cluster_sum<1>(s_sum, 0, csize, crank, ss);
     v = fma4(scale4(v, 1.0f / sqrtf(ss[0] / (float)a.width + a.eps)), ow, x);
@@ -408,6 +407,156 @@ __global__ void __launch_bounds__(kThreads) qkv_prep_kernel(const QkvPrepArgs a,
       }
     }
   }
+}
+
+// One column of a projection: its partial sums in order.
+__device__ __forceinline__ float sum_column(const PartialSums& y, int row, int col) {
+  const float* p = y.y + (size_t)row * y.ldy + col;
+  float t[kMaxParts];
+#pragma unroll
+  for (int s = 0; s < kMaxParts; ++s)
+    if (s < y.splits) t[s] = p[(size_t)s * y.split_stride];
+  float v = t[0];
+#pragma unroll
+  for (int s = 1; s < kMaxParts; ++s)
+    if (s < y.splits) v += t[s];
+  return v;
+}
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+
+// Per head: a warp takes one head of q, k or v through its norm (or the value mixing) to where it goes; one more
+// warp per 32 heads does the gates.  grid (warps of a row / 8, rows)
+template <typename T>
+__global__ void __launch_bounds__(kThreads) heads_prep_kernel(const HeadsPrepArgs a) {
+  constexpr int KEEP = 8;                  // values a lane keeps between the norm's two passes
+  const int lane = threadIdx.x & 31, r = (int)blockIdx.y;
+  int u = (int)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
+  grid_dep_launch();
+  grid_dep_wait();
+  const int pos = a.r.pos[r];
+  const size_t crow = pos < 0 ? 0 : (size_t)a.r.slots[r] * a.geom.rows + a.geom.row_of(pos);
+  if (u < a.heads + a.kv_heads) {
+    const bool is_q = u < a.heads;
+    const int h = is_q ? u : u - a.heads, col = (is_q ? a.q_off : a.k_off) + h * a.dim;
+    float v[KEEP], ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j)
+      if (lane + 32 * j < a.dim) {
+        v[j] = sum_column(a.y, r, col + lane + 32 * j);
+        ss = fmaf(v[j], v[j], ss);
+      }
+    for (int c = lane + 32 * KEEP; c < a.dim; c += 32) {
+      const float x = sum_column(a.y, r, col + c);
+      ss = fmaf(x, x, ss);
+    }
+    const float inv = a.unit_norm ? 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps) : 1.f;
+    T* dst = is_q ? static_cast<T*>(a.q) + ((size_t)r * a.heads + h) * a.dpad
+                  : static_cast<T*>(a.k_cache) + crow * (size_t)(a.kv_heads * a.dpad) + h * a.dpad;
+    if (!is_q && pos < 0) return;
+#pragma unroll
+    for (int j = 0; j < KEEP; ++j)
+      if (lane + 32 * j < a.dim) dst[lane + 32 * j] = (T)(v[j] * inv);
+    for (int c = lane + 32 * KEEP; c < a.dim; c += 32) dst[c] = (T)(sum_column(a.y, r, col + c) * inv);
+    return;
+  }
+  u -= a.heads + a.kv_heads;
+  if (u < a.kv_heads) {
+    T* dst = static_cast<T*>(a.v_cache) + crow * (size_t)(a.kv_heads * a.vpad) + u * a.vpad;
+    float* first = a.v_first ? a.v_first + (size_t)r * a.kv_heads * a.vdim + u * a.vdim : nullptr;
+    for (int c = lane; c < a.vdim; c += 32) {
+      float v = sum_column(a.y, r, a.v_off + u * a.vdim + c);
+      if (first && a.keep_first_values) first[c] = v;
+      else if (first) v = fmaf(a.mix, first[c], (1.f - a.mix) * v);
+      if (pos >= 0) dst[c] = (T)v;
+    }
+    return;
+  }
+  const int g = (u - a.kv_heads) * 32 + lane;
+  if (a.gate && g < a.heads) a.gate[(size_t)r * a.heads + g] = 1.0f / (1.0f + expf(-sum_column(a.y, r, a.g_off + g)));
+}
+
+// Rotation of dimensions 2i, 2i + 1 below `dims` at position pos; the others pass.
+__device__ __forceinline__ float rotated(const float2* table, int dims, int pos, int c, float own, float other) {
+  if (c >= dims || pos < 0) return own;
+  const float2 cs = table[(size_t)pos * (dims >> 1) + (c >> 1)];
+  return (c & 1) ? fmaf(own, cs.x, other * cs.y) : fmaf(own, cs.x, -other * cs.y);
+}
+
+// The latents of a row.  grid (2, rows): block 0 the query latent, normed, as the next product's operand; block 1
+// the key/value latent, normed, and the shared rotated key part, into the cache.
+template <typename T>
+__global__ void __launch_bounds__(kThreads) latent_prep_kernel(const LatentPrepArgs a) {
+  extern __shared__ float s_lat[];
+  __shared__ ClusterSum<1> s_sum;
+  const int tid = threadIdx.x, r = (int)blockIdx.y;
+  const bool is_q = blockIdx.x == 0;
+  const int n = is_q ? a.q_rank : a.kv_rank, off = is_q ? 0 : a.kv_off;
+  grid_dep_launch();
+  grid_dep_wait();
+  const int pos = a.r.pos[r];
+  float ss[1] = {0.f};
+  for (int c = tid; c < n; c += kThreads) {
+    const float v = sum_column(a.y, r, off + c);
+    s_lat[c] = v;
+    ss[0] = fmaf(v, v, ss[0]);
+  }
+  cluster_sum<1>(s_sum, 0, 1, 0, ss);
+  const float inv = 1.0f / sqrtf(ss[0] / (float)n + a.eps);
+  if (is_q) {
+    for (int c = tid; c < a.out.kp; c += kThreads) act_store1<sizeof(T) == 2>(a.out, r, c, c < n ? s_lat[c] * inv * a.q_norm[c] : 0.f);
+    return;
+  }
+  if (pos < 0) return;
+  T* row = static_cast<T*>(a.cache) + ((size_t)a.r.slots[r] * a.geom.rows + a.geom.row_of(pos)) * (size_t)a.dpad;
+  for (int c = tid; c < n; c += kThreads) row[c] = (T)(s_lat[c] * inv * a.kv_norm[c]);
+  for (int c = tid; c < a.rot_dim; c += kThreads) {
+    const float own = sum_column(a.y, r, off + n + c), other = c < a.rot_dims ? sum_column(a.y, r, off + n + (c ^ 1)) : 0.f;
+    row[n + c] = (T)rotated(a.table, a.rot_dims, pos, c, own, other);
+  }
+}
+
+// The heads' queries after the up-projection: the unrotated part as the operand of the product with the head's
+// key matrix, the rotated part behind the place of that product in the query.  Warp per head, grid (heads / 8, rows)
+template <typename T>
+__global__ void __launch_bounds__(kThreads) latent_query_kernel(const LatentQueryArgs a) {
+  const int lane = threadIdx.x & 31, r = (int)blockIdx.y, h = (int)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
+  grid_dep_launch();
+  grid_dep_wait();
+  if (h >= a.heads) return;
+  const int pos = a.r.pos[r], col = h * (a.dim + a.rot_dim);
+  ActOperand out = a.out;
+  out.data = static_cast<unsigned char*>(out.data) + (size_t)h * out.mp * out.kp * sizeof(T);
+  for (int c = lane; c < out.kp; c += 32) act_store1<sizeof(T) == 2>(out, r, c, c < a.dim ? sum_column(a.y, r, col + c) : 0.f);
+  T* q = static_cast<T*>(a.q) + ((size_t)r * a.heads + h) * a.dpad + a.kv_rank;
+  for (int c = lane; c < a.rot_dim; c += 32) {
+    const float own = sum_column(a.y, r, col + a.dim + c), other = c < a.rot_dims ? sum_column(a.y, r, col + a.dim + (c ^ 1)) : 0.f;
+    q[c] = (T)rotated(a.table, a.rot_dims, pos, c, own, other);
+  }
+}
+
+// grid (columns / 1024, rows)
+template <bool BF16>
+__global__ void __launch_bounds__(kThreads) relu2_kernel(const PartialSums z, const ActOperand out) {
+  const int k = ((int)blockIdx.x * kThreads + threadIdx.x) * 4, r = (int)blockIdx.y;
+  grid_dep_launch();
+  grid_dep_wait();
+  if (k >= out.kp) return;
+  float4 v = sum_partials(z, r, k);
+  v = make_float4(fmaxf(v.x, 0.f), fmaxf(v.y, 0.f), fmaxf(v.z, 0.f), fmaxf(v.w, 0.f));
+  act_store4<BF16>(out, r, k, mul4(v, v));
+}
+
+// Angles in fp64, so that a far position turns by its angle and not by a rounded one.
+__global__ void __launch_bounds__(kThreads) rotation_table_kernel(float2* table, int64_t n, int half, double base) {
+  const int64_t i = (int64_t)blockIdx.x * kThreads + threadIdx.x;
+  if (i >= n) return;
+  double sn, cs;
+  sincos((double)(i / half) * pow(base, -(double)(i % half) / (double)half), &sn, &cs);
+  table[i] = make_float2((float)cs, (float)sn);
 }
 
 template <bool BF16>
@@ -504,6 +653,41 @@ tb_status launch_qkv_prep(Precision p, const QkvPrepArgs& a, cudaStream_t st) {
   const dim3 grid((unsigned)(a.r.rows * c));
   if (p == Precision::kBf16) return launch_kernel(qkv_prep_kernel<__nv_bfloat16>, grid, dim3(kThreads), smem, st, a.pdl, c, a, e4);
   return launch_kernel(qkv_prep_kernel<float>, grid, dim3(kThreads), smem, st, a.pdl, c, a, e4);
+}
+
+tb_status launch_heads_prep(Precision p, const HeadsPrepArgs& a, cudaStream_t st) {
+  const int warps = a.heads + 2 * a.kv_heads + (a.gate ? (a.heads + 31) / 32 : 0);
+  const dim3 grid((unsigned)((warps + kThreads / 32 - 1) / (kThreads / 32)), (unsigned)a.r.rows);
+  return p == Precision::kBf16 ? launch_kernel(heads_prep_kernel<__nv_bfloat16>, grid, dim3(kThreads), 0, st, a.pdl, 1, a)
+                               : launch_kernel(heads_prep_kernel<float>, grid, dim3(kThreads), 0, st, a.pdl, 1, a);
+}
+
+tb_status launch_latent_prep(Precision p, const LatentPrepArgs& a, cudaStream_t st) {
+  const size_t smem = (size_t)(a.q_rank > a.kv_rank ? a.q_rank : a.kv_rank) * sizeof(float);
+  if (smem > 200 * 1024) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: latents of %d and %d", a.q_rank, a.kv_rank);
+  const dim3 grid(2, (unsigned)a.r.rows);
+  return p == Precision::kBf16 ? launch_kernel(latent_prep_kernel<__nv_bfloat16>, grid, dim3(kThreads), smem, st, a.pdl, 1, a)
+                               : launch_kernel(latent_prep_kernel<float>, grid, dim3(kThreads), smem, st, a.pdl, 1, a);
+}
+
+tb_status launch_latent_query(Precision p, const LatentQueryArgs& a, cudaStream_t st) {
+  const dim3 grid((unsigned)((a.heads + kThreads / 32 - 1) / (kThreads / 32)), (unsigned)a.r.rows);
+  return p == Precision::kBf16 ? launch_kernel(latent_query_kernel<__nv_bfloat16>, grid, dim3(kThreads), 0, st, a.pdl, 1, a)
+                               : launch_kernel(latent_query_kernel<float>, grid, dim3(kThreads), 0, st, a.pdl, 1, a);
+}
+
+tb_status launch_relu2(Precision p, int rows, const PartialSums& z, const ActOperand& out, bool pdl, cudaStream_t st) {
+  const dim3 grid((unsigned)((out.kp / 4 + kThreads - 1) / kThreads), (unsigned)rows);
+  return p == Precision::kBf16 ? launch_kernel(relu2_kernel<true>, grid, dim3(kThreads), 0, st, pdl, 1, z, out)
+                               : launch_kernel(relu2_kernel<false>, grid, dim3(kThreads), 0, st, pdl, 1, z, out);
+}
+
+tb_status fill_rotation_table(float2* table, int64_t positions, int dims, double base) {
+  const int64_t n = positions * (dims / 2);
+  if (n == 0) return TB_OK;
+  rotation_table_kernel<<<(unsigned)((n + kThreads - 1) / kThreads), kThreads>>>(table, n, dims / 2, base);
+  TB_CUDA_TRY(cudaGetLastError());
+  return TB_OK;
 }
 
 tb_status launch_poly_norm(Precision p, const PolyNormArgs& a, cudaStream_t st) {

@@ -48,34 +48,6 @@ __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], 
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// The block's keys.  pos0: position of the block's first query, last: of its last one.
-struct BlockKeys {
-  int pos0, lo, nk, count;
-  __device__ BlockKeys(int p0, int last, int window, int keep_first) : pos0(p0) {
-    const VisibleRange a(p0, window, keep_first);
-    lo = a.lo;
-    nk = a.nk;
-    count = nk + last - lo + 1;
-  }
-  __device__ int position(int v) const { return v < nk ? v : v - nk + lo; }
-};
-
-// Cache rows of numbered keys near number v0 (less than a ring apart) with one division for all of them.
-struct RunRows {
-  int nk, lo, keep, ring, base_pos, base_row;
-  __device__ RunRows(const BlockKeys& k, const CacheGeom& g, int v0) : nk(k.nk), lo(k.lo), keep(g.keep), ring(g.ring) {
-    const int p = k.position(v0 > k.nk ? v0 : k.nk);   // first key of the run at or after v0
-    base_pos = p > keep ? p : keep;
-    base_row = g.row_of(base_pos);
-  }
-  __device__ int row(int v) const {
-    const int p = v < nk ? v : v - nk + lo;
-    if (ring == 0 || p < keep) return p;
-    const int r = base_row + (p - base_pos);
-    return r >= keep + ring ? r - ring : r;
-  }
-};
-
 struct MmaShape {
   int64_t stride;   // floats per (row, head) of the score scratch
   int row0, rows;   // rows of this pass

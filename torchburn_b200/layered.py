@@ -16,7 +16,8 @@ from .decoder import DecoderHandle, _is_torch
 @dataclass
 class LayerSpec:
     """Sizes and constants of one layer, and its tensors by the names of ``tb_layered_layer`` (bfloat16: raw
-    16-bit numpy arrays or torch tensors; a missing optional tensor leaves its mechanism out)."""
+    16-bit numpy arrays or torch tensors; a missing optional tensor leaves its mechanism out).  A layer with a
+    ``kv_rank`` is latent attention (``num_kv_heads`` 1, ``head_dim`` its unrotated part)."""
     num_heads: int
     num_kv_heads: int
     head_dim: int
@@ -27,6 +28,20 @@ class LayerSpec:
     ff: int = 0                    # 0: no feed-forward
     weights_of: Optional[int] = None
     tensors: Dict[str, Any] = field(default_factory=dict)
+    activation: str = "polynorm"   # of the feed-forward: polynorm, relu2
+    mask_chunk: int = 0            # 0: no chunks
+    qk_unit_norm: bool = False     # per-head norm of queries and keys without a weight
+    score_softcap: float = 0.0     # 0: none
+    distance_bias: float = 0.0     # slope 2^(-distance_bias (h + 1) / heads); 0: none
+    value_mix: bool = False
+    q_rank: int = 0
+    kv_rank: int = 0
+    rot_dim: int = 0
+    rot_dims: int = 0
+    rot_base: float = 0.0
+
+
+_MLP = {"polynorm": _lib.TB_MLP_POLYNORM, "relu2": _lib.TB_MLP_RELU2}
 
 
 class _Bf16Operands:
@@ -65,7 +80,8 @@ class LayeredDecoder(DecoderHandle):
 
     def __init__(self, layers: Sequence[LayerSpec], embed, final_norm, pos_table=None, *, hidden_size: int, vocab_size: int,
                  norm_eps: float, max_seq_len: int, embed_scale: float = 1.0, conv_taps: int = 0, dtype: str = "bfloat16",
-                 max_batch: int = 1, prefill_rows: int = 0, debug: bool = False, pdl: bool = True):
+                 max_batch: int = 1, prefill_rows: int = 0, debug: bool = False, pdl: bool = True, embed_norm=None, head=None,
+                 norm_offset: float = 0.0):
         self._h = None
         if dtype not in _lib.TB_PRECISION:
             raise ValueError(f"dtype {dtype!r}: expected one of {sorted(_lib.TB_PRECISION)}")
@@ -75,19 +91,24 @@ class LayeredDecoder(DecoderHandle):
             unknown = set(s.tensors) - set(LAYERED_TENSORS)
             if unknown:
                 raise ValueError(f"unknown layer tensors {sorted(unknown)}")
-            dst.mixer = _lib.TB_MIXER_ATTENTION
-            dst.mlp = _lib.TB_MLP_POLYNORM if s.ff else _lib.TB_MLP_NONE
+            if s.activation not in _MLP:
+                raise ValueError(f"activation {s.activation!r}: expected one of {sorted(_MLP)}")
+            dst.mixer = _lib.TB_MIXER_LATENT if s.kv_rank else _lib.TB_MIXER_ATTENTION
+            dst.mlp = _MLP[s.activation] if s.ff else _lib.TB_MLP_NONE
             dst.weights_of = -1 if s.weights_of is None else s.weights_of
             dst.num_heads, dst.num_kv_heads, dst.head_dim, dst.value_dim = s.num_heads, s.num_kv_heads, s.head_dim, s.value_dim
             dst.mask_window, dst.mask_keep_first, dst.score_scale, dst.ff = s.mask_window, s.mask_keep_first, s.score_scale, s.ff
+            dst.mask_chunk, dst.qk_unit_norm, dst.score_softcap, dst.distance_bias = s.mask_chunk, s.qk_unit_norm, s.score_softcap, s.distance_bias
+            dst.value_mix, dst.q_rank, dst.kv_rank = s.value_mix, s.q_rank, s.kv_rank
+            dst.rot_dim, dst.rot_dims, dst.rot_base = s.rot_dim, s.rot_dims, s.rot_base
             for name, t in s.tensors.items():
                 setattr(dst, name, ops.ptr(t))
         flags = (_lib.TB_DECODER_NO_GRAPH if debug else 0) | (0 if pdl else _lib.TB_DECODER_NO_PDL)
         self.cfg = LayeredConfig(vocab_size=vocab_size, hidden_size=hidden_size, num_layers=len(layers), conv_taps=conv_taps,
                                  norm_eps=norm_eps, embed_scale=embed_scale, max_seq_len=max_seq_len, max_batch=max_batch,
-                                 prefill_rows=prefill_rows, precision=_lib.TB_PRECISION[dtype], flags=flags)
-        emb_p, pos_p, fn_p = ops.ptr(embed), ops.ptr(pos_table), ops.ptr(final_norm)
+                                 prefill_rows=prefill_rows, precision=_lib.TB_PRECISION[dtype], flags=flags, norm_offset=norm_offset)
+        tables = [ops.ptr(t) for t in (embed, embed_norm, pos_table, final_norm, head)]
         h = C.c_void_p()
-        check(lib().tb_decoder_create_layered(C.byref(h), C.byref(self.cfg), C.cast(arr, C.c_void_p), emb_p, pos_p, fn_p,
+        check(lib().tb_decoder_create_layered(C.byref(h), C.byref(self.cfg), C.cast(arr, C.c_void_p), *tables,
                                               ops.space if ops.space is not None else TB_HOST))
         self._adopt(h, vocab_size, max_batch, max_seq_len)

@@ -61,6 +61,12 @@ def _load_dabevik(model_dir, config, dtype, max_seq_len, **options):
     return dabevik.build(config, checkpoint.read_model_tensors(model_dir), dtype, max_seq_len, **options)
 
 
+def _load_sukalorn(model_dir, config, dtype, max_seq_len, **options):
+    from . import sukalorn
+
+    return sukalorn.build(config, checkpoint.read_model_tensors(model_dir), dtype, max_seq_len, **options)
+
+
 def _load_int4(model_dir, config, dtype, max_seq_len, group_size: int = 64, **options):
     """Llama / Qwen2 style checkpoints on the INT4 decoder: the folder's quantized cache if there is one, else
     its float tensors quantized on the GPU (python/torchburn/llm/loader.py:92-173, 376-537)."""
@@ -96,5 +102,6 @@ def _load_int4(model_dir, config, dtype, max_seq_len, group_size: int = 64, **op
 
 
 register(Design("dabevik", lambda c: c.get("architecture") == "Dabevik", _load_dabevik, ("bfloat16", "float32"), "dense"))
+register(Design("sukalorn", lambda c: c.get("architecture") == "Sukalorn", _load_sukalorn, ("bfloat16", "float32"), "dense"))
 register(Design("llama-int4", lambda c: c.get("model_type") in ("llama", "qwen2") or bool(
     {"LlamaForCausalLM", "Qwen2ForCausalLM"} & set(c.get("architectures") or ())), _load_int4, ("int4",)))

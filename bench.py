@@ -1,7 +1,7 @@
 """Headline benchmark: INT4 decode tokens/s of a Llama-3-8B-shaped model on B200(s).
 
     python bench.py [--gpus N] [--steps K] [--warmup W] [--batch B] [--impl reference]
-    python bench.py --design dabevik     # a layered design beside the INT4 decoder (another JSON line)
+    python bench.py --design sukalorn    # a layered design beside the closest other model (another JSON line); or dabevik
 
 N=1 workload: the headline configuration "Llama-3-8B-architecture INT4 decode" - hidden 4096,
 32 layers, 32 q / 8 kv heads, head_dim 128, intermediate 14336, vocab 128256,
@@ -771,21 +771,34 @@ def time_config3(torch, tb, device, args):
 
 
 # ----------------------------------------------------------------- layered designs (--design)
-# Layers like a real model's, random weights.  The feed-forward of the design has two matrices where the INT4
-# model has three: 1.5 times the width gives both the same number of weights.
+# Layers like a real model's, random weights.  The feed-forward of the designs has two matrices where the INT4
+# model has three: 1.5 times the width gives both the same number of weights.  latent: the sizes of Sukalorn's
+# latent attention, in three layers of eight.
 DESIGN_SIZES = {
-    "llama-3-8b-layers": dict(width=4096, layers=8, heads=32, kv_heads=8, dim=128, ff=21504, vocab=128256),
-    "qwen2.5-0.5b": dict(width=896, layers=24, heads=14, kv_heads=2, dim=64, ff=7296, vocab=151936),
+    "llama-3-8b-layers": dict(width=4096, layers=8, heads=32, kv_heads=8, dim=128, ff=21504, vocab=128256,
+                              latent=dict(q_rank=1536, kv_rank=512, dim=128, rot_dim=64, vdim=128)),
+    "qwen2.5-0.5b": dict(width=896, layers=24, heads=14, kv_heads=2, dim=64, ff=7296, vocab=151936,
+                         latent=dict(q_rank=448, kv_rank=256, dim=64, rot_dim=32, vdim=64)),
 }
 
 
+class RandomWeights:
+    """bfloat16 tensors on the device, and how many numbers they have."""
+
+    def __init__(self, torch, device, seed):
+        self.torch, self.device, self.count = torch, device, 0
+        self.gen = torch.Generator(device).manual_seed(seed)
+
+    def __call__(self, *shape, std=0.02, mean=0.0):
+        self.count += int(np.prod(shape))
+        return (mean + std * self.torch.randn(*shape, device=self.device, generator=self.gen)).to(self.torch.bfloat16)
+
+
+# Builders return (decoder, stats): weights read per token without and with the output matrix, cache bytes per position, and
+# the floating-point operations of one query position with one key (query/key and value products, keys written out).
 def build_dabevik(torch, tb, z, device, context, max_batch, prefill_rows, seed=3, dtype="bfloat16"):
     """A Dabevik model of these sizes; the window spans the context, four first tokens are kept."""
-    gen = torch.Generator(device).manual_seed(seed)
-
-    def rnd(*shape, std=0.02, mean=0.0):
-        return (mean + std * torch.randn(*shape, device=device, generator=gen)).to(torch.bfloat16)
-
+    rnd = RandomWeights(torch, device, seed)
     w, h, kv, d, ff = z["width"], z["heads"], z["kv_heads"], z["dim"], z["ff"]
     positions = context + 512
     specs = []
@@ -795,14 +808,51 @@ def build_dabevik(torch, tb, z, device, context, max_batch, prefill_rows, seed=3
                  v_w=rnd(kv * d, w), v_b=rnd(kv * d), q_norm=rnd(h * d, mean=1.0), k_norm=rnd(kv * d, mean=1.0), talk=rnd(h, h, std=0.2),
                  o_w=rnd(w, h * d), o_b=rnd(w), up_w=rnd(ff, w), down_w=rnd(w, ff), act=rnd(4, std=0.5))
         specs.append(tb.LayerSpec(h, kv, d, d, d ** -0.5, context, 4, ff, None, t))
-    return tb.LayeredDecoder(specs, rnd(z["vocab"], w, std=1.0), rnd(w, mean=1.0), rnd(positions, w), hidden_size=w, vocab_size=z["vocab"],
-                             norm_eps=1e-5, max_seq_len=positions, embed_scale=1.0, conv_taps=4, max_batch=max_batch,
-                             prefill_rows=prefill_rows, dtype=dtype)
+    dec = tb.LayeredDecoder(specs, rnd(z["vocab"], w, std=1.0), rnd(w, mean=1.0), rnd(positions, w), hidden_size=w, vocab_size=z["vocab"],
+                            norm_eps=1e-5, max_seq_len=positions, embed_scale=1.0, conv_taps=4, max_batch=max_batch,
+                            prefill_rows=prefill_rows, dtype=dtype)
+    body = z["layers"] * (w * d * (2 * h + 2 * kv) + 2 * w * ff)
+    return dec, dict(body=body, all=body + z["vocab"] * w, kv=z["layers"] * 2 * kv * d * 2, key_flops=z["layers"] * 4.0 * h * d)
+
+
+def build_sukalorn(torch, tb, z, device, context, max_batch, prefill_rows, seed=3, dtype="bfloat16"):
+    """A Sukalorn model of these sizes: layers attention, latent, attention, attention, latent, ...; one chunk spans the context."""
+    rnd = RandomWeights(torch, device, seed)
+    w, h, kv, d, ff, lat = z["width"], z["heads"], z["kv_heads"], z["dim"], z["ff"], z["latent"]
+    positions = context + 512
+    specs, kv_bytes, key_flops = [], 0, 0.0
+    tables = dict(embed=rnd(z["vocab"], w, std=1.0), embed_norm=rnd(w), final_norm=rnd(w))
+    rnd.count = 0
+    for i in range(z["layers"]):
+        common = dict(ff=ff, activation="relu2")
+        t = dict(norm1=rnd(w), norm2=rnd(w), up_w=rnd(ff, w), down_w=rnd(w, ff))
+        if i % 3 == 1:
+            qr, kr, ld, rd, vd = lat["q_rank"], lat["kv_rank"], lat["dim"], lat["rot_dim"], lat["vdim"]
+            t.update(dq_w=rnd(qr, w), dq_norm=rnd(qr, mean=1.0), uq_w=rnd(h * (ld + rd), qr), dkv_w=rnd(kr + rd, w), dkv_norm=rnd(kr, mean=1.0),
+                     uk_w=rnd(h * ld, kr), uv_w=rnd(h * vd, kr), o_w=rnd(w, h * vd))
+            specs.append(tb.LayerSpec(h, 1, ld, vd, (ld + rd) ** -0.5, tensors=t, q_rank=qr, kv_rank=kr, rot_dim=rd, rot_dims=rd, rot_base=50000.0, **common))
+            kv_bytes += (kr + rd) * 2
+            key_flops += 2.0 * h * (ld + rd + vd)
+        else:
+            t.update(q_w=rnd(h * d, w), k_w=rnd(kv * d, w), v_w=rnd(kv * d, w), gate_w=rnd(h, w), o_w=rnd(w, h * d), vmix=rnd(1, std=0.1, mean=0.5))
+            specs.append(tb.LayerSpec(h, kv, d, d, d ** -0.5, tensors=t, mask_chunk=positions, qk_unit_norm=True, score_softcap=50.0, distance_bias=8.0,
+                                      value_mix=True, **common))
+            kv_bytes += 2 * kv * d * 2
+            key_flops += 4.0 * h * d
+    body = rnd.count
+    dec = tb.LayeredDecoder(specs, tables["embed"], tables["final_norm"], embed_norm=tables["embed_norm"], head=rnd(z["vocab"], w), hidden_size=w,
+                            vocab_size=z["vocab"], norm_eps=1e-6, norm_offset=1.0, max_seq_len=positions, max_batch=max_batch,
+                            prefill_rows=prefill_rows, dtype=dtype)
+    return dec, dict(body=body, all=body + z["vocab"] * w, kv=kv_bytes, key_flops=key_flops)
+
+
+DESIGNS = {"dabevik": build_dabevik, "sukalorn": build_sukalorn}
 
 
 def run_design(args):
-    """Decode and prompt throughput of a layered design beside the INT4 decoder of equal size: CUDA events on the
-    decoder's stream around K steps (decode), wall clock around whole prompts (token ids in, last logits left on the device)."""
+    """Decode and prompt throughput of a layered design beside the closest other model of equal size (Dabevik: the INT4
+    decoder; the others: Dabevik): CUDA events on the decoder's stream around K steps (decode), wall clock around whole prompts
+    (token ids in, last logits left on the device)."""
     import torch
 
     import torchburn_b200 as tb
@@ -829,47 +879,53 @@ def run_design(args):
             times.append((time.perf_counter() - t0) * 1e3)
         return float(np.median(times))
 
+    def prompt_row(ms, flops):
+        return {"tokens": ctx, "ms": ms, "tokens_per_s": ctx * 1e3 / ms, "frac_of_bf16_peak": flops / (ms * 1e-3) / 1e12 / tflops}
+
+    def layered(design, z, ids, r):
+        build = DESIGNS[design]
+        for rows in (512, 1024):
+            dec, stats = build(torch, tb, z, device, ctx, 1, rows)
+            # a position of the prompt sees half of it on average
+            flops = ctx * (2.0 * stats["body"] + stats["key_flops"] * (ctx / 2))
+            r["prompt"][f"{design}_{rows}_rows"] = prompt_row(prompt_ms(lambda: dec.prefill_tokens(ids, 0)), flops)
+            dec.close()
+        dec, stats = build(torch, tb, z, device, ctx, max(batches), 512)
+        for s in range(max(batches)):
+            dec.extend(ids[:ctx - 256], 0, seq=s)
+        for b in batches:
+            ms = float(np.median(timed_steps(torch, None, tb, dec, device, 1, b, ctx - 256, K, W, args.repeats))) / K
+            by = 2.0 * stats["all"] + b * (ctx - 256 + W + K // 2) * stats["kv"]
+            r["decode"][f"{design}_batch{b}"] = {"tokens_per_s": b * 1e3 / ms, "ms_per_step": ms, "launches_per_step": dec.launches_per_step(),
+                                                 "frac_of_hbm_peak": by / (ms * 1e-3) / 1e9 / peak}
+        dec.close()
+
+    def int4(z, ids, r):
+        """The INT4 decoder with as many weights, heads and positions as a Dabevik model."""
+        c = dict(vocab_size=z["vocab"], hidden_size=z["width"], intermediate_size=z["ff"] * 2 // 3, num_layers=z["layers"], num_heads=z["heads"],
+                 num_kv_heads=z["kv_heads"], head_dim=z["dim"], group_size=32, rms_norm_eps=1e-6, rope_theta=500000.0)
+        model = build_model(torch, tb, c, device, 1, 0)
+        dec = make_decoder(tb, c, model, ctx + 512, max(batches), 1, 0, args)
+        prefill_kv(torch, dec, c, device, ctx - 256, max(batches), 1, 0)
+        for b in batches:
+            ms = float(np.median(timed_steps(torch, None, tb, dec, device, 1, b, ctx - 256, K, W, args.repeats))) / K
+            by = step_weight_bytes(c) + b * kv_bytes_per_seq(c, ctx - 256 + W + K // 2)
+            r["decode"][f"int4_batch{b}"] = {"tokens_per_s": b * 1e3 / ms, "ms_per_step": ms, "launches_per_step": dec.launches_per_step(),
+                                             "frac_of_hbm_peak": by / (ms * 1e-3) / 1e9 / peak}
+        body = z["layers"] * (z["width"] * z["dim"] * (2 * z["heads"] + 2 * z["kv_heads"]) + 2 * z["width"] * z["ff"])
+        flops = ctx * (2.0 * (body + z["vocab"] * z["width"]) + 4.0 * z["layers"] * z["heads"] * z["dim"] * (ctx / 2))
+        r["prompt"]["int4_32_rows"] = prompt_row(prompt_ms(lambda: dec.prefill_tokens(ids, 0)), flops)
+        dec.close()
+
     with ClockSampler(0) as clocks:
         for name, z in DESIGN_SIZES.items():
             ids = np.random.default_rng(1).integers(0, z["vocab"], ctx).tolist()
             r = {"size": name, "layers": z["layers"], "context": ctx, "decode": {}, "prompt": {}}
-            body = z["layers"] * (z["width"] * z["dim"] * (2 * z["heads"] + 2 * z["kv_heads"]) + 2 * z["width"] * z["ff"])
-            head = z["vocab"] * z["width"]
-            # keys the positions of the prompt see, on average, times the query/key and value products of a position and key
-            attn_flops = 4.0 * z["layers"] * z["heads"] * z["dim"] * (ctx / 2)
-            for rows in (512, 1024):
-                dec = build_dabevik(torch, tb, z, device, ctx, 1, rows)
-                ms = prompt_ms(lambda: dec.prefill_tokens(ids, 0))
-                r["prompt"][f"dabevik_{rows}_rows"] = {"tokens": ctx, "ms": ms, "tokens_per_s": ctx * 1e3 / ms,
-                                                      "frac_of_bf16_peak": ctx * (2.0 * body + attn_flops) / (ms * 1e-3) / 1e12 / tflops}
-                dec.close()
-            dec = build_dabevik(torch, tb, z, device, ctx, max(batches), 512)
-            for s in range(max(batches)):
-                dec.extend(ids[:ctx - 256], 0, seq=s)
-            for b in batches:
-                start = ctx - 256 + W
-                ms = float(np.median(timed_steps(torch, None, tb, dec, device, 1, b, ctx - 256, K, W, args.repeats))) / K
-                kv = z["layers"] * b * (start + K // 2) * 2 * z["kv_heads"] * z["dim"] * 2
-                by = 2.0 * (body + head) + kv
-                r["decode"][f"dabevik_batch{b}"] = {"tokens_per_s": b * 1e3 / ms, "ms_per_step": ms, "launches_per_step": dec.launches_per_step(),
-                                                    "frac_of_hbm_peak": by / (ms * 1e-3) / 1e9 / peak}
-            dec.close()
-            # the INT4 decoder with the same weights count, heads and context
-            c = dict(vocab_size=z["vocab"], hidden_size=z["width"], intermediate_size=z["ff"] * 2 // 3, num_layers=z["layers"], num_heads=z["heads"],
-                     num_kv_heads=z["kv_heads"], head_dim=z["dim"], group_size=32, rms_norm_eps=1e-6, rope_theta=500000.0)
-            model = build_model(torch, tb, c, device, 1, 0)
-            dec = make_decoder(tb, c, model, ctx + 512, max(batches), 1, 0, args)
-            prefill_kv(torch, dec, c, device, ctx - 256, max(batches), 1, 0)
-            for b in batches:
-                ms = float(np.median(timed_steps(torch, None, tb, dec, device, 1, b, ctx - 256, K, W, args.repeats))) / K
-                by = step_weight_bytes(c) + b * kv_bytes_per_seq(c, ctx - 256 + W + K // 2)
-                r["decode"][f"int4_batch{b}"] = {"tokens_per_s": b * 1e3 / ms, "ms_per_step": ms, "launches_per_step": dec.launches_per_step(),
-                                                 "frac_of_hbm_peak": by / (ms * 1e-3) / 1e9 / peak}
-            ms = prompt_ms(lambda: dec.prefill_tokens(ids, 0))
-            r["prompt"]["int4_32_rows"] = {"tokens": ctx, "ms": ms, "tokens_per_s": ctx * 1e3 / ms,
-                                           "frac_of_bf16_peak": ctx * (2.0 * (body + head) + attn_flops) / (ms * 1e-3) / 1e12 / tflops}
-            dec.close()
-            del model
+            layered(args.design, z, ids, r)
+            if args.design == "dabevik":
+                int4(z, ids, r)
+            else:
+                layered("dabevik", z, ids, r)
             torch.cuda.empty_cache()
             out.append(r)
     _RESULT_LINE.append(json.dumps({"metric": "design_tokens_per_s", "design": args.design, "steps": K, "warmup": W, "data": "synthetic",
@@ -889,8 +945,8 @@ def main():
     ap.add_argument("--impl", default="b200", choices=["b200", "reference"])
     ap.add_argument("--model", default="llama8b", choices=["llama8b", "qwen05b", "llama70b"],
                     help="qwen05b: workload configuration 3; llama70b: configuration 5 (8 GPUs, --batch 16); both with --quick")
-    ap.add_argument("--design", default=None, choices=["dabevik"],
-                    help="instead of the headline workload: decode and prompt throughput of a layered design beside the INT4 decoder of equal size")
+    ap.add_argument("--design", default=None, choices=sorted(DESIGNS),
+                    help="instead of the headline workload: decode and prompt throughput of a layered design beside the closest other model of equal size")
     ap.add_argument("--repeats", type=int, default=5, help="timed regions of --steps steps each; the median is reported")
     ap.add_argument("--no-batch-sweep", dest="batch_sweep", action="store_false", help="skip the batch 2 / 4 / 8 / 32 measurements")
     ap.add_argument("--no-config3", dest="config3", action="store_false", help="skip the Qwen2.5-0.5B-shaped measurement")

@@ -28,6 +28,10 @@ MODELS = {
     "wide": o.make_config(vocab=700, width=264, layers=[
         o.latent_layer(12, 64, 32, 64, 384, 200, scale=0.12, base=10000.0, ff=520), o.attention_layer(16, 4, 128, 96, 100, scale=0.15, cap=20.0, ff=136),
         o.attention_layer(8, 4, 160, 96, 70, scale=0.15, ff=None)]),
+    # sizes that the tcgen05 kernel of portions takes, with the cap's small arguments and without
+    "even": o.make_config(vocab=130, width=128, layers=[
+        o.attention_layer(8, 2, 64, 64, 200, scale=0.1, cap=30.0, ff=256), o.latent_layer(6, 32, 16, 40, 136, 72, ff=None),
+        o.attention_layer(6, 2, 48, 64, 77, scale=0.5, cap=5.0, ff=96), o.latent_layer(4, 128, 64, 128, 512, 96, scale=0.07, ff=80)]),
     # a latent beyond the tensor-core kernel's tiles
     "large": o.make_config(vocab=60, width=64, layers=[o.latent_layer(3, 12, 20, 16, 720, 48, ff=48)]),
 }
@@ -94,7 +98,7 @@ def test_prompt_portions_and_decoding(models, name, dtype):
 @pytest.mark.parametrize("dtype", DTYPES)
 def test_whole_prompt_in_one_step(models, dtype):
     """Portions of several hundred rows, and a long cache behind short ones."""
-    for name in ("mixed", "wide"):
+    for name in ("mixed", "wide", "even"):
         path, cfg, w = models[name]
         toks = tokens_for(cfg, 430, 7)
         want = o.forward(cfg, w, toks)
@@ -106,6 +110,22 @@ def test_whole_prompt_in_one_step(models, dtype):
         dec.reset_sequence(0)
         dec.extend(toks[:420], 0)
         assert err(np.stack([dec.step(toks[p], p) for p in range(420, 430)]), want[420:]) < TOL[dtype]
+
+
+def test_long_prompts_wrap_every_ring(models):
+    """Portions of 64 positions and of odd sizes in front of rings that hold a chunk and 128 positions."""
+    path, cfg, w = models["even"]
+    toks = tokens_for(cfg, 1000, 17)
+    want = o.forward(cfg, w, toks)
+    dec = load(path, "bfloat16", prefill_rows=64, max_seq_len=1024)
+    for cuts in ([1000], [100, 63, 65, 200, 129, 333, 110], [17, 400, 31, 552]):
+        dec.reset_sequence(0)
+        rows, at = [], 0
+        for c in cuts:
+            rows.append(dec.extend(toks[at:at + c], at, list(range(c))))
+            at += c
+        assert err(np.concatenate(rows), want) < TOL["bfloat16"], cuts
+    assert fault() == 0
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -342,19 +362,19 @@ def test_going_back(models):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("size,keep", [(7, 3), (1, 2), (33, 0), (64, 8), (500, 4)])
-def test_flash_attention_with_windows_and_kept_positions(size, keep, dtype):
+@pytest.mark.parametrize("size,keep,vdim", [(7, 3, 20), (1, 2, 20), (33, 0, 20), (64, 8, 24), (500, 4, 20), (33, 0, 24), (150, 0, 40), (500, 0, 24)])
+def test_flash_attention_with_windows_and_kept_positions(size, keep, vdim, dtype):
     """Layers whose heads are not mixed run on the same kernels with a window and kept first positions."""
     import torchburn_b200 as tb
 
-    cfg = dab.make_config(vocab=90, width=72, taps=3, layers=[dab.make_layer(6, 2, 24, 20, size=size, keep_first=keep, ff=88)])
+    cfg = dab.make_config(vocab=90, width=72, taps=3, layers=[dab.make_layer(6, 2, 24, vdim, size=size, keep_first=keep, ff=88)])
     w = dab.make_weights(cfg, 9)
     w["l0.mix.talk"] = np.eye(6)
     raw = {n: (np.ascontiguousarray(a, np.float32).view(np.uint32) >> 16).astype(np.uint16) for n, a in w.items()}
     names = {"norm1": "norm1", "norm1_after": "norm1b", "conv1": "canon1", "q_w": "mix.q", "q_b": "mix.q.b", "k_w": "mix.k", "k_b": "mix.k.b",
              "v_w": "mix.v", "v_b": "mix.v.b", "q_norm": "mix.q.norm", "k_norm": "mix.k.norm", "o_w": "mix.o", "o_b": "mix.o.b", "norm2": "norm2",
              "norm2_after": "norm2b", "conv2": "canon2", "up_w": "mlp.up", "down_w": "mlp.down", "act": "mlp.act"}
-    spec = tb.LayerSpec(6, 2, 24, 20, 0.21, size, keep, 88, None, {k: raw["l0." + v] for k, v in names.items()})
+    spec = tb.LayerSpec(6, 2, 24, vdim, 0.21, size, keep, 88, None, {k: raw["l0." + v] for k, v in names.items()})
     dec = tb.LayeredDecoder([spec], raw["embed"], raw["final.norm"], raw["pos"], hidden_size=72, vocab_size=90, norm_eps=1e-5, max_seq_len=400,
                             embed_scale=3.0, conv_taps=3, dtype=dtype, prefill_rows=48)
     toks = tokens_for(cfg, 300, 5)

@@ -550,6 +550,7 @@ tb_status run_positions_layered(tb_decoder* d, int seq, const int64_t* tokens, i
       LayeredStep s;
       s.r.tokens = d->d_tokens; s.r.slots = d->d_slots; s.r.offsets = d->d_offsets; s.r.rows = m;
       s.one_sequence = true;
+      s.start = start_offset + i;
       s.row_map = d->d_row_map; s.logit_rows = lr; s.logits = d->logits; s.pdl = d->pdl; s.snapshots = debug;
       d->debug_rows = m;
       int launches = 0;

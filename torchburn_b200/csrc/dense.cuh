@@ -242,13 +242,26 @@ tb_status launch_latent_prep(Precision p, const LatentPrepArgs& a, cudaStream_t 
 struct LatentQueryArgs {
   StepRows r;
   PartialSums y;                         // [heads][dim | rot_dim]
-  int heads = 0, dim = 0, rot_dim = 0, rot_dims = 0, kv_rank = 0, dpad = 0;
+  int heads = 0, dim = 0, rot_dim = 0, rot_dims = 0, dpad = 0;
+  int rot_at = 0;                        // where the rotated part begins in a head's query
   const float2* table = nullptr;
-  ActOperand out;                        // one operand of K = dim per head, one after the other
+  ActOperand out;                        // one operand of K = dim per head, one after the other; data null: the
+                                         // unrotated part goes to the beginning of the head's query
   void* q = nullptr;                     // [rows, heads * dpad] of the activation type
   bool pdl = false;
 };
 tb_status launch_latent_query(Precision p, const LatentQueryArgs& a, cudaStream_t st);
+// The bf16 latents of positions [lo, lo + n) of the step's first row's sequence as the operand of a product.
+struct LatentRowsArgs {
+  StepRows r;
+  const void* cache = nullptr;           // [slots][cache rows][dpad]
+  CacheGeom geom;
+  int kv_rank = 0, dpad = 0;             // multiples of 8
+  int lo = 0, n = 0;
+  ActOperand out;
+  bool pdl = false;
+};
+tb_status launch_latent_rows(const LatentRowsArgs& a, cudaStream_t st);
 // cos and sin of position * base^(-2i / dims).
 tb_status fill_rotation_table(float2* table, int64_t positions, int dims, double base);
 
@@ -282,6 +295,13 @@ struct FlashArgs {
   int window = 0;                        // position i sees j when i - j < window and i / chunk = j / chunk (chunk > 0),
   int keep_first = 0;                    // or j < keep_first
   int chunk = 0;
+  bool unit_norm = false;                // queries and keys have a root mean square of one
+  // Keys and values written out by position instead of the caches (portions of one sequence): position p of head g
+  // is row p - key_base, its first key_cols key columns at key_rows + g key_cols, its values at value_rows + g vdim;
+  // the other key columns, the same for every head, are columns from rest_col on of k_cache's rows of cache_row.
+  const void* key_rows = nullptr;
+  const void* value_rows = nullptr;
+  int key_cols = 0, key_base = 0, row_stride = 0, rest_col = 0, cache_row = 0;
   const float* gate = nullptr;           // [rows, heads] factors of the heads' outputs, or null
   int64_t max_visible = 0;               // most positions one row can see
   float* parts = nullptr;                // scratch [part_slots][vdim]
@@ -294,6 +314,8 @@ struct FlashArgs {
 };
 int64_t flash_part_slots(int64_t rows, int64_t heads);   // what the splits a step can use need
 tb_status launch_flash_attention(Precision p, const FlashArgs& a, cudaStream_t st, int* launches);
+bool flash_tc5_fits(int dpad, int vdim);                 // sizes that the tcgen05 kernel for portions takes
+int flash_fault_flag();
 
 // ---- windowed attention with mixed heads (window_attention.cu) -----------------------------------
 struct WindowAttnArgs {

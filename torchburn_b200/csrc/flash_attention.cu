@@ -10,8 +10,10 @@
 // memory as two bf16 pieces (the second one what the rounding of the first left: 16 mantissa bits), then the values
 // with the warps side by side over the value columns.  CTAs that share a block's keys leave (max, sum, unnormalised
 // output) and a last kernel merges them in a fixed order.
+// Portions of one sequence take the tcgen05 kernel of flash_tc5.cu where its tiles fit.
 // fp32, and sizes beyond the tiles (flash_simple_kernel): a CTA per row and up to four heads, fp32 products.
 #include "dense.cuh"
+#include "flash_attention.cuh"
 #include "window_attention.cuh"
 
 namespace tb {
@@ -21,13 +23,6 @@ namespace {
 constexpr int kThreads = 256;
 constexpr float kLog2E = 1.44269504f;
 constexpr int kMaxSplits = 512;
-
-struct FlashShape {
-  int run_rows;   // rows that share a sequence: the whole step, or one
-  int tiles;      // CTAs' shares of a run's (query, head) pairs
-  int splits;     // CTAs that share a tile's keys
-  int pair_tile;  // kernel's pairs per tile
-};
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void cp16z(void* dst, const void* src, bool live) {   // zeros when not live
@@ -49,11 +44,6 @@ __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], 
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
 
-// Elements behind a head's output that the next product's padded K covers: column c of head h for c in [vdim, limit).
-__host__ __device__ __forceinline__ int column_limit(const FlashArgs& a, int h) {
-  if (a.out_per_head) return a.out.kp;
-  return h == a.heads - 1 ? a.out.kp - h * a.vdim : a.vdim;
-}
 template <bool BF16>
 __device__ __forceinline__ void store_column(const FlashArgs& a, int row, int h, int c, float v) {
   if (!a.out_per_head) {
@@ -306,7 +296,7 @@ __global__ void __launch_bounds__(kThreads, NV <= 8 ? 2 : 1) flash_mma_kernel(co
       }
     }
     if (whole && wc == 0)
-      for (int c = a.vdim + (lane & 3); c < column_limit(a, head[e]); c += 4) store_column<true>(a, qrow[e], head[e], c, 0.f);
+      for (int c = a.vdim + (lane & 3); c < flash_column_limit(a, head[e]); c += 4) store_column<true>(a, qrow[e], head[e], c, 0.f);
   }
 }
 
@@ -336,7 +326,7 @@ __global__ void __launch_bounds__(128) flash_merge_kernel(const FlashArgs a, con
   if ((tid & 31) == 0) s_sum[tid >> 5] = l;
   __syncthreads();
   l = (s_sum[0] + s_sum[1]) + (s_sum[2] + s_sum[3]);
-  if (c >= column_limit(a, h)) return;
+  if (c >= flash_column_limit(a, h)) return;
   float v = 0.f;
   if (c < a.vdim) {
     const float* p = a.parts + at * a.vdim + c;
@@ -446,7 +436,7 @@ __global__ void __launch_bounds__(kThreads) flash_simple_kernel(const FlashArgs 
   for (int h = 0; h < nh; ++h) {
     float f = s_l[h] > 0.f ? 1.f / s_l[h] : 0.f;
     if (a.gate) f *= a.gate[(size_t)r * a.heads + h0 + h];
-    for (int c = tid; c < column_limit(a, h0 + h); c += kThreads)
+    for (int c = tid; c < flash_column_limit(a, h0 + h); c += kThreads)
       store_column<sizeof(T) == 2>(a, r, h0 + h, c, c < a.vdim ? s_o[h * a.vdim + c] * f : 0.f);
   }
 }
@@ -486,6 +476,19 @@ tb_status launch_flash_attention(Precision p, const FlashArgs& a, cudaStream_t s
     return fail(TB_ERR_SHAPE, "flash attention: bad shape");
   if (p == Precision::kF32) return launch_simple<float>(a, st, launches);
   const int gq = a.heads / a.kv_heads, rows = a.r.rows;
+  auto merge = [&](int splits) -> tb_status {
+    ++*launches;
+    if (splits == 1) return TB_OK;
+    ++*launches;
+    const int cols = a.out_per_head ? a.out.kp : a.out.kp - (a.heads - 1) * a.vdim;
+    return launch_kernel(flash_merge_kernel, dim3((unsigned)a.heads, (unsigned)rows, (unsigned)((cols + 127) / 128)), dim3(128), 0, st, a.pdl, 1, a, splits);
+  };
+  if (flash_tc5_supported(a)) {
+    int splits = 1;
+    TB_TRY(launch_flash_tc5(a, st, &splits));
+    return merge(splits);
+  }
+  if (a.key_rows) return fail(TB_ERR_SHAPE, "flash attention: keys in two pieces of %d and %d columns", a.key_cols, a.dim - a.key_cols);
   FlashShape sh;
   sh.run_rows = a.one_sequence ? rows : 1;
   const int runs = a.one_sequence ? 1 : rows;
@@ -506,23 +509,19 @@ tb_status launch_flash_attention(Precision p, const FlashArgs& a, cudaStream_t s
     if (kern) break;
   }
   if (kern == nullptr) return launch_simple<__nv_bfloat16>(a, st, launches);
-  sh.pair_tile = 16 * mg;
-  sh.tiles = (int)((pairs + sh.pair_tile - 1) / sh.pair_tile);
+  const int pair_tile = 16 * mg;
+  sh.tiles = (int)((pairs + pair_tile - 1) / pair_tile);
   const size_t smem = mma_bytes(a, mg, kt);
   const int64_t ctas = (int64_t)sh.tiles * a.kv_heads * runs, slots = (int64_t)sm_count() * (smem <= 112 * 1024 ? 2 : 1);
   int64_t splits = slots / ctas;
-  const int64_t ktiles = (a.max_visible + (a.one_sequence ? sh.pair_tile / gq : 0) + kt - 1) / kt;
+  const int64_t ktiles = (a.max_visible + (a.one_sequence ? pair_tile / gq : 0) + kt - 1) / kt;
   if (splits > ktiles) splits = ktiles;
   if (splits > kMaxSplits) splits = kMaxSplits;
   if (splits > a.part_slots / ((int64_t)rows * a.heads)) splits = a.part_slots / ((int64_t)rows * a.heads);
   if (splits < 1) splits = 1;
   sh.splits = (int)splits;
   TB_TRY(launch_kernel(kern, dim3((unsigned)(sh.tiles * sh.splits), (unsigned)a.kv_heads, (unsigned)runs), dim3(kThreads), smem, st, a.pdl, 1, a, sh));
-  ++*launches;
-  if (sh.splits == 1) return TB_OK;
-  ++*launches;
-  const int cols = a.out_per_head ? a.out.kp : a.out.kp - (a.heads - 1) * a.vdim;
-  return launch_kernel(flash_merge_kernel, dim3((unsigned)a.heads, (unsigned)rows, (unsigned)((cols + 127) / 128)), dim3(128), 0, st, a.pdl, 1, a, sh.splits);
+  return merge(sh.splits);
 }
 
 int64_t flash_part_slots(int64_t rows, int64_t heads) {

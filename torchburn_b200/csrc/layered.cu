@@ -9,6 +9,7 @@
 //   glue -> QKV (+ gate) product -> per-head norm, value mixing, cache append -> flash attention (-> merge) -> ...
 //   glue -> latent product -> latent norms, rotation, cache append -> query product -> rotation -> key product per
 //   head -> flash attention over the latents (-> merge) -> value product per head -> ...
+//   (long portions: the latents of the sequence -> all heads' keys and values -> flash attention -> ...)
 // and the final norm with the output product for the rows whose logits are wanted.  Every buffer between
 // two kernels is written by exactly one of them and read by the next, so one buffer of partial sums and one
 // operand buffer per kind serve the whole stack; the residual stream alternates between two buffers because
@@ -23,6 +24,7 @@
 #include <vector>
 
 #include "layered.cuh"
+#include "window_attention.cuh"
 
 namespace tb {
 
@@ -32,6 +34,8 @@ constexpr int kHistory = 128;      // positions a sequence can always be taken b
 constexpr int kMaxSplits = 8;
 constexpr size_t kScoreBudget = 1024u << 20;
 constexpr int kManyRows = 64;       // from here on the glue with a convolution is two kernels
+constexpr int kExpandRows = 64;     // portions from here on write out the keys and values of latents
+constexpr size_t kExpandBudget = (size_t)4096 << 20;
 constexpr double kLaunchStages = 16.0;  // stages of a product's K loop that a kernel of its own costs
 
 struct LayerWeights {
@@ -47,6 +51,8 @@ struct LayerWeights {
   float vmix = 0.f;
   int q_rank = 0, kv_rank = 0, rot_dim = 0;
   DenseWeight uq, uk, uv;            // uk: per head [kv_rank, dim], uv: per head [vdim, kv_rank]
+  DenseWeight ukv;                   // [all heads' keys | all heads' values, kv_rank], where portions write them out
+  int xpad = 0;                      // padded size of a written-out key
   float *dq_norm = nullptr, *dkv_norm = nullptr;
   float *qkv_b = nullptr, *q_norm = nullptr, *k_norm = nullptr, *talk = nullptr, *o_b = nullptr;
   float *norm1 = nullptr, *norm1b = nullptr, *norm2 = nullptr, *norm2b = nullptr;
@@ -102,6 +108,8 @@ struct LayeredModel {
   int64_t y_floats = 0;
   void *act_x = nullptr, *act_o = nullptr, *act_z = nullptr;
   void *act_c = nullptr, *act_q = nullptr, *act_v = nullptr;   // latent layers: query latent; per head the plain query, the attended latent
+  void* act_l = nullptr;           // latents of a sequence as an operand, and what they are written out to: [positions][keys | values]
+  __nv_bfloat16* expanded = nullptr;
   float *v_first = nullptr, *gates = nullptr;
   float2* part_ml = nullptr;       // splits of the flash attention, with flash_parts
   float* flash_parts = nullptr;
@@ -221,6 +229,14 @@ tb_status load_latent(LayeredModel* m, LayerWeights& w, const tb_layered_layer& 
   TB_TRY(dense_weight_fill(&w.uk, 0, s.uk_w, w.kv_rank, w.dim, space, true));
   TB_TRY(dense_matrix(m, &w.uv, w.vdim, w.kv_rank, w.heads));
   TB_TRY(dense_weight_fill(&w.uv, 0, s.uv_w, w.vdim, w.kv_rank, space));
+  w.xpad = (int)pad_to(w.dim + w.rot_dim, 16);
+  const int64_t row = (int64_t)w.heads * (w.dim + w.vdim);
+  if (m->prec == Precision::kBf16 && flash_tc5_fits(w.xpad, w.vdim) && w.dim % 8 == 0 && w.rot_dim % 8 == 0 && w.kv_rank % 8 == 0 &&
+      (size_t)(m->cfg.max_seq_len * row) * 2 <= kExpandBudget) {
+    TB_TRY(dense_matrix(m, &w.ukv, row, w.kv_rank));
+    TB_TRY(dense_weight_fill(&w.ukv, 0, s.uk_w, (int64_t)w.heads * w.dim, w.kv_rank, space));
+    TB_TRY(dense_weight_fill(&w.ukv, (int64_t)w.heads * w.dim, s.uv_w, (int64_t)w.heads * w.vdim, w.kv_rank, space));
+  }
   TB_TRY(dev_vector(m, &w.dq_norm, s.dq_norm, w.q_rank, w.q_rank, space, "dq_norm"));
   TB_TRY(dev_vector(m, &w.dkv_norm, s.dkv_norm, w.kv_rank, w.kv_rank, space, "dkv_norm"));
   return TB_OK;
@@ -285,7 +301,7 @@ tb_status create_impl(LayeredModel* m, const tb_layered_layer* layers, const Lay
   m->w.resize((size_t)m->L);
   m->runs.resize((size_t)m->L);
   int64_t max_cols = m->embed.rows > 0 ? pad_to(m->width, 128) : 0, max_q = 0, max_o = 0, max_z = 0, max_score_row = 0, max_heads = 1;
-  int64_t max_c = 0, max_qn = 0, max_ctx = 0, max_gates = 0, flash_vdim = 0;
+  int64_t max_c = 0, max_qn = 0, max_ctx = 0, max_gates = 0, flash_vdim = 0, max_lat = 0, max_expanded = 0;
   const LayerRun* first_values = nullptr;
   m->rollback = m->ring - 2 * (m->taps - 1);
   for (int i = 0; i < m->L; ++i)
@@ -364,8 +380,12 @@ tb_status create_impl(LayeredModel* m, const tb_layered_layer* layers, const Lay
     most(max_qn, w.heads * w.uk.kp);
     most(max_ctx, w.heads * w.uv.kp);
     if (w.gate) most(max_gates, w.heads);
-    if (!w.talk) most(flash_vdim, w.latent ? w.kv_rank : w.vdim);
-    const int64_t q = (int64_t)w.heads * w.dpad;
+    if (!w.talk) most(flash_vdim, w.latent && w.kv_rank > w.vdim ? w.kv_rank : w.vdim);
+    if (w.ukv.img) {
+      most(max_lat, w.ukv.kp);
+      most(max_expanded, (int64_t)w.heads * (w.dim + w.vdim));
+    }
+    const int64_t q = (int64_t)w.heads * (w.dpad > w.xpad ? w.dpad : w.xpad);
     if (q > max_q) max_q = q;
     if (w.o.kp > max_o) max_o = w.o.kp;
     if (w.down.kp > max_z) max_z = w.down.kp;
@@ -393,6 +413,11 @@ tb_status create_impl(LayeredModel* m, const tb_layered_layer* layers, const Lay
   m->act_q = b;
   TB_TRY(dev_alloc(m, &b, rp * max_ctx * esz, true));
   m->act_v = b;
+  if (max_lat > 0) {
+    TB_TRY(dev_alloc(m, &b, (size_t)(dense_row_pad((int)S) * max_lat * 2), true));
+    m->act_l = b;
+    TB_TRY(dev_alloc(m, &m->expanded, (size_t)(S * max_expanded), true));
+  }
   if (first_values) {
     const LayerWeights& f = m->w[(size_t)first_values->weights];
     TB_TRY(dev_alloc(m, &m->v_first, (size_t)R * f.kv_heads * f.vdim, true));
@@ -488,14 +513,17 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
   int n = 0, cur = 0;
   const ActOperand ax{m->act_x, mp, m->xs};
 
+  // partial sums that the shared buffer holds of a product
+  auto split_room = [&](const DenseWeight& w) -> int {
+    const int64_t cap = m->y_floats / ((int64_t)rows * w.rows);
+    return cap < kMaxSplits ? (int)cap : kMaxSplits;
+  };
   // one product: partial sums into the shared buffer
   auto product = [&](const DenseWeight& w, const ActOperand& x, PartialSums* y) -> tb_status {
     const int64_t per = (int64_t)rows * w.rows;
-    int64_t cap = m->y_floats / per;
-    if (cap > kMaxSplits) cap = kMaxSplits;
     DenseGemmArgs a;
     a.w = &w; a.x = x; a.rows = rows; a.out = m->y; a.ldo = w.rows; a.n_valid = w.rows;
-    a.splits = dense_splits(prec, w.rows, w.kp, rows, (int)cap);
+    a.splits = dense_splits(prec, w.rows, w.kp, rows, split_room(w));
     a.split_stride = (size_t)per;
     a.pdl = s.pdl;
     y->y = m->y; y->splits = a.splits; y->split_stride = a.split_stride; y->ldy = a.ldo;
@@ -565,6 +593,7 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
     FlashArgs fa;
     fa.heads = w.heads; fa.kv_heads = w.kv_heads; fa.dim = w.dim; fa.vdim = w.vdim; fa.dpad = w.dpad; fa.vpad = w.vpad;
     fa.gate = w.gate ? m->gates : nullptr;
+    fa.unit_norm = run.unit_norm;
     fa.out = out;
     if (run.unit_norm || run.value_mix || w.gate) {
       HeadsPrepArgs ha;
@@ -609,10 +638,34 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
     TB_TRY(launch_latent_prep(prec, la, st));
     TB_TRY(product(w.uq, la.out, &y));
     LatentQueryArgs lq;
-    lq.r = r; lq.y = y; lq.heads = w.heads; lq.dim = w.dim; lq.rot_dim = w.rot_dim; lq.rot_dims = run.rot_dims; lq.kv_rank = w.kv_rank;
-    lq.dpad = w.dpad; lq.table = run.rotation; lq.pdl = s.pdl;
-    lq.out = ActOperand{m->act_q, mp, (int)w.uk.kp};
+    lq.r = r; lq.y = y; lq.heads = w.heads; lq.dim = w.dim; lq.rot_dim = w.rot_dim; lq.rot_dims = run.rot_dims;
+    lq.table = run.rotation; lq.pdl = s.pdl;
     lq.q = prec == Precision::kBf16 ? static_cast<void*>(m->q16) : m->q;
+    if (w.ukv.img && s.one_sequence && s.start >= 0 && rows >= kExpandRows && run.keep_first == 0) {
+      // a portion: fewer operations with the keys and values of what it sees written out for this layer
+      lq.dpad = w.xpad; lq.rot_at = w.dim;
+      TB_TRY(launch_latent_query(prec, lq, st));
+      LatentRowsArgs lr;
+      lr.r = r; lr.cache = run.k_cache; lr.geom = run.geom; lr.kv_rank = w.kv_rank; lr.dpad = w.dpad; lr.pdl = s.pdl;
+      lr.lo = VisibleRange((int)s.start, run.window, 0, run.chunk).lo;
+      lr.n = (int)s.start + rows - lr.lo;
+      lr.out = ActOperand{m->act_l, dense_row_pad(lr.n), (int)w.ukv.kp};
+      TB_TRY(launch_latent_rows(lr, st));
+      const int64_t row = (int64_t)w.heads * (w.dim + w.vdim);
+      DenseGemmArgs xa;
+      xa.w = &w.ukv; xa.x = lr.out; xa.rows = lr.n; xa.n_valid = row; xa.pdl = s.pdl;
+      xa.sink = DenseSink::kRows; xa.out = m->expanded; xa.ldo = row;
+      TB_TRY(launch_dense_gemm(prec, xa, st));
+      n += 4;
+      FlashArgs fa;
+      fa.heads = fa.kv_heads = w.heads; fa.dim = w.dim + w.rot_dim; fa.vdim = w.vdim; fa.dpad = w.xpad; fa.vpad = (int)pad_to(w.vdim, 16);
+      fa.key_rows = m->expanded; fa.value_rows = m->expanded + (int64_t)w.heads * w.dim;
+      fa.key_cols = w.dim; fa.key_base = lr.lo; fa.row_stride = (int)row; fa.rest_col = w.kv_rank; fa.cache_row = w.dpad;
+      fa.out = out;
+      return flash(fa, run);
+    }
+    lq.dpad = w.dpad; lq.rot_at = w.kv_rank;
+    lq.out = ActOperand{m->act_q, mp, (int)w.uk.kp};
     TB_TRY(launch_latent_query(prec, lq, st));
     n += 2;
     DenseGemmArgs ka;
@@ -632,7 +685,7 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
     PartialSums y;
     if (run.mlp == TB_MLP_RELU2) {
       double gain = 0.0;
-      dense_splits(prec, w.up.rows, w.up.kp, rows, kMaxSplits, &gain);
+      dense_splits(prec, w.up.rows, w.up.kp, rows, split_room(w.up), &gain);
       if (gain < kLaunchStages) {   // the activation in the product's epilogue
         DenseGemmArgs a;
         a.w = &w.up; a.x = ax; a.rows = rows; a.n_valid = out.kp; a.pdl = s.pdl;

@@ -12,6 +12,7 @@ struct LayeredModel;
 struct LayeredStep {
   StepRows r;                      // tokens / slots / offsets on the device
   bool one_sequence = false;       // the rows are consecutive positions of one sequence
+  int64_t start = -1;              // then the first row's position, where the host knows it
   const int32_t* row_map = nullptr;  // row -> logits row or -1; null: every row in place
   int logit_rows = 0;
   float* logits = nullptr;         // [logit_rows, vocab]

@@ -528,14 +528,30 @@ __global__ void __launch_bounds__(kThreads) latent_query_kernel(const LatentQuer
   grid_dep_wait();
   if (h >= a.heads) return;
   const int pos = a.r.pos[r], col = h * (a.dim + a.rot_dim);
-  ActOperand out = a.out;
-  out.data = static_cast<unsigned char*>(out.data) + (size_t)h * out.mp * out.kp * sizeof(T);
-  for (int c = lane; c < out.kp; c += 32) act_store1<sizeof(T) == 2>(out, r, c, c < a.dim ? sum_column(a.y, r, col + c) : 0.f);
-  T* q = static_cast<T*>(a.q) + ((size_t)r * a.heads + h) * a.dpad + a.kv_rank;
+  T* q = static_cast<T*>(a.q) + ((size_t)r * a.heads + h) * a.dpad;
+  if (a.out.data) {
+    ActOperand out = a.out;
+    out.data = static_cast<unsigned char*>(out.data) + (size_t)h * out.mp * out.kp * sizeof(T);
+    for (int c = lane; c < out.kp; c += 32) act_store1<sizeof(T) == 2>(out, r, c, c < a.dim ? sum_column(a.y, r, col + c) : 0.f);
+  } else {
+    for (int c = lane; c < a.dim; c += 32) q[c] = (T)sum_column(a.y, r, col + c);
+  }
+  q += a.rot_at;
   for (int c = lane; c < a.rot_dim; c += 32) {
     const float own = sum_column(a.y, r, col + a.dim + c), other = c < a.rot_dims ? sum_column(a.y, r, col + a.dim + (c ^ 1)) : 0.f;
     q[c] = (T)rotated(a.table, a.rot_dims, pos, c, own, other);
   }
+}
+
+// grid (positions, pieces / 256)
+__global__ void __launch_bounds__(kThreads) latent_rows_kernel(const LatentRowsArgs a) {
+  const int c = (int)blockIdx.y * kThreads + threadIdx.x, i = (int)blockIdx.x;
+  grid_dep_launch();
+  grid_dep_wait();
+  if (c >= a.out.kp >> 3) return;
+  const __nv_bfloat16* row = static_cast<const __nv_bfloat16*>(a.cache) + ((size_t)a.r.slots[0] * a.geom.rows + a.geom.row_of(a.lo + i)) * (size_t)a.dpad;
+  const uint4 v = c * 8 < a.kv_rank ? *reinterpret_cast<const uint4*>(row + c * 8) : make_uint4(0u, 0u, 0u, 0u);
+  *reinterpret_cast<uint4*>(static_cast<unsigned char*>(a.out.data) + image_offset(a.out.mp, i, c * 8)) = v;
 }
 
 // grid (columns / 1024, rows)
@@ -674,6 +690,11 @@ tb_status launch_latent_query(Precision p, const LatentQueryArgs& a, cudaStream_
   const dim3 grid((unsigned)((a.heads + kThreads / 32 - 1) / (kThreads / 32)), (unsigned)a.r.rows);
   return p == Precision::kBf16 ? launch_kernel(latent_query_kernel<__nv_bfloat16>, grid, dim3(kThreads), 0, st, a.pdl, 1, a)
                                : launch_kernel(latent_query_kernel<float>, grid, dim3(kThreads), 0, st, a.pdl, 1, a);
+}
+
+tb_status launch_latent_rows(const LatentRowsArgs& a, cudaStream_t st) {
+  const int pieces = a.out.kp >> 3, threads = pieces < kThreads ? (pieces + 31) / 32 * 32 : kThreads;
+  return launch_kernel(latent_rows_kernel, dim3((unsigned)a.n, (unsigned)((pieces + kThreads - 1) / kThreads)), dim3((unsigned)threads), 0, st, a.pdl, 1, a);
 }
 
 tb_status launch_relu2(Precision p, int rows, const PartialSums& z, const ActOperand& out, bool pdl, cudaStream_t st) {

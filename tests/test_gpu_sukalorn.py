@@ -346,13 +346,13 @@ def test_long_decoding_wraps_every_ring(models, dtype):
 
 def test_going_back(models):
     path, cfg, w = models["mixed"]
-    dec = load(path, "float32", prefill_rows=32, max_seq_len=400)
-    toks = tokens_for(cfg, 300, 12)
+    dec = load(path, "float32", prefill_rows=32, max_seq_len=600)
+    toks = tokens_for(cfg, 500, 12)
     dec.extend(toks, 0)
-    other = toks[:220] + tokens_for(cfg, 30, 13)         # an earlier continuation point, other tokens
-    assert err(dec.extend(other[220:], 220, list(range(30))), o.forward(cfg, w, other)[220:]) < TOL["float32"]
+    other = toks[:420] + tokens_for(cfg, 30, 13)         # an earlier continuation point, other tokens
+    assert err(dec.extend(other[420:], 420, list(range(30))), o.forward(cfg, w, other)[420:]) < TOL["float32"]
     with pytest.raises(ValueError, match="cannot go on"):
-        dec.step(3, 260)
+        dec.step(3, 460)
     with pytest.raises(ValueError, match="cannot go back"):
         dec.step(3, 100)
     assert err(dec.extend(toks[:5], 0, [4]), o.forward(cfg, w, toks[:5])[[4]]) < TOL["float32"]

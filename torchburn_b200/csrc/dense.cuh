@@ -288,6 +288,7 @@ struct FlashArgs {
   const void* v_cache = nullptr;
   bool values_in_keys = false;           // one key/value head whose values are the first vdim elements of its keys
   CacheGeom geom;
+  int cache_slots = 0;                   // sequences that the caches hold
   int heads = 0, kv_heads = 0, dim = 0, vdim = 0, dpad = 0, vpad = 0;
   float scale = 1.f;
   float softcap = 0.f;                   // 0: none
@@ -297,11 +298,11 @@ struct FlashArgs {
   int chunk = 0;
   bool unit_norm = false;                // queries and keys have a root mean square of one
   // Keys and values written out by position instead of the caches (portions of one sequence): position p of head g
-  // is row p - key_base, its first key_cols key columns at key_rows + g key_cols, its values at value_rows + g vdim;
+  // is row p - key_base of key_count, its first key_cols key columns at key_rows + g key_cols, its values at value_rows + g vdim;
   // the other key columns, the same for every head, are columns from rest_col on of k_cache's rows of cache_row.
   const void* key_rows = nullptr;
   const void* value_rows = nullptr;
-  int key_cols = 0, key_base = 0, row_stride = 0, rest_col = 0, cache_row = 0;
+  int key_cols = 0, key_base = 0, key_count = 0, row_stride = 0, rest_col = 0, cache_row = 0;
   const float* gate = nullptr;           // [rows, heads] factors of the heads' outputs, or null
   int64_t max_visible = 0;               // most positions one row can see
   float* parts = nullptr;                // scratch [part_slots][vdim]

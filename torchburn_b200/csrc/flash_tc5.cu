@@ -9,11 +9,16 @@
 //                            one what the rounding of the first left)
 //   O += P V                 P from tensor memory, V as it lies in the cache ([key][column]: MN-major)
 //
-// While one warpgroup is at its softmax the tensor core works for the other.  Three warps bring keys and values by
-// cp.async (rows of a cache are gathered: rings, several heads side by side), one thread issues the MMAs.  The output
-// is rescaled only when the maximum has grown by more than 8 powers of two; weights stay exact relative to the sum.
-// Keys may come in two pieces: columns from one matrix, the rest (a rotated part that heads share) from another.
+// While one warpgroup is at its softmax the tensor core works for the other.  Keys and values come by TMA, panels of 64
+// columns by 128 positions, swizzled on the way; tiles begin at multiples of 128 positions, so that one lies in one
+// piece in a ring of a multiple of 128 rows too.  Other rings, and keys in pieces of other than 64 columns, come by
+// cp.async from three warps.  One thread issues the MMAs.  The output is rescaled only when the maximum has grown by
+// more than 8 powers of two; weights stay exact relative to the sum.  Keys may come in two pieces: columns from one
+// matrix, the rest (a rotated part that heads share) from another.
 #include <climits>
+#include <cstring>
+
+#include <cuda.h>
 
 #include "dense.cuh"
 #include "flash_attention.cuh"
@@ -79,6 +84,16 @@ __device__ __forceinline__ void mma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, ui
       : "memory");
 }
 
+// A panel of 64 columns x 128 rows of a row-major matrix, from (x, y) on; x on a 16-byte boundary.
+__device__ __forceinline__ void tma_panel(uint32_t dst, const CUtensorMap* map, int x, int y, uint64_t* bar) {
+  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst), "l"(map), "r"(x),
+               "r"(y), "r"(smem_u32(bar))
+               : "memory");
+}
+struct FlashMaps {
+  CUtensorMap k, rest, v;
+};
+
 // Rows of keys or values: key v of the block is row base + v, less `ring` from `end` on.
 struct Rows {
   const __nv_bfloat16* p;
@@ -131,10 +146,10 @@ __device__ __forceinline__ float tanh_series(float x) {
 
 // CAP: 0 none, 1 small arguments (|scale q.k / softcap| <= 1/2 by the caller's promise), 2 any.
 // grid (tiles * splits, kv heads)
-template <int CAP>
-__global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs a, const FlashShape sh) {
+template <int CAP, bool TMA>
+__global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs a, const FlashShape sh, const __grid_constant__ FlashMaps maps) {
   extern __shared__ __align__(1024) unsigned char s_raw[];
-  __shared__ __align__(8) uint64_t k_full[2], v_full[2], s_ready[2], p_ready[2], pv_done[2], finished;
+  __shared__ __align__(8) uint64_t k_full[2], v_full[2], s_ready[2], p_ready[2], pv_done[2], q_full, finished;
   __shared__ uint32_t s_tmem;
   __shared__ int s_abort;
   __shared__ float2 s_ml[2][kM];
@@ -149,12 +164,13 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
   if (tid == 0) {
     s_abort = 0;
     for (int w = 0; w < 2; ++w) {
-      mbar_init(&k_full[w], kLoaders);
-      mbar_init(&v_full[w], kLoaders);
+      mbar_init(&k_full[w], TMA ? 1 : kLoaders);
+      mbar_init(&v_full[w], TMA ? 1 : kLoaders);
       mbar_init(&s_ready[w], 1);
       mbar_init(&p_ready[w], 128);
       mbar_init(&pv_done[w], 1);
     }
+    mbar_init(&q_full, kLoaders);
     mbar_init(&finished, 1);
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
@@ -172,24 +188,15 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
   const int first = pos_r + p0 / gq;
   int last = pos_r + (p0 + np - 1) / gq;
   if (a.geom.ring == 0) last = min(last, (int)a.geom.rows - 1);
-  const BlockKeys keys(first, pos_r < 0 ? -1 : last, a.window, 0, a.chunk);
-  const int tiles = (keys.count + kKeys - 1) / kKeys;
+  const int begin = TMA ? VisibleRange(first, a.window, 0, a.chunk).lo / kKeys * kKeys : VisibleRange(first, a.window, 0, a.chunk).lo;
+  const int count = pos_r < 0 ? 0 : last - begin + 1;       // keys from position `begin` on
+  const int tiles = (count + kKeys - 1) / kKeys;
   const int t0 = (int)((int64_t)tiles * split / sh.splits), t1 = (int)((int64_t)tiles * (split + 1) / sh.splits);
   const int nj[2] = {(t1 - t0 + 1) / 2, (t1 - t0) / 2};   // tiles t0 + 2 j + w of warpgroup w
 
   if (warp >= 9) {   // ---- copies ----
     const int lt = tid - 288;
     const int slot = pos_r < 0 ? 0 : a.r.slots[0];
-    Rows ks, ks2, vs;
-    const int split_piece = a.key_rows ? a.key_cols >> 3 : kpieces, total = a.dim >> 3;
-    if (a.key_rows) {   // written out by position, the rest of a key in the cache
-      ks = Rows{static_cast<const __nv_bfloat16*>(a.key_rows) + (size_t)kv * a.key_cols, a.row_stride, keys.lo - a.key_base, INT_MAX, 0};
-      vs = Rows{static_cast<const __nv_bfloat16*>(a.value_rows) + (size_t)kv * a.vdim, a.row_stride, keys.lo - a.key_base, INT_MAX, 0};
-      ks2 = cache_rows(a, static_cast<const __nv_bfloat16*>(a.k_cache) + a.rest_col, 1, a.cache_row, 0, slot, keys.lo);
-    } else {
-      ks = ks2 = cache_rows(a, a.k_cache, a.kv_heads, a.dpad, kv, slot, keys.lo);
-      vs = cache_rows(a, a.v_cache, a.kv_heads, a.vpad, kv, slot, keys.lo);
-    }
     {   // the queries
       const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q);
       int r = lt / kpieces, c = lt - r * kpieces;
@@ -206,6 +213,58 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
           ++r;
         }
       }
+    }
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+    mbar_arrive(&q_full);
+    if constexpr (TMA) {
+      if (lt == 0) {
+        const int kpanels = kbytes / kPanel, vpanels = vbytes / kPanel, kfirst = a.key_rows ? a.key_cols >> 6 : kpanels;
+        const size_t slot_row = (size_t)slot * a.geom.rows;
+        int k_issued[2] = {0, 0}, v_issued[2] = {0, 0};
+        bool ok = true;
+        for (int j = 0; ok && j < nj[0]; ++j) {
+          for (int w = 0; w < 2; ++w) {
+            if (j >= nj[w]) continue;
+            if (j > 0 && !(ok = mbar_wait(&s_ready[w], (uint32_t)(j - 1) & 1u, &s_abort, &g_flash_fault))) break;
+            const int k0 = begin + (t0 + 2 * j + w) * kKeys, crow = (int)(slot_row + a.geom.row_of(k0));
+            k_issued[w] = j + 1;
+            mbar_expect_tx(&k_full[w], (uint32_t)kbytes);
+            for (int c = 0; c < kpanels; ++c) {
+              const uint32_t dst = k_at + (uint32_t)(w * kbytes + c * kPanel);
+              if (c >= kfirst) tma_panel(dst, &maps.rest, a.rest_col + (c - kfirst) * 64, crow, &k_full[w]);
+              else if (a.key_rows) tma_panel(dst, &maps.k, kv * a.key_cols + c * 64, k0 - a.key_base, &k_full[w]);
+              else tma_panel(dst, &maps.k, kv * a.dpad + c * 64, crow, &k_full[w]);
+            }
+          }
+          for (int w = 0; ok && w < 2; ++w) {
+            if (j >= nj[w]) continue;
+            if (j > 0 && !(ok = mbar_wait(&pv_done[w], (uint32_t)(j - 1) & 1u, &s_abort, &g_flash_fault))) break;
+            const int k0 = begin + (t0 + 2 * j + w) * kKeys, crow = (int)(slot_row + a.geom.row_of(k0));
+            v_issued[w] = j + 1;
+            mbar_expect_tx(&v_full[w], (uint32_t)vbytes);
+            for (int c = 0; c < vpanels; ++c)
+              tma_panel(v_at + (uint32_t)(w * vbytes + c * kPanel), &maps.v, kv * (a.key_rows ? a.vdim : a.vpad) + c * 64, a.key_rows ? k0 - a.key_base : crow, &v_full[w]);
+          }
+        }
+        if (!ok) {   // copies in flight land before the shared memory is given back: the last one issued per slot
+          int no_abort = 0;
+          for (int w = 0; w < 2; ++w) {
+            if (k_issued[w] > 0) mbar_wait(&k_full[w], (uint32_t)(k_issued[w] - 1) & 1u, &no_abort, &g_flash_fault);
+            if (v_issued[w] > 0) mbar_wait(&v_full[w], (uint32_t)(v_issued[w] - 1) & 1u, &no_abort, &g_flash_fault);
+          }
+        }
+      }
+    } else {
+    Rows ks, ks2, vs;
+    const int split_piece = a.key_rows ? a.key_cols >> 3 : kpieces, total = a.dim >> 3;
+    if (a.key_rows) {   // written out by position, the rest of a key in the cache
+      ks = Rows{static_cast<const __nv_bfloat16*>(a.key_rows) + (size_t)kv * a.key_cols, a.row_stride, begin - a.key_base, INT_MAX, 0};
+      vs = Rows{static_cast<const __nv_bfloat16*>(a.value_rows) + (size_t)kv * a.vdim, a.row_stride, begin - a.key_base, INT_MAX, 0};
+      ks2 = cache_rows(a, static_cast<const __nv_bfloat16*>(a.k_cache) + a.rest_col, 1, a.cache_row, 0, slot, begin);
+    } else {
+      ks = ks2 = cache_rows(a, a.k_cache, a.kv_heads, a.dpad, kv, slot, begin);
+      vs = cache_rows(a, a.v_cache, a.kv_heads, a.vpad, kv, slot, begin);
     }
     uint64_t* pending = nullptr;   // the load in flight in front of the one being issued
     auto flush = [&] {
@@ -234,24 +293,25 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
       for (int w = 0; ok && w < 2; ++w) {
         if (j >= nj[w]) continue;
         if (j > 0 && !(ok = freed(&s_ready[w], j - 1))) break;
-        load_tile(k_at + (uint32_t)(w * kbytes), ks, ks2, split_piece, a.key_rows ? total : kpieces, kpieces, (t0 + 2 * j + w) * kKeys, keys.count, lt);
+        load_tile(k_at + (uint32_t)(w * kbytes), ks, ks2, split_piece, a.key_rows ? total : kpieces, kpieces, (t0 + 2 * j + w) * kKeys, count, lt);
         issued(&k_full[w]);
       }
       for (int w = 0; ok && w < 2; ++w) {
         if (j >= nj[w]) continue;
         if (j > 0 && !(ok = freed(&pv_done[w], j - 1))) break;
-        load_tile(v_at + (uint32_t)(w * vbytes), vs, vs, vpieces, a.key_rows ? a.vdim >> 3 : vpieces, vpieces, (t0 + 2 * j + w) * kKeys, keys.count, lt);
+        load_tile(v_at + (uint32_t)(w * vbytes), vs, vs, vpieces, a.key_rows ? a.vdim >> 3 : vpieces, vpieces, (t0 + 2 * j + w) * kKeys, count, lt);
         issued(&v_full[w]);
       }
     }
     flush();
     asm volatile("cp.async.wait_all;" ::: "memory");
+    }
   } else if (warp == 8) {
     if (lane == 0) {   // ---- MMA issue ----
       constexpr uint32_t idesc_s = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(kKeys >> 3) << 17) | ((uint32_t)(kM >> 4) << 24);
       const uint32_t idesc_o = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(a.vpad >> 3) << 17) | ((uint32_t)(kM >> 4) << 24);
       const int ksteps = a.dpad >> 4;
-      bool ok = true;
+      bool ok = mbar_wait(&q_full, 0u, &s_abort, &g_flash_fault);
       for (int j = 0; ok && j <= nj[0]; ++j)
         for (int w = 0; ok && w < 2; ++w) {
           if (j >= 1 && j - 1 < nj[w]) {   // the output of the tile before
@@ -304,7 +364,7 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
 #pragma unroll
       for (int c = 0; c < kKeys; c += 32) tmem_ld32(st + (uint32_t)c, s + c);
       tmem_wait_ld();
-      const int v0 = (t0 + 2 * j + w) * kKeys, k0 = keys.lo + v0;   // position of the tile's first key
+      const int v0 = (t0 + 2 * j + w) * kKeys, k0 = begin + v0;   // position of the tile's first key
       const float base = -slope * (float)(pos - k0);
 #pragma unroll
       for (int c = 0; c < kKeys; ++c) {
@@ -451,6 +511,23 @@ size_t tc5_bytes(int dpad, int vpad) {
   return (tiles > out ? tiles : out) + 1024;
 }
 
+// Panels of 64 columns x 128 rows of a row-major bf16 matrix, 128-byte swizzle, zeros outside.
+bool panel_map(CUtensorMap* map, const void* base, int64_t cols, int64_t rows, int64_t stride) {
+  using Encode = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                              const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+  static Encode encode = [] {
+    void* fn = nullptr;
+    cudaDriverEntryPointQueryResult found;
+    if (cudaGetDriverEntryPointByVersion("cuTensorMapEncodeTiled", &fn, 12000, cudaEnableDefault, &found) != cudaSuccess || found != cudaDriverEntryPointSuccess) fn = nullptr;
+    return reinterpret_cast<Encode>(fn);
+  }();
+  if (!encode || rows < 1 || rows > INT_MAX) return false;
+  const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)stride * 2};
+  const cuuint32_t box[2] = {64, (cuuint32_t)kKeys}, steps[2] = {1, 1};
+  return encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, steps, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+
 }  // namespace
 
 int flash_fault_flag() {
@@ -483,10 +560,25 @@ tb_status launch_flash_tc5(const FlashArgs& a, cudaStream_t st, int* splits_out)
   *splits_out = sh.splits;
   const dim3 grid((unsigned)(sh.tiles * sh.splits), (unsigned)a.kv_heads);
   const size_t smem = tc5_bytes(a.dpad, a.vpad);
-  if (a.softcap <= 0.f) return launch_kernel(flash_tc5_kernel<0>, grid, dim3(kThreads), smem, st, a.pdl, 1, a, sh);
   // unit-norm queries and keys, rounded to bf16: |q . k| <= 1.01 dim
-  if (a.unit_norm && 1.01f * fabsf(a.scale) * (float)a.dim <= 0.5f * a.softcap) return launch_kernel(flash_tc5_kernel<1>, grid, dim3(kThreads), smem, st, a.pdl, 1, a, sh);
-  return launch_kernel(flash_tc5_kernel<2>, grid, dim3(kThreads), smem, st, a.pdl, 1, a, sh);
+  const int cap = a.softcap <= 0.f ? 0 : (a.unit_norm && 1.01f * fabsf(a.scale) * (float)a.dim <= 0.5f * a.softcap ? 1 : 2);
+  FlashMaps maps;
+  memset(&maps, 0, sizeof(maps));
+  bool tma = a.geom.ring % kKeys == 0 && a.geom.keep == 0 && a.cache_slots > 0;
+  if (a.key_rows) {
+    const int64_t n = a.key_count;
+    tma = tma && a.key_cols % 64 == 0 && a.key_base % kKeys == 0 && panel_map(&maps.k, a.key_rows, (int64_t)a.kv_heads * a.key_cols, n, a.row_stride) &&
+          panel_map(&maps.v, a.value_rows, (int64_t)a.kv_heads * a.vdim, n, a.row_stride) &&
+          panel_map(&maps.rest, a.k_cache, a.cache_row, a.cache_slots * a.geom.rows, a.cache_row);
+  } else {
+    const int64_t n = (int64_t)a.cache_slots * a.geom.rows, kw = (int64_t)a.kv_heads * a.dpad, vw = (int64_t)a.kv_heads * a.vpad;
+    tma = tma && panel_map(&maps.k, a.k_cache, kw, n, kw) && panel_map(&maps.v, a.v_cache, vw, n, vw);
+  }
+  using Kernel = void (*)(FlashArgs, FlashShape, FlashMaps);
+  static const Kernel kernels[3][2] = {{flash_tc5_kernel<0, false>, flash_tc5_kernel<0, true>},
+                                       {flash_tc5_kernel<1, false>, flash_tc5_kernel<1, true>},
+                                       {flash_tc5_kernel<2, false>, flash_tc5_kernel<2, true>}};
+  return launch_kernel(kernels[cap][tma ? 1 : 0], grid, dim3(kThreads), smem, st, a.pdl, 1, a, sh, maps);
 }
 
 }  // namespace tb

@@ -354,7 +354,7 @@ tb_status create_impl(LayeredModel* m, const tb_layered_layer* layers, const Lay
     r.max_visible = (int64_t)reach + r.keep_first < S ? (int64_t)reach + r.keep_first : S;
     // ring behind the window or the chunk: everything the first row of a step sees must survive the rows appended with
     // it, and a sequence taken back by up to kHistory positions still finds its window
-    const int64_t ring = (int64_t)reach + (m->max_rows > kHistory ? m->max_rows : kHistory);
+    const int64_t ring = pad_to((int64_t)reach + (m->max_rows > kHistory ? m->max_rows : kHistory), r.keep_first == 0 ? 128 : 1);   // 128: whole tiles of keys
     if (r.keep_first + ring < S) {
       r.geom.keep = r.keep_first;
       r.geom.ring = (int)ring;
@@ -562,7 +562,7 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
 
   // ---- mixers: the normed rows in ax -> operand of the output product ----
   auto flash = [&](FlashArgs& fa, const LayerRun& run) -> tb_status {
-    fa.r = r; fa.k_cache = run.k_cache; fa.v_cache = run.v_cache; fa.geom = run.geom;
+    fa.r = r; fa.k_cache = run.k_cache; fa.v_cache = run.v_cache; fa.geom = run.geom; fa.cache_slots = m->B;
     fa.scale = run.scale; fa.softcap = run.softcap; fa.slopes = run.slopes;
     fa.window = run.window; fa.keep_first = run.keep_first; fa.chunk = run.chunk; fa.max_visible = run.max_visible;
     fa.parts = m->flash_parts; fa.part_ml = m->part_ml; fa.part_slots = m->flash_slots;
@@ -647,7 +647,7 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
       TB_TRY(launch_latent_query(prec, lq, st));
       LatentRowsArgs lr;
       lr.r = r; lr.cache = run.k_cache; lr.geom = run.geom; lr.kv_rank = w.kv_rank; lr.dpad = w.dpad; lr.pdl = s.pdl;
-      lr.lo = VisibleRange((int)s.start, run.window, 0, run.chunk).lo;
+      lr.lo = VisibleRange((int)s.start, run.window, 0, run.chunk).lo / 128 * 128;   // whole tiles of keys
       lr.n = (int)s.start + rows - lr.lo;
       lr.out = ActOperand{m->act_l, dense_row_pad(lr.n), (int)w.ukv.kp};
       TB_TRY(launch_latent_rows(lr, st));
@@ -660,7 +660,7 @@ tb_status layered_enqueue(LayeredModel* m, const LayeredStep& s, cudaStream_t st
       FlashArgs fa;
       fa.heads = fa.kv_heads = w.heads; fa.dim = w.dim + w.rot_dim; fa.vdim = w.vdim; fa.dpad = w.xpad; fa.vpad = (int)pad_to(w.vdim, 16);
       fa.key_rows = m->expanded; fa.value_rows = m->expanded + (int64_t)w.heads * w.dim;
-      fa.key_cols = w.dim; fa.key_base = lr.lo; fa.row_stride = (int)row; fa.rest_col = w.kv_rank; fa.cache_row = w.dpad;
+      fa.key_cols = w.dim; fa.key_base = lr.lo; fa.key_count = lr.n; fa.row_stride = (int)row; fa.rest_col = w.kv_rank; fa.cache_row = w.dpad;
       fa.out = out;
       return flash(fa, run);
     }

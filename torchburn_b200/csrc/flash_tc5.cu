@@ -323,8 +323,9 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
             const uint32_t pt = tmem + (uint32_t)(w * 128), ot = tmem + 256u + (uint32_t)(w * 128);
 #pragma unroll
             for (int kk = 0; kk < kKeys / 16; ++kk) {
-              mma_bf16_ts(ot, pt + (uint32_t)(kk * 8), v_lo + (uint32_t)(kk * 128), idesc_o, (j > 1 || kk > 0) ? 1u : 0u);
-              mma_bf16_ts(ot, pt + 64u + (uint32_t)(kk * 8), v_lo + (uint32_t)(kk * 128), idesc_o, 1u);
+              const uint32_t at = pt + (uint32_t)((kk >> 1) * 32 + (kk & 1) * 8);   // per 32 keys: 16 columns of the one piece, 16 of the other
+              mma_bf16_ts(ot, at, v_lo + (uint32_t)(kk * 128), idesc_o, (j > 1 || kk > 0) ? 1u : 0u);
+              mma_bf16_ts(ot, at + 16u, v_lo + (uint32_t)(kk * 128), idesc_o, 1u);
             }
             mma_commit(&pv_done[w]);
           }
@@ -360,29 +361,36 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) break;
       tc_fence_after();
-      float s[kKeys];
-#pragma unroll
-      for (int c = 0; c < kKeys; c += 32) tmem_ld32(st + (uint32_t)c, s + c);
-      tmem_wait_ld();
       const int v0 = (t0 + 2 * j + w) * kKeys, k0 = begin + v0;   // position of the tile's first key
-      const float base = -slope * (float)(pos - k0);
+      const bool edge = !(k0 + kKeys - 1 <= first && k0 >= lo_last);   // not every row sees every key
+      const int jlo = lo - k0, jhi = row_live ? pos - k0 : -1;
+      float mx = -INFINITY;
+      // 32 columns at a time: few registers, and code that the instruction cache holds
+#pragma unroll 1
+      for (int q = 0; q < kKeys; q += 32) {
+        float s[32];
+        tmem_ld32(st + (uint32_t)q, s);
+        tmem_wait_ld();
+        const float base = -slope * (float)(pos - k0 - q);
 #pragma unroll
-      for (int c = 0; c < kKeys; ++c) {
-        float x = s[c] * in;
-        if (CAP == 1) x = fmaf(cap, tanh_series(x), base);
-        else if (CAP == 2) x = fmaf(-2.f * cap, __fdividef(1.f, ex2(x) + 1.f), cap + base);
-        else x += base;
-        s[c] = fmaf(slope, (float)c, x);
+        for (int c = 0; c < 32; ++c) {
+          float x = s[c] * in;
+          if (CAP == 1) x = fmaf(cap, tanh_series(x), base);
+          else if (CAP == 2) x = fmaf(-2.f * cap, __fdividef(1.f, ex2(x) + 1.f), cap + base);
+          else x += base;
+          s[c] = fmaf(slope, (float)c, x);
+        }
+        if (edge) {
+#pragma unroll
+          for (int c = 0; c < 32; ++c)
+            if (q + c < jlo || q + c > jhi) s[c] = -INFINITY;
+        }
+#pragma unroll
+        for (int c = 0; c < 32; ++c) mx = fmaxf(mx, s[c]);
+        tmem_st16(st + (uint32_t)q, reinterpret_cast<const uint32_t*>(s));
+        tmem_st16(st + (uint32_t)q + 16u, reinterpret_cast<const uint32_t*>(s) + 16);
       }
-      if (!(k0 + kKeys - 1 <= first && k0 >= lo_last)) {   // not every row sees every key
-        const int jlo = lo - k0, jhi = row_live ? pos - k0 : -1;
-#pragma unroll
-        for (int c = 0; c < kKeys; ++c)
-          if (c < jlo || c > jhi) s[c] = -INFINITY;
-      }
-      float mx = s[0];
-#pragma unroll
-      for (int c = 1; c < kKeys; ++c) mx = fmaxf(mx, s[c]);
+      tmem_wait_st();
       // the reference the weights are taken against moves only when it must
       const bool grow = mx > m + kGrow || m == -INFINITY;
       const float m1 = grow ? fmaxf(m, mx) : m;
@@ -404,12 +412,15 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
       m = m1;
       const float ref = m == -INFINITY ? 0.f : m;   // nothing seen yet: weights 2^-inf = 0
       float sum0 = 0.f, sum1 = 0.f;
-#pragma unroll
-      for (int c = 0; c < kKeys; c += 32) {
+#pragma unroll 1
+      for (int q = 0; q < kKeys; q += 32) {   // the two pieces of 32 weights take the place of their scores
+        float s[32];
         uint32_t hi[16], rest[16];
+        tmem_ld32(st + (uint32_t)q, s);
+        tmem_wait_ld();
 #pragma unroll
         for (int x = 0; x < 16; ++x) {
-          const float w0 = ex2(s[c + 2 * x] - ref), w1 = ex2(s[c + 2 * x + 1] - ref);
+          const float w0 = ex2(s[2 * x] - ref), w1 = ex2(s[2 * x + 1] - ref);
           sum0 += w0;
           sum1 += w1;
           const __nv_bfloat162 h2 = __floats2bfloat162_rn(w0, w1);
@@ -417,8 +428,8 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
           const __nv_bfloat162 r2 = __floats2bfloat162_rn(w0 - __uint_as_float(hi[x] << 16), w1 - __uint_as_float(hi[x] & 0xFFFF0000u));
           rest[x] = *reinterpret_cast<const uint32_t*>(&r2);
         }
-        tmem_st16(st + (uint32_t)(c >> 1), hi);
-        tmem_st16(st + 64u + (uint32_t)(c >> 1), rest);
+        tmem_st16(st + (uint32_t)q, hi);
+        tmem_st16(st + (uint32_t)q + 16u, rest);
       }
       l += sum0 + sum1;
       tmem_wait_st();

@@ -23,6 +23,7 @@ using namespace tc5;
 
 constexpr int kTile = 128;            // output features per CTA
 constexpr int kTileBytes = 16384;     // 128 rows x 64 bf16
+constexpr int kShortLoop = 16;        // K blocks
 
 __device__ int g_dense_fault = 0;
 
@@ -148,6 +149,8 @@ __global__ void __launch_bounds__(192) dense_tc5_kernel(const GemmParams p) {
       float* dst = static_cast<float*>(p.out) + (size_t)split * p.split_stride + (size_t)row0 * p.ldo + n;
       const int64_t col = (int64_t)batch * p.batch_cols + n;
       const int nrows = min(p.rows - row0, BN);
+      // eight features of a row lie side by side, on a 16-byte boundary
+      const bool wide = p.sink != DenseSink::kPartials && ((p.n_valid | p.batch_cols | (p.sink == DenseSink::kRows ? p.ldo : 0)) & 7) == 0;
 #pragma unroll 1
       for (int c = 0; c < nrows; c += 16) {
         uint32_t r[2][8];
@@ -158,6 +161,25 @@ __global__ void __launch_bounds__(192) dense_tc5_kernel(const GemmParams p) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
             if (c + j < nrows) dst[(size_t)(c + j) * p.ldo] = __uint_as_float(r[j >> 3][j & 7]);
+        } else if (wide) {
+          // through the warp's corner of the first stage (every MMA has read it): 16 rows x 32 features, then 8 features
+          // per store
+          __nv_bfloat16* t = reinterpret_cast<__nv_bfloat16*>(smem) + warp * (16 * 40);
+#pragma unroll
+          for (int j = 0; j < 16; ++j) t[j * 40 + lane] = __float2bfloat16_rn(activate(p.act, __uint_as_float(r[j >> 3][j & 7])));
+          __syncwarp();
+#pragma unroll
+          for (int h = 0; h < 2; ++h) {
+            const int j = (lane >> 2) + h * 8, f = (lane & 3) * 8;
+            if (c + j < nrows && n - lane + f < p.n_valid) {
+              const uint4 v = *reinterpret_cast<const uint4*>(t + j * 40 + f);
+              const int64_t k = col - lane + f;
+              if (p.sink == DenseSink::kOperand)
+                *reinterpret_cast<uint4*>(static_cast<unsigned char*>(p.operand.data) + image_offset(p.operand.mp, row0 + c + j, (int)k)) = v;
+              else *reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.out) + (size_t)(row0 + c + j) * p.ldo + k) = v;
+            }
+          }
+          __syncwarp();
         } else if (live) {
 #pragma unroll
           for (int j = 0; j < 16; ++j)
@@ -359,7 +381,10 @@ tb_status launch_dense_gemm(Precision prec, const DenseGemmArgs& a, cudaStream_t
     case 32: return launch_tc5<32, 5>(p, n_tiles, nz, a.pdl, st);
     case 64: return launch_tc5<64, 4>(p, n_tiles, nz, a.pdl, st);
     case 128: return launch_tc5<128, 6>(p, n_tiles, nz, a.pdl, st);
-    default: return launch_tc5<256, 4>(p, n_tiles, nz, a.pdl, st);
+    default:
+      // a short K loop is mostly epilogue: two CTAs per SM, one stores while the other computes
+      if (p.kb_per <= kShortLoop) return launch_tc5<256, 2>(p, n_tiles, nz, a.pdl, st);
+      return launch_tc5<256, 4>(p, n_tiles, nz, a.pdl, st);
   }
 }
 

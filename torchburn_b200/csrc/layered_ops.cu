@@ -430,7 +430,14 @@ __device__ __forceinline__ float warp_sum(float v) {
 
 // Per head: a warp takes one head of q, k or v through its norm (or the value mixing) to where it goes; one more
 // warp per 32 heads does the gates.  grid (warps of a row / 8, rows)
-template <typename T>
+__device__ __forceinline__ void store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
+  const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+
+// V4: sizes are multiples of four, a lane takes four columns at a time; else one.
+template <typename T, bool V4>
 __global__ void __launch_bounds__(kThreads) heads_prep_kernel(const HeadsPrepArgs a) {
   constexpr int KEEP = 8;                  // values a lane keeps between the norm's two passes
   const int lane = threadIdx.x & 31, r = (int)blockIdx.y;
@@ -443,20 +450,34 @@ __global__ void __launch_bounds__(kThreads) heads_prep_kernel(const HeadsPrepArg
     const bool is_q = u < a.heads;
     const int h = is_q ? u : u - a.heads, col = (is_q ? a.q_off : a.k_off) + h * a.dim;
     float v[KEEP], ss = 0.f;
-#pragma unroll
-    for (int j = 0; j < KEEP; ++j)
-      if (lane + 32 * j < a.dim) {
-        v[j] = sum_column(a.y, r, col + lane + 32 * j);
-        ss = fmaf(v[j], v[j], ss);
+    float4 w4[2];
+    if constexpr (V4) {
+      for (int c = lane * 4, e = 0; c < a.dim; c += 128, ++e) {
+        const float4 x = sum_partials(a.y, r, col + c);
+        if (e == 0) w4[0] = x;
+        else if (e == 1) w4[1] = x;
+        ss += dot4(x);
       }
-    for (int c = lane + 32 * KEEP; c < a.dim; c += 32) {
-      const float x = sum_column(a.y, r, col + c);
-      ss = fmaf(x, x, ss);
+    } else {
+#pragma unroll
+      for (int j = 0; j < KEEP; ++j)
+        if (lane + 32 * j < a.dim) {
+          v[j] = sum_column(a.y, r, col + lane + 32 * j);
+          ss = fmaf(v[j], v[j], ss);
+        }
+      for (int c = lane + 32 * KEEP; c < a.dim; c += 32) {
+        const float x = sum_column(a.y, r, col + c);
+        ss = fmaf(x, x, ss);
+      }
     }
     const float inv = a.unit_norm ? 1.0f / sqrtf(warp_sum(ss) / (float)a.dim + a.eps) : 1.f;
     T* dst = is_q ? static_cast<T*>(a.q) + ((size_t)r * a.heads + h) * a.dpad
                   : static_cast<T*>(a.k_cache) + crow * (size_t)(a.kv_heads * a.dpad) + h * a.dpad;
     if (!is_q && pos < 0) return;
+    if constexpr (V4) {
+      for (int c = lane * 4, e = 0; c < a.dim; c += 128, ++e) store4(dst + c, scale4(e == 0 ? w4[0] : (e == 1 ? w4[1] : sum_partials(a.y, r, col + c)), inv));
+      return;
+    }
 #pragma unroll
     for (int j = 0; j < KEEP; ++j)
       if (lane + 32 * j < a.dim) dst[lane + 32 * j] = (T)(v[j] * inv);
@@ -467,6 +488,15 @@ __global__ void __launch_bounds__(kThreads) heads_prep_kernel(const HeadsPrepArg
   if (u < a.kv_heads) {
     T* dst = static_cast<T*>(a.v_cache) + crow * (size_t)(a.kv_heads * a.vpad) + u * a.vpad;
     float* first = a.v_first ? a.v_first + (size_t)r * a.kv_heads * a.vdim + u * a.vdim : nullptr;
+    if constexpr (V4) {
+      for (int c = lane * 4; c < a.vdim; c += 128) {
+        float4 v = sum_partials(a.y, r, a.v_off + u * a.vdim + c);
+        if (first && a.keep_first_values) store4(first + c, v);
+        else if (first) v = fma4(f4(a.mix), ld4(first + c), scale4(v, 1.f - a.mix));
+        if (pos >= 0) store4(dst + c, v);
+      }
+      return;
+    }
     for (int c = lane; c < a.vdim; c += 32) {
       float v = sum_column(a.y, r, a.v_off + u * a.vdim + c);
       if (first && a.keep_first_values) first[c] = v;
@@ -521,7 +551,7 @@ __global__ void __launch_bounds__(kThreads) latent_prep_kernel(const LatentPrepA
 
 // The heads' queries after the up-projection: the unrotated part as the operand of the product with the head's
 // key matrix, the rotated part behind the place of that product in the query.  Warp per head, grid (heads / 8, rows)
-template <typename T>
+template <typename T, bool V4>
 __global__ void __launch_bounds__(kThreads) latent_query_kernel(const LatentQueryArgs a) {
   const int lane = threadIdx.x & 31, r = (int)blockIdx.y, h = (int)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
   grid_dep_launch();
@@ -529,6 +559,23 @@ __global__ void __launch_bounds__(kThreads) latent_query_kernel(const LatentQuer
   if (h >= a.heads) return;
   const int pos = a.r.pos[r], col = h * (a.dim + a.rot_dim);
   T* q = static_cast<T*>(a.q) + ((size_t)r * a.heads + h) * a.dpad;
+  if constexpr (V4) {
+    ActOperand out = a.out;
+    if (out.data) out.data = static_cast<unsigned char*>(out.data) + (size_t)h * out.mp * out.kp * sizeof(T);
+    const int n = out.data ? out.kp : a.dim;
+    for (int c = lane * 4; c < n; c += 128) {
+      const float4 v = c < a.dim ? sum_partials(a.y, r, col + c) : f4(0.f);
+      if (out.data) act_store4<sizeof(T) == 2>(out, r, c, v);
+      else store4(q + c, v);
+    }
+    q += a.rot_at;
+    for (int c = lane * 4; c < a.rot_dim; c += 128) {
+      const float4 v = sum_partials(a.y, r, col + a.dim + c);
+      store4(q + c, make_float4(rotated(a.table, a.rot_dims, pos, c, v.x, v.y), rotated(a.table, a.rot_dims, pos, c + 1, v.y, v.x),
+                                rotated(a.table, a.rot_dims, pos, c + 2, v.z, v.w), rotated(a.table, a.rot_dims, pos, c + 3, v.w, v.z)));
+    }
+    return;
+  }
   if (a.out.data) {
     ActOperand out = a.out;
     out.data = static_cast<unsigned char*>(out.data) + (size_t)h * out.mp * out.kp * sizeof(T);
@@ -644,7 +691,7 @@ tb_status launch_glue(Precision p, const GlueArgs& a, cudaStream_t st) {
   }
   const int c = row_cluster(n, a.xs / 4);
   int per = 1;
-  if (c == 1)
+  if (c == 1 && a.conv_w)
     while (per < 4 && n / (per * 2) >= sm_count()) per *= 2;   // fewer rows computed again in front of each block
   const int e4 = (a.xs / 4 + c * kThreads - 1) / (c * kThreads);
   const int taps = a.conv_w ? a.taps : 1;
@@ -674,8 +721,10 @@ tb_status launch_qkv_prep(Precision p, const QkvPrepArgs& a, cudaStream_t st) {
 tb_status launch_heads_prep(Precision p, const HeadsPrepArgs& a, cudaStream_t st) {
   const int warps = a.heads + 2 * a.kv_heads + (a.gate ? (a.heads + 31) / 32 : 0);
   const dim3 grid((unsigned)((warps + kThreads / 32 - 1) / (kThreads / 32)), (unsigned)a.r.rows);
-  return p == Precision::kBf16 ? launch_kernel(heads_prep_kernel<__nv_bfloat16>, grid, dim3(kThreads), 0, st, a.pdl, 1, a)
-                               : launch_kernel(heads_prep_kernel<float>, grid, dim3(kThreads), 0, st, a.pdl, 1, a);
+  using Kernel = void (*)(HeadsPrepArgs);
+  static const Kernel kernels[2][2] = {{heads_prep_kernel<__nv_bfloat16, false>, heads_prep_kernel<__nv_bfloat16, true>},
+                                       {heads_prep_kernel<float, false>, heads_prep_kernel<float, true>}};
+  return launch_kernel(kernels[p == Precision::kF32][a.dim % 4 == 0 && a.vdim % 4 == 0], grid, dim3(kThreads), 0, st, a.pdl, 1, a);
 }
 
 tb_status launch_latent_prep(Precision p, const LatentPrepArgs& a, cudaStream_t st) {
@@ -688,8 +737,11 @@ tb_status launch_latent_prep(Precision p, const LatentPrepArgs& a, cudaStream_t 
 
 tb_status launch_latent_query(Precision p, const LatentQueryArgs& a, cudaStream_t st) {
   const dim3 grid((unsigned)((a.heads + kThreads / 32 - 1) / (kThreads / 32)), (unsigned)a.r.rows);
-  return p == Precision::kBf16 ? launch_kernel(latent_query_kernel<__nv_bfloat16>, grid, dim3(kThreads), 0, st, a.pdl, 1, a)
-                               : launch_kernel(latent_query_kernel<float>, grid, dim3(kThreads), 0, st, a.pdl, 1, a);
+  using Kernel = void (*)(LatentQueryArgs);
+  static const Kernel kernels[2][2] = {{latent_query_kernel<__nv_bfloat16, false>, latent_query_kernel<__nv_bfloat16, true>},
+                                       {latent_query_kernel<float, false>, latent_query_kernel<float, true>}};
+  const bool v4 = a.dim % 4 == 0 && a.rot_dim % 4 == 0 && a.rot_at % 4 == 0;
+  return launch_kernel(kernels[p == Precision::kF32][v4], grid, dim3(kThreads), 0, st, a.pdl, 1, a);
 }
 
 tb_status launch_latent_rows(const LatentRowsArgs& a, cudaStream_t st) {

@@ -383,7 +383,7 @@ tb_status launch_dense_gemm(Precision prec, const DenseGemmArgs& a, cudaStream_t
     case 128: return launch_tc5<128, 6>(p, n_tiles, nz, a.pdl, st);
     default:
       // a short K loop is mostly epilogue: two CTAs per SM, one stores while the other computes
-      if (p.kb_per <= kShortLoop) return launch_tc5<256, 2>(p, n_tiles, nz, a.pdl, st);
+      if (p.kb_per <= kShortLoop && (int64_t)(p.mp / 256) * n_tiles * nz > sm_count()) return launch_tc5<256, 2>(p, n_tiles, nz, a.pdl, st);
       return launch_tc5<256, 4>(p, n_tiles, nz, a.pdl, st);
   }
 }

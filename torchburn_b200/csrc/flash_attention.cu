@@ -4,7 +4,10 @@
 //
 //   score(i, j) = cap(scale q_i . k_j) - slope_h (i - j),   cap(s) = softcap tanh(s / softcap)
 //
-// bf16 (flash_mma_kernel): a CTA takes up to 64 (query, head) pairs of one key/value head - the heads of one row in
+// bf16, decode steps with up to eight query heads per key head (flash_decode_kernel): a warp takes 32 keys at a time from
+// their load to its own running output and needs no other warp until the end; keys are the 16-row side of mma.sync, the
+// heads its eight columns.
+// bf16 otherwise (flash_mma_kernel): a CTA takes up to 64 (query, head) pairs of one key/value head - the heads of one row in
 // a decode step, several queries times the heads in a portion - so that heads that share keys share their loads.
 // Per tile of 32 or 64 keys: scores by mma.sync with the warps side by side over the keys, softmax weights to shared
 // memory as two bf16 pieces (the second one what the rounding of the first left: 16 mantissa bits), then the values
@@ -300,6 +303,239 @@ __global__ void __launch_bounds__(kThreads, NV <= 8 ? 2 : 1) flash_mma_kernel(co
   }
 }
 
+// The 8 x 8 matrix of 16-bit elements that a warp holds (row lane / 4, columns 2 (lane & 3) and the next), transposed.
+__device__ __forceinline__ uint32_t transposed(uint32_t v) {
+  uint32_t r;
+  asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
+  return r;
+}
+__device__ __forceinline__ uint32_t pack2(float x, float y) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+constexpr int kDecodeKeys = 32;   // keys a warp takes at a time
+constexpr int kDecodeHeads = 8;
+
+// grid (splits, kv heads, rows); DT: at most 16 DT elements of a key, of a value
+template <int DT>
+__global__ void __launch_bounds__(kThreads) flash_decode_kernel(const FlashArgs a, const FlashShape sh) {
+  extern __shared__ __align__(16) unsigned char s_raw[];
+  constexpr int KT = kDecodeKeys, NH = kDecodeHeads;
+  const int gq = a.heads / a.kv_heads, kv = (int)blockIdx.y, r = (int)blockIdx.z, split = (int)blockIdx.x;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = (int)blockDim.x >> 5;
+  const int ld = a.dpad + 8, vld = a.vpad + 8;
+  __nv_bfloat16* s_k = reinterpret_cast<__nv_bfloat16*>(s_raw) + (size_t)warp * 2 * KT * (ld + vld);   // the warp's [2][KT][ld], [2][KT][vld]
+  __nv_bfloat16* s_v = s_k + 2 * KT * ld;
+  grid_dep_launch();
+  grid_dep_wait();
+  const int pos = a.r.pos[r];
+  const BlockKeys keys(pos, pos, a.window, a.keep_first, a.chunk);
+  const int krow = a.kv_heads * a.dpad, vrow = a.kv_heads * a.vpad;
+  const size_t slot = pos < 0 ? 0 : (size_t)a.r.slots[r] * a.geom.rows;
+  const __nv_bfloat16* kc = static_cast<const __nv_bfloat16*>(a.k_cache) + slot * krow + (size_t)kv * a.dpad;
+  const __nv_bfloat16* vc = static_cast<const __nv_bfloat16*>(a.v_cache) + slot * vrow + (size_t)kv * a.vpad;
+  const int tiles = (keys.count + KT - 1) / KT;
+  const int t0 = (int)((int64_t)tiles * split / sh.splits), t1 = (int)((int64_t)tiles * (split + 1) / sh.splits);
+  // 32 rows of `pieces` 16-byte pieces each; row v of a whole tile in one piece of the cache is `row` elements behind row v - 1
+  auto rows_in = [&](__nv_bfloat16* dst, int dld, const __nv_bfloat16* src, int row, int pieces, const RunRows& rr, int v0, bool one_piece) {
+    int y = lane / pieces, c = lane - y * pieces;
+    const int dy = 32 / pieces, dc = 32 - dy * pieces;
+    if (one_piece) {
+      const __nv_bfloat16* s0 = src + (size_t)rr.row(v0) * row;
+      for (int i = 0; i < pieces; ++i) {
+        cp16z(dst + y * dld + c * 8, s0 + (size_t)(uint32_t)(y * row) + c * 8, true);
+        y += dy;
+        c += dc;
+        if (c >= pieces) { c -= pieces; ++y; }
+      }
+    } else {
+      for (int i = 0; i < pieces; ++i) {
+        const bool live = v0 + y < keys.count;
+        cp16z(dst + y * dld + c * 8, src + (size_t)(live ? rr.row(v0 + y) : 0) * row + c * 8, live);
+        y += dy;
+        c += dc;
+        if (c >= pieces) { c -= pieces; ++y; }
+      }
+    }
+  };
+  auto fetch = [&](int t, int buf) {
+    const int v0 = t * KT;
+    const RunRows rr(keys, a.geom, v0);
+    const bool one_piece = v0 + KT <= keys.count && rr.row(v0 + KT - 1) - rr.row(v0) == KT - 1;
+    rows_in(s_k + buf * KT * ld, ld, kc, krow, a.dpad >> 3, rr, v0, one_piece);
+    rows_in(s_v + buf * KT * vld, vld, vc, vrow, a.vpad >> 3, rr, v0, one_piece);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  if (t0 + warp < t1) fetch(t0 + warp, 0);
+  // the queries as the eight columns: element (k, head) with head lane / 4, k 2 (lane & 3) and the next, and 8 on
+  uint32_t qb[DT][2];
+  {
+    const int h = lane >> 2;
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q) + ((size_t)r * a.heads + kv * gq + (h < gq ? h : 0)) * a.dpad + (lane & 3) * 2;
+#pragma unroll
+    for (int ks = 0; ks < DT; ++ks) {
+      const bool live = h < gq && ks * 16 < a.dpad;
+      qb[ks][0] = live ? *reinterpret_cast<const uint32_t*>(q + ks * 16) : 0u;
+      qb[ks][1] = live ? *reinterpret_cast<const uint32_t*>(q + ks * 16 + 8) : 0u;
+    }
+  }
+  float slope[2], m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};   // of heads 2 (lane & 3) and the next
+#pragma unroll
+  for (int y = 0; y < 2; ++y) {
+    const int h = (lane & 3) * 2 + y;
+    slope[y] = a.slopes && h < gq ? a.slopes[kv * gq + h] * kLog2E : 0.f;
+  }
+  const float scale2 = a.scale * kLog2E, cap_in = a.softcap > 0.f ? 2.f * kLog2E * a.scale / a.softcap : 0.f, cap = a.softcap * kLog2E;
+  float acc[DT][4];
+#pragma unroll
+  for (int n = 0; n < DT; ++n)
+#pragma unroll
+    for (int i = 0; i < 4; ++i) acc[n][i] = 0.f;
+  int buf = 0;
+  for (int t = t0 + warp; t < t1; t += nw, buf ^= 1) {
+    if (t + nw < t1) {
+      fetch(t + nw, buf ^ 1);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncwarp();
+    const __nv_bfloat16 *k = s_k + buf * KT * ld, *v = s_v + buf * KT * vld;
+    float d[2][4];
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int i = 0; i < 4; ++i) d[x][i] = 0.f;
+#pragma unroll
+    for (int ks = 0; ks < DT; ++ks) {
+      if (ks * 16 >= a.dpad) break;
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        uint32_t ka[4];
+        ldm4(ka, k + (x * 16 + (lane & 15)) * ld + ks * 16 + (lane >> 4) * 8);
+        mma16816(d[x], ka, qb[ks][0], qb[ks][1]);
+      }
+    }
+    // d[x][2 z + y]: key 16 x + lane / 4 + 8 z, head 2 (lane & 3) + y.  Every numbered key of the row's own block is seen.
+    float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+      for (int z = 0; z < 2; ++z) {
+        const int n = t * KT + x * 16 + (lane >> 2) + 8 * z;
+        const float dist = (float)(pos - keys.position(n));
+#pragma unroll
+        for (int y = 0; y < 2; ++y) {
+          float s = d[x][2 * z + y];
+          if (a.softcap > 0.f) s = fmaf(-2.f * cap, __fdividef(1.f, exp2f(s * cap_in) + 1.f), cap);
+          else s *= scale2;
+          s = n < keys.count ? fmaf(-slope[y], dist, s) : -INFINITY;
+          d[x][2 * z + y] = s;
+          mx[y] = fmaxf(mx[y], s);
+        }
+      }
+    float alpha[2];
+#pragma unroll
+    for (int y = 0; y < 2; ++y) {
+#pragma unroll
+      for (int o = 16; o > 2; o >>= 1) mx[y] = fmaxf(mx[y], __shfl_xor_sync(0xffffffffu, mx[y], o));
+      const float mn = fmaxf(m[y], mx[y]);   // a tile holds at least one visible key
+      alpha[y] = exp2f(m[y] - mn);
+      m[y] = mn;
+      float sum = 0.f;
+#pragma unroll
+      for (int x = 0; x < 2; ++x)
+#pragma unroll
+        for (int z = 0; z < 2; ++z) {
+          const float w = exp2f(d[x][2 * z + y] - mn);
+          d[x][2 * z + y] = w;
+          sum += w;
+        }
+      l[y] = fmaf(l[y], alpha[y], sum);
+    }
+    if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
+#pragma unroll
+      for (int n = 0; n < DT; ++n)
+#pragma unroll
+        for (int i = 0; i < 4; ++i) acc[n][i] *= alpha[i & 1];
+    }
+#pragma unroll
+    for (int x = 0; x < 2; ++x) {   // 16 keys: weights in two pieces, [key][head] -> [head][key]
+      uint32_t hi[2], rest[2];
+#pragma unroll
+      for (int z = 0; z < 2; ++z) {
+        const float w0 = d[x][2 * z], w1 = d[x][2 * z + 1];
+        const uint32_t p = pack2(w0, w1);
+        hi[z] = transposed(p);
+        rest[z] = transposed(pack2(w0 - __uint_as_float(p << 16), w1 - __uint_as_float(p & 0xFFFF0000u)));
+      }
+#pragma unroll
+      for (int n = 0; n < DT; ++n) {
+        if (n * 16 >= a.vpad) break;
+        uint32_t va[4];   // 16 columns x 16 keys out of [key][column]
+        ldm4t(va, v + (x * 16 + (lane & 7) + (lane >> 4) * 8) * vld + n * 16 + ((lane >> 3) & 1) * 8);
+        mma16816(acc[n], va, hi[0], hi[1]);
+        mma16816(acc[n], va, rest[0], rest[1]);
+      }
+    }
+    __syncwarp();
+  }
+  // ---- the warps' shares ----
+  asm volatile("cp.async.wait_all;" ::: "memory");
+  __syncthreads();
+#pragma unroll
+  for (int y = 0; y < 2; ++y)
+#pragma unroll
+    for (int o = 16; o > 2; o >>= 1) l[y] += __shfl_xor_sync(0xffffffffu, l[y], o);
+  float2* s_ml = reinterpret_cast<float2*>(s_raw);                 // [warps][NH]
+  float* s_o = reinterpret_cast<float*>(s_ml + nw * NH);           // [warps][NH][vpad + 4]
+  const int old = a.vpad + 4;
+  if (lane < 4)
+#pragma unroll
+    for (int y = 0; y < 2; ++y) s_ml[warp * NH + lane * 2 + y] = make_float2(m[y], l[y]);
+#pragma unroll
+  for (int n = 0; n < DT; ++n) {
+    if (n * 16 >= a.vpad) break;
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {   // column lane / 4 + 8 (i / 2), head 2 (lane & 3) + (i & 1)
+      const int h = (lane & 3) * 2 + (i & 1);
+      if (h < gq) s_o[(warp * NH + h) * old + n * 16 + (lane >> 2) + (i >> 1) * 8] = acc[n][i];
+    }
+  }
+  __syncthreads();
+  const bool whole = sh.splits == 1;
+  for (int h = warp; h < gq; h += nw) {
+    const int head = kv * gq + h;
+    float mm = -INFINITY, sum = 0.f;
+    for (int w = 0; w < nw; ++w) mm = fmaxf(mm, s_ml[w * NH + h].x);
+    for (int w = 0; w < nw; ++w) {
+      const float2 p = s_ml[w * NH + h];
+      if (p.x != -INFINITY) sum = fmaf(p.y, exp2f(p.x - mm), sum);
+    }
+    float f = 1.f;
+    if (whole) {
+      f = sum > 0.f ? 1.f / sum : 0.f;
+      if (a.gate) f *= a.gate[(size_t)r * a.heads + head];
+    }
+    const size_t part = ((size_t)split * a.r.rows + r) * a.heads + head;
+    if (!whole && lane == 0) a.part_ml[part] = make_float2(mm, sum);
+    const int limit = whole ? flash_column_limit(a, head) : a.vdim;
+    for (int c = lane; c < limit; c += 32) {
+      float o = 0.f;
+      if (c < a.vdim)
+        for (int w = 0; w < nw; ++w) {
+          const float x = s_ml[w * NH + h].x;
+          if (x != -INFINITY) o = fmaf(s_o[(w * NH + h) * old + c], exp2f(x - mm), o);
+        }
+      if (whole) store_column<true>(a, r, head, c, o * f);
+      else a.parts[part * a.vdim + c] = o;
+    }
+  }
+}
+
+size_t decode_warp_bytes(const FlashArgs& a) { return (size_t)2 * kDecodeKeys * (a.dpad + a.vpad + 16) * 2; }
+
 // Merges the shares of a row's keys.  grid (heads, rows, columns / 128)
 __global__ void __launch_bounds__(128) flash_merge_kernel(const FlashArgs a, const int splits) {
   __shared__ float s_w[kMaxSplits], s_red[4], s_sum[4];
@@ -487,6 +723,23 @@ tb_status launch_flash_attention(Precision p, const FlashArgs& a, cudaStream_t s
     int splits = 1;
     TB_TRY(launch_flash_tc5(a, st, &splits));
     return merge(splits);
+  }
+  if (!a.one_sequence && !a.values_in_keys && gq <= kDecodeHeads && a.dpad <= 256 && a.vpad <= 256) {
+    // three CTAs per SM, or one of one warp
+    const size_t per = decode_warp_bytes(a);   // also holds a warp's merge: 8 (vpad + 4) floats and its statistics
+    int warps = (int)(72 * 1024 / per);
+    warps = warps < 1 ? 1 : (warps > 8 ? 8 : warps);
+    const int64_t tiles = (a.max_visible + kDecodeKeys - 1) / kDecodeKeys;
+    FlashShape sd;
+    int64_t splits = 3 * (int64_t)sm_count() / ((int64_t)rows * a.kv_heads);
+    if (splits > (tiles + warps - 1) / warps) splits = (tiles + warps - 1) / warps;
+    if (splits > kMaxSplits) splits = kMaxSplits;
+    if (splits > a.part_slots / ((int64_t)rows * a.heads)) splits = a.part_slots / ((int64_t)rows * a.heads);
+    sd.splits = splits < 1 ? 1 : (int)splits;
+    const int most = a.dpad > a.vpad ? a.dpad : a.vpad;
+    FlashKernel dec = most <= 64 ? flash_decode_kernel<4> : (most <= 128 ? flash_decode_kernel<8> : flash_decode_kernel<16>);
+    TB_TRY(launch_kernel(dec, dim3((unsigned)sd.splits, (unsigned)a.kv_heads, (unsigned)rows), dim3((unsigned)warps * 32), per * warps, st, a.pdl, 1, a, sd));
+    return merge(sd.splits);
   }
   if (a.key_rows) return fail(TB_ERR_SHAPE, "flash attention: keys in two pieces of %d and %d columns", a.key_cols, a.dim - a.key_cols);
   FlashShape sh;

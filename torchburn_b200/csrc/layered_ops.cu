@@ -284,6 +284,43 @@ __global__ void __launch_bounds__(kThreads) glue_kernel(const GlueArgs a, const 
   }
 }
 
+// Many rows, x' = x + y without a norm of y and without a convolution: one CTA per row, everything in registers.
+template <bool BF16, int E>
+__global__ void __launch_bounds__(kThreads) glue_row_kernel(const GlueArgs a) {
+  __shared__ ClusterSum<1> s_sum;
+  const int tid = threadIdx.x, r = a.row0 + (int)blockIdx.x, xs4 = a.xs >> 2;
+  grid_dep_launch();
+  grid_dep_wait();
+  const int pos = a.r.pos[r], orow = a.row_map != nullptr ? a.row_map[r] : r;
+  float4 v[E], y[E];
+  float ss[1] = {0.f};
+#pragma unroll
+  for (int e = 0; e < E; ++e) {
+    const int i = tid + e * kThreads;
+    if (i >= xs4) continue;
+    v[e] = ld4(a.x_in + (size_t)r * a.xs + i * 4);
+    y[e] = sum_partials(a.y, r, i * 4);
+  }
+#pragma unroll
+  for (int e = 0; e < E; ++e) {
+    const int i = tid + e * kThreads;
+    if (i >= xs4) continue;
+    if (a.y_bias) y[e] = add4(y[e], ld4(a.y_bias + i * 4));
+    v[e] = add4(v[e], y[e]);
+    ss[0] += dot4(v[e]);
+    if (a.x_out) *reinterpret_cast<float4*>(a.x_out + (size_t)r * a.xs + i * 4) = v[e];
+    if (a.snapshot) *reinterpret_cast<float4*>(a.snapshot + (size_t)r * a.xs + i * 4) = v[e];
+  }
+  cluster_sum<1>(s_sum, 0, 1, 0, ss);
+  if (a.out.data == nullptr || orow < 0) return;
+  const float inv = 1.0f / sqrtf(ss[0] / (float)a.width + a.eps);
+#pragma unroll
+  for (int e = 0; e < E; ++e) {
+    const int i = tid + e * kThreads;
+    if (i < xs4) act_store4<BF16>(a.out, orow, i * 4, pos < 0 ? f4(0.f) : mul4(scale4(v[e], inv), ld4(a.pre_w + i * 4)));
+  }
+}
+
 // Decode rows: every row its own sequence, four features per thread.  The same arithmetic as glue_kernel; the
 // weights are read before the grid dependency wait, everything else as soon as its address is known.
 constexpr int kStepTaps = 8;
@@ -700,6 +737,12 @@ tb_status launch_glue(Precision p, const GlueArgs& a, cudaStream_t st) {
     const dim3 grid((unsigned)(n * c));
     return p == Precision::kBf16 ? launch_kernel(glue_step_kernel<true>, grid, dim3(kThreads), 0, st, a.pdl, c, a)
                                  : launch_kernel(glue_step_kernel<false>, grid, dim3(kThreads), 0, st, a.pdl, c, a);
+  }
+  if (c == 1 && !a.conv_w && !a.post_w && !a.embed.img && a.y.y != nullptr && e4 <= 4) {
+    using Kernel = void (*)(GlueArgs);
+    static const Kernel kernels[2][4] = {{glue_row_kernel<true, 1>, glue_row_kernel<true, 2>, glue_row_kernel<true, 3>, glue_row_kernel<true, 4>},
+                                         {glue_row_kernel<false, 1>, glue_row_kernel<false, 2>, glue_row_kernel<false, 3>, glue_row_kernel<false, 4>}};
+    return launch_kernel(kernels[p == Precision::kF32][e4 - 1], dim3((unsigned)n), dim3(kThreads), 0, st, a.pdl, 1, a);
   }
   if (smem > 200 * 1024 || taps > 32) return fail(TB_ERR_UNSUPPORTED, "TB_UNSUPPORTED: hidden size %d with %d taps", a.width, a.taps);
   const dim3 grid((unsigned)((n + per - 1) / per * c));

@@ -303,6 +303,16 @@ __global__ void __launch_bounds__(kThreads, NV <= 8 ? 2 : 1) flash_mma_kernel(co
   }
 }
 
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+}
+__device__ __forceinline__ void ldm4(uint32_t (&r)[4], uint32_t at) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at));
+}
+__device__ __forceinline__ void ldm4t(uint32_t (&r)[4], uint32_t at) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at));
+}
+
 // The 8 x 8 matrix of 16-bit elements that a warp holds (row lane / 4, columns 2 (lane & 3) and the next), transposed.
 __device__ __forceinline__ uint32_t transposed(uint32_t v) {
   uint32_t r;
@@ -317,14 +327,14 @@ __device__ __forceinline__ uint32_t pack2(float x, float y) {
 constexpr int kDecodeKeys = 32;   // keys a warp takes at a time
 constexpr int kDecodeHeads = 8;
 
-// grid (splits, kv heads, rows); DT: at most 16 DT elements of a key, of a value
-template <int DT>
+// grid (splits, kv heads, rows); DT: at most 16 DT elements of a key, of a value (EXACT: that many of both)
+template <int DT, bool EXACT>
 __global__ void __launch_bounds__(kThreads) flash_decode_kernel(const FlashArgs a, const FlashShape sh) {
   extern __shared__ __align__(16) unsigned char s_raw[];
   constexpr int KT = kDecodeKeys, NH = kDecodeHeads;
   const int gq = a.heads / a.kv_heads, kv = (int)blockIdx.y, r = (int)blockIdx.z, split = (int)blockIdx.x;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, nw = (int)blockDim.x >> 5;
-  const int ld = a.dpad + 8, vld = a.vpad + 8;
+  const int ld = EXACT ? 16 * DT + 8 : a.dpad + 8, vld = EXACT ? 16 * DT + 8 : a.vpad + 8;
   __nv_bfloat16* s_k = reinterpret_cast<__nv_bfloat16*>(s_raw) + (size_t)warp * 2 * KT * (ld + vld);   // the warp's [2][KT][ld], [2][KT][vld]
   __nv_bfloat16* s_v = s_k + 2 * KT * ld;
   grid_dep_launch();
@@ -341,7 +351,17 @@ __global__ void __launch_bounds__(kThreads) flash_decode_kernel(const FlashArgs 
   auto rows_in = [&](__nv_bfloat16* dst, int dld, const __nv_bfloat16* src, int row, int pieces, const RunRows& rr, int v0, bool one_piece) {
     int y = lane / pieces, c = lane - y * pieces;
     const int dy = 32 / pieces, dc = 32 - dy * pieces;
-    if (one_piece) {
+    if (EXACT && one_piece) {   // 2 DT pieces: whole rows at a time
+      constexpr int P = 2 * DT, DY = 32 / P;
+      const __nv_bfloat16* s0 = src + (size_t)rr.row(v0) * row + (size_t)(uint32_t)(lane / P * row) + (lane % P) * 8;
+      uint32_t d0 = smem_addr(dst + lane / P * (16 * DT + 8) + (lane % P) * 8);
+      const int64_t step = (int64_t)DY * row;
+#pragma unroll
+      for (int i = 0; i < P; ++i) {
+        cp16(d0 + (uint32_t)(i * DY * (16 * DT + 8) * 2), s0);
+        s0 += step;
+      }
+    } else if (one_piece) {
       const __nv_bfloat16* s0 = src + (size_t)rr.row(v0) * row;
       for (int i = 0; i < pieces; ++i) {
         cp16z(dst + y * dld + c * 8, s0 + (size_t)(uint32_t)(y * row) + c * 8, true);
@@ -407,13 +427,14 @@ __global__ void __launch_bounds__(kThreads) flash_decode_kernel(const FlashArgs 
     for (int x = 0; x < 2; ++x)
 #pragma unroll
       for (int i = 0; i < 4; ++i) d[x][i] = 0.f;
+    const uint32_t k_at = smem_addr(k + (lane & 15) * ld + (lane >> 4) * 8), k_half = (uint32_t)ld * 32;
 #pragma unroll
     for (int ks = 0; ks < DT; ++ks) {
-      if (ks * 16 >= a.dpad) break;
+      if (!EXACT && ks * 16 >= a.dpad) break;
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
         uint32_t ka[4];
-        ldm4(ka, k + (x * 16 + (lane & 15)) * ld + ks * 16 + (lane >> 4) * 8);
+        ldm4(ka, k_at + (uint32_t)x * k_half + (uint32_t)(ks * 32));
         mma16816(d[x], ka, qb[ks][0], qb[ks][1]);
       }
     }
@@ -470,11 +491,12 @@ __global__ void __launch_bounds__(kThreads) flash_decode_kernel(const FlashArgs 
         hi[z] = transposed(p);
         rest[z] = transposed(pack2(w0 - __uint_as_float(p << 16), w1 - __uint_as_float(p & 0xFFFF0000u)));
       }
+      const uint32_t v_at = smem_addr(v + (x * 16 + (lane & 7) + (lane >> 4) * 8) * vld + ((lane >> 3) & 1) * 8);
 #pragma unroll
       for (int n = 0; n < DT; ++n) {
-        if (n * 16 >= a.vpad) break;
+        if (!EXACT && n * 16 >= a.vpad) break;
         uint32_t va[4];   // 16 columns x 16 keys out of [key][column]
-        ldm4t(va, v + (x * 16 + (lane & 7) + (lane >> 4) * 8) * vld + n * 16 + ((lane >> 3) & 1) * 8);
+        ldm4t(va, v_at + (uint32_t)(n * 32));
         mma16816(acc[n], va, hi[0], hi[1]);
         mma16816(acc[n], va, rest[0], rest[1]);
       }
@@ -737,7 +759,10 @@ tb_status launch_flash_attention(Precision p, const FlashArgs& a, cudaStream_t s
     if (splits > a.part_slots / ((int64_t)rows * a.heads)) splits = a.part_slots / ((int64_t)rows * a.heads);
     sd.splits = splits < 1 ? 1 : (int)splits;
     const int most = a.dpad > a.vpad ? a.dpad : a.vpad;
-    FlashKernel dec = most <= 64 ? flash_decode_kernel<4> : (most <= 128 ? flash_decode_kernel<8> : flash_decode_kernel<16>);
+    const bool exact = a.dpad == a.vpad && (most == 64 || most == 128 || most == 256);
+    FlashKernel dec = most <= 64 ? (exact ? flash_decode_kernel<4, true> : flash_decode_kernel<4, false>)
+                      : most <= 128 ? (exact ? flash_decode_kernel<8, true> : flash_decode_kernel<8, false>)
+                                    : (exact ? flash_decode_kernel<16, true> : flash_decode_kernel<16, false>);
     TB_TRY(launch_kernel(dec, dim3((unsigned)sd.splits, (unsigned)a.kv_heads, (unsigned)rows), dim3((unsigned)warps * 32), per * warps, st, a.pdl, 1, a, sd));
     return merge(sd.splits);
   }

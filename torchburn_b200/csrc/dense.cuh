@@ -317,6 +317,7 @@ int64_t flash_part_slots(int64_t rows, int64_t heads);   // what the splits a st
 tb_status launch_flash_attention(Precision p, const FlashArgs& a, cudaStream_t st, int* launches);
 bool flash_tc5_fits(int dpad, int vdim);                 // sizes that the tcgen05 kernel for portions takes
 int flash_fault_flag();
+int flash_latent_fault_flag();
 
 // ---- windowed attention with mixed heads (window_attention.cu) -----------------------------------
 struct WindowAttnArgs {

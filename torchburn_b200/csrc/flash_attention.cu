@@ -13,7 +13,8 @@
 // memory as two bf16 pieces (the second one what the rounding of the first left: 16 mantissa bits), then the values
 // with the warps side by side over the value columns.  CTAs that share a block's keys leave (max, sum, unnormalised
 // output) and a last kernel merges them in a fixed order.
-// Portions of one sequence take the tcgen05 kernel of flash_tc5.cu where its tiles fit.
+// Portions of one sequence take the tcgen05 kernel of flash_tc5.cu where its tiles fit, decode steps over latents that of
+// flash_latent.cu.
 // fp32, and sizes beyond the tiles (flash_simple_kernel): a CTA per row and up to four heads, fp32 products.
 #include "dense.cuh"
 #include "flash_attention.cuh"
@@ -45,17 +46,6 @@ __device__ __forceinline__ void mma16816(float (&d)[4], const uint32_t (&a)[4], 
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-
-template <bool BF16>
-__device__ __forceinline__ void store_column(const FlashArgs& a, int row, int h, int c, float v) {
-  if (!a.out_per_head) {
-    act_store1<BF16>(a.out, row, h * a.vdim + c, v);
-    return;
-  }
-  ActOperand o = a.out;
-  o.data = static_cast<unsigned char*>(o.data) + (size_t)h * o.mp * o.kp * (BF16 ? 2 : 4);
-  act_store1<BF16>(o, row, c, v);
 }
 
 // First positions that a row sees in its own run.
@@ -294,12 +284,12 @@ __global__ void __launch_bounds__(kThreads, NV <= 8 ? 2 : 1) flash_mma_kernel(co
       for (int i = 0; i < 2; ++i) {
         const int c = col0 + n * 8 + (lane & 3) * 2 + i;
         if (c >= a.vdim) continue;
-        if (whole) store_column<true>(a, qrow[e], head[e], c, acc[n][2 * e + i] * f);
+        if (whole) flash_store_column<true>(a, qrow[e], head[e], c, acc[n][2 * e + i] * f);
         else dst[c] = acc[n][2 * e + i];
       }
     }
     if (whole && wc == 0)
-      for (int c = a.vdim + (lane & 3); c < flash_column_limit(a, head[e]); c += 4) store_column<true>(a, qrow[e], head[e], c, 0.f);
+      for (int c = a.vdim + (lane & 3); c < flash_column_limit(a, head[e]); c += 4) flash_store_column<true>(a, qrow[e], head[e], c, 0.f);
   }
 }
 
@@ -550,7 +540,7 @@ __global__ void __launch_bounds__(kThreads) flash_decode_kernel(const FlashArgs 
           const float x = s_ml[w * NH + h].x;
           if (x != -INFINITY) o = fmaf(s_o[(w * NH + h) * old + c], exp2f(x - mm), o);
         }
-      if (whole) store_column<true>(a, r, head, c, o * f);
+      if (whole) flash_store_column<true>(a, r, head, c, o * f);
       else a.parts[part * a.vdim + c] = o;
     }
   }
@@ -595,7 +585,7 @@ __global__ void __launch_bounds__(128) flash_merge_kernel(const FlashArgs a, con
     if (a.gate) f *= a.gate[at];
     v *= f;
   }
-  store_column<true>(a, r, h, c, v);
+  flash_store_column<true>(a, r, h, c, v);
 }
 
 __device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
@@ -695,7 +685,7 @@ __global__ void __launch_bounds__(kThreads) flash_simple_kernel(const FlashArgs 
     float f = s_l[h] > 0.f ? 1.f / s_l[h] : 0.f;
     if (a.gate) f *= a.gate[(size_t)r * a.heads + h0 + h];
     for (int c = tid; c < flash_column_limit(a, h0 + h); c += kThreads)
-      store_column<sizeof(T) == 2>(a, r, h0 + h, c, c < a.vdim ? s_o[h * a.vdim + c] * f : 0.f);
+      flash_store_column<sizeof(T) == 2>(a, r, h0 + h, c, c < a.vdim ? s_o[h * a.vdim + c] * f : 0.f);
   }
 }
 
@@ -744,6 +734,11 @@ tb_status launch_flash_attention(Precision p, const FlashArgs& a, cudaStream_t s
   if (flash_tc5_supported(a)) {
     int splits = 1;
     TB_TRY(launch_flash_tc5(a, st, &splits));
+    return merge(splits);
+  }
+  if (flash_latent_supported(a)) {
+    int splits = 1;
+    TB_TRY(launch_flash_latent(a, st, &splits));
     return merge(splits);
   }
   if (!a.one_sequence && !a.values_in_keys && gq <= kDecodeHeads && a.dpad <= 256 && a.vpad <= 256) {

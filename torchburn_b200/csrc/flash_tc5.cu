@@ -18,11 +18,10 @@
 #include <climits>
 #include <cstring>
 
-#include <cuda.h>
-
 #include "dense.cuh"
 #include "flash_attention.cuh"
 #include "tc5.cuh"
+#include "tma_panel.cuh"
 #include "window_attention.cuh"
 
 namespace tb {
@@ -84,12 +83,6 @@ __device__ __forceinline__ void mma_bf16_ts(uint32_t d_tmem, uint32_t a_tmem, ui
       : "memory");
 }
 
-// A panel of 64 columns x 128 rows of a row-major matrix, from (x, y) on; x on a 16-byte boundary.
-__device__ __forceinline__ void tma_panel(uint32_t dst, const CUtensorMap* map, int x, int y, uint64_t* bar) {
-  asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst), "l"(map), "r"(x),
-               "r"(y), "r"(smem_u32(bar))
-               : "memory");
-}
 struct FlashMaps {
   CUtensorMap k, rest, v;
 };
@@ -232,9 +225,9 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
             mbar_expect_tx(&k_full[w], (uint32_t)kbytes);
             for (int c = 0; c < kpanels; ++c) {
               const uint32_t dst = k_at + (uint32_t)(w * kbytes + c * kPanel);
-              if (c >= kfirst) tma_panel(dst, &maps.rest, a.rest_col + (c - kfirst) * 64, crow, &k_full[w]);
-              else if (a.key_rows) tma_panel(dst, &maps.k, kv * a.key_cols + c * 64, k0 - a.key_base, &k_full[w]);
-              else tma_panel(dst, &maps.k, kv * a.dpad + c * 64, crow, &k_full[w]);
+              if (c >= kfirst) tma_panel(dst, &maps.rest, a.rest_col + (c - kfirst) * 64, crow, smem_u32(&k_full[w]));
+              else if (a.key_rows) tma_panel(dst, &maps.k, kv * a.key_cols + c * 64, k0 - a.key_base, smem_u32(&k_full[w]));
+              else tma_panel(dst, &maps.k, kv * a.dpad + c * 64, crow, smem_u32(&k_full[w]));
             }
           }
           for (int w = 0; ok && w < 2; ++w) {
@@ -244,7 +237,7 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
             v_issued[w] = j + 1;
             mbar_expect_tx(&v_full[w], (uint32_t)vbytes);
             for (int c = 0; c < vpanels; ++c)
-              tma_panel(v_at + (uint32_t)(w * vbytes + c * kPanel), &maps.v, kv * (a.key_rows ? a.vdim : a.vpad) + c * 64, a.key_rows ? k0 - a.key_base : crow, &v_full[w]);
+              tma_panel(v_at + (uint32_t)(w * vbytes + c * kPanel), &maps.v, kv * (a.key_rows ? a.vdim : a.vpad) + c * 64, a.key_rows ? k0 - a.key_base : crow, smem_u32(&v_full[w]));
           }
         }
         if (!ok) {   // copies in flight land before the shared memory is given back: the last one issued per slot
@@ -522,23 +515,6 @@ size_t tc5_bytes(int dpad, int vpad) {
   return (tiles > out ? tiles : out) + 1024;
 }
 
-// Panels of 64 columns x 128 rows of a row-major bf16 matrix, 128-byte swizzle, zeros outside.
-bool panel_map(CUtensorMap* map, const void* base, int64_t cols, int64_t rows, int64_t stride) {
-  using Encode = CUresult (*)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
-                              const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-  static Encode encode = [] {
-    void* fn = nullptr;
-    cudaDriverEntryPointQueryResult found;
-    if (cudaGetDriverEntryPointByVersion("cuTensorMapEncodeTiled", &fn, 12000, cudaEnableDefault, &found) != cudaSuccess || found != cudaDriverEntryPointSuccess) fn = nullptr;
-    return reinterpret_cast<Encode>(fn);
-  }();
-  if (!encode || rows < 1 || rows > INT_MAX) return false;
-  const cuuint64_t dims[2] = {(cuuint64_t)cols, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)stride * 2};
-  const cuuint32_t box[2] = {64, (cuuint32_t)kKeys}, steps[2] = {1, 1};
-  return encode(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, steps, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
 }  // namespace
 
 int flash_fault_flag() {
@@ -578,12 +554,12 @@ tb_status launch_flash_tc5(const FlashArgs& a, cudaStream_t st, int* splits_out)
   bool tma = a.geom.ring % kKeys == 0 && a.geom.keep == 0 && a.cache_slots > 0;
   if (a.key_rows) {
     const int64_t n = a.key_count;
-    tma = tma && a.key_cols % 64 == 0 && a.key_base % kKeys == 0 && panel_map(&maps.k, a.key_rows, (int64_t)a.kv_heads * a.key_cols, n, a.row_stride) &&
-          panel_map(&maps.v, a.value_rows, (int64_t)a.kv_heads * a.vdim, n, a.row_stride) &&
-          panel_map(&maps.rest, a.k_cache, a.cache_row, a.cache_slots * a.geom.rows, a.cache_row);
+    tma = tma && a.key_cols % 64 == 0 && a.key_base % kKeys == 0 && tma_panel_map(&maps.k, a.key_rows, (int64_t)a.kv_heads * a.key_cols, n, a.row_stride, kKeys) &&
+          tma_panel_map(&maps.v, a.value_rows, (int64_t)a.kv_heads * a.vdim, n, a.row_stride, kKeys) &&
+          tma_panel_map(&maps.rest, a.k_cache, a.cache_row, a.cache_slots * a.geom.rows, a.cache_row, kKeys);
   } else {
     const int64_t n = (int64_t)a.cache_slots * a.geom.rows, kw = (int64_t)a.kv_heads * a.dpad, vw = (int64_t)a.kv_heads * a.vpad;
-    tma = tma && panel_map(&maps.k, a.k_cache, kw, n, kw) && panel_map(&maps.v, a.v_cache, vw, n, vw);
+    tma = tma && tma_panel_map(&maps.k, a.k_cache, kw, n, kw, kKeys) && tma_panel_map(&maps.v, a.v_cache, vw, n, vw, kKeys);
   }
   using Kernel = void (*)(FlashArgs, FlashShape, FlashMaps);
   static const Kernel kernels[3][2] = {{flash_tc5_kernel<0, false>, flash_tc5_kernel<0, true>},

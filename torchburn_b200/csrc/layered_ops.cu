@@ -476,7 +476,7 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
 // V4: sizes are multiples of four, a lane takes four columns at a time; else one.
 template <typename T, bool V4>
 __global__ void __launch_bounds__(kThreads) heads_prep_kernel(const HeadsPrepArgs a) {
-  constexpr int KEEP = 8;                  // values a lane keeps between the norm's two passes
+  [[maybe_unused]] constexpr int KEEP = 8;                  // values a lane keeps between the norm's two passes
   const int lane = threadIdx.x & 31, r = (int)blockIdx.y;
   int u = (int)blockIdx.x * (kThreads / 32) + (threadIdx.x >> 5);
   grid_dep_launch();
@@ -513,12 +513,12 @@ __global__ void __launch_bounds__(kThreads) heads_prep_kernel(const HeadsPrepArg
     if (!is_q && pos < 0) return;
     if constexpr (V4) {
       for (int c = lane * 4, e = 0; c < a.dim; c += 128, ++e) store4(dst + c, scale4(e == 0 ? w4[0] : (e == 1 ? w4[1] : sum_partials(a.y, r, col + c)), inv));
-      return;
-    }
+    } else {
 #pragma unroll
-    for (int j = 0; j < KEEP; ++j)
-      if (lane + 32 * j < a.dim) dst[lane + 32 * j] = (T)(v[j] * inv);
-    for (int c = lane + 32 * KEEP; c < a.dim; c += 32) dst[c] = (T)(sum_column(a.y, r, col + c) * inv);
+      for (int j = 0; j < KEEP; ++j)
+        if (lane + 32 * j < a.dim) dst[lane + 32 * j] = (T)(v[j] * inv);
+      for (int c = lane + 32 * KEEP; c < a.dim; c += 32) dst[c] = (T)(sum_column(a.y, r, col + c) * inv);
+    }
     return;
   }
   u -= a.heads + a.kv_heads;
@@ -532,13 +532,13 @@ __global__ void __launch_bounds__(kThreads) heads_prep_kernel(const HeadsPrepArg
         else if (first) v = fma4(f4(a.mix), ld4(first + c), scale4(v, 1.f - a.mix));
         if (pos >= 0) store4(dst + c, v);
       }
-      return;
-    }
-    for (int c = lane; c < a.vdim; c += 32) {
-      float v = sum_column(a.y, r, a.v_off + u * a.vdim + c);
-      if (first && a.keep_first_values) first[c] = v;
-      else if (first) v = fmaf(a.mix, first[c], (1.f - a.mix) * v);
-      if (pos >= 0) dst[c] = (T)v;
+    } else {
+      for (int c = lane; c < a.vdim; c += 32) {
+        float v = sum_column(a.y, r, a.v_off + u * a.vdim + c);
+        if (first && a.keep_first_values) first[c] = v;
+        else if (first) v = fmaf(a.mix, first[c], (1.f - a.mix) * v);
+        if (pos >= 0) dst[c] = (T)v;
+      }
     }
     return;
   }
@@ -611,19 +611,19 @@ __global__ void __launch_bounds__(kThreads) latent_query_kernel(const LatentQuer
       store4(q + c, make_float4(rotated(a.table, a.rot_dims, pos, c, v.x, v.y), rotated(a.table, a.rot_dims, pos, c + 1, v.y, v.x),
                                 rotated(a.table, a.rot_dims, pos, c + 2, v.z, v.w), rotated(a.table, a.rot_dims, pos, c + 3, v.w, v.z)));
     }
-    return;
-  }
-  if (a.out.data) {
-    ActOperand out = a.out;
-    out.data = static_cast<unsigned char*>(out.data) + (size_t)h * out.mp * out.kp * sizeof(T);
-    for (int c = lane; c < out.kp; c += 32) act_store1<sizeof(T) == 2>(out, r, c, c < a.dim ? sum_column(a.y, r, col + c) : 0.f);
   } else {
-    for (int c = lane; c < a.dim; c += 32) q[c] = (T)sum_column(a.y, r, col + c);
-  }
-  q += a.rot_at;
-  for (int c = lane; c < a.rot_dim; c += 32) {
-    const float own = sum_column(a.y, r, col + a.dim + c), other = c < a.rot_dims ? sum_column(a.y, r, col + a.dim + (c ^ 1)) : 0.f;
-    q[c] = (T)rotated(a.table, a.rot_dims, pos, c, own, other);
+    if (a.out.data) {
+      ActOperand out = a.out;
+      out.data = static_cast<unsigned char*>(out.data) + (size_t)h * out.mp * out.kp * sizeof(T);
+      for (int c = lane; c < out.kp; c += 32) act_store1<sizeof(T) == 2>(out, r, c, c < a.dim ? sum_column(a.y, r, col + c) : 0.f);
+    } else {
+      for (int c = lane; c < a.dim; c += 32) q[c] = (T)sum_column(a.y, r, col + c);
+    }
+    q += a.rot_at;
+    for (int c = lane; c < a.rot_dim; c += 32) {
+      const float own = sum_column(a.y, r, col + a.dim + c), other = c < a.rot_dims ? sum_column(a.y, r, col + a.dim + (c ^ 1)) : 0.f;
+      q[c] = (T)rotated(a.table, a.rot_dims, pos, c, own, other);
+    }
   }
 }
 

@@ -578,9 +578,8 @@ __global__ void __launch_bounds__(128) flash_merge_kernel(const FlashArgs a, con
   float v = 0.f;
   if (c < a.vdim) {
     const float* p = a.parts + at * a.vdim + c;
-#pragma unroll 8
-    for (int z = 0; z < splits; ++z)
-      if (s_w[z] > 0.f) v = fmaf(s_w[z], p[(size_t)z * stride * a.vdim], v);   // a share that saw nothing left zeros or nothing
+#pragma unroll 16
+    for (int z = 0; z < splits; ++z) v = fmaf(s_w[z], p[(size_t)z * stride * a.vdim], v);   // a share that saw nothing left zeros
     float f = l > 0.f ? 1.f / l : 0.f;
     if (a.gate) f *= a.gate[at];
     v *= f;

@@ -7,10 +7,11 @@
 //   S^T [64 keys, heads]       = K Q^T      K as it lies in the cache, K-major
 //   O^T [value columns, heads] += V^T P^T   the same tile read MN-major: V is K's first columns; P^T from shared memory
 //
-// 64 keys per tile (the upper 64 rows of the first product are whatever lies behind the tile, and nobody reads them), tiles
-// by TMA, swizzled, two to four of them in flight.  Two warps hold a key per lane: maxima over the lanes by redux, weights as two
-// bf16 pieces (the second one what the rounding of the first left).  The output is rescaled, by all four warps,
-// only when a maximum has grown by more than 8 powers of two.  CTAs that share a row's keys leave parts for the merge.
+// 64 keys per tile, tiles by TMA, swizzled, two to four of them in flight.  Four warps hold the scores of 16 keys each (the way
+// an MMA of 64 rows leaves them).  Weights are two bf16 pieces, the second one what the rounding of the first left; the
+// pieces of the heads are the columns of one MMA, and their outputs are added at the end.  The output is rescaled only
+// when a maximum has grown by more than 8 powers of two.  One thread issues the MMAs, scores or outputs, whatever is
+// ready.  CTAs that share a row's keys leave parts for the merge.
 #include <climits>
 
 #include "flash_attention.cuh"
@@ -28,7 +29,7 @@ constexpr int kKeys = 64;            // keys per tile
 constexpr int kPanel = kKeys * 128;  // 64 columns of a tile
 constexpr int kThreads = 192;        // four softmax / output warps, one for TMA, one for the MMAs
 constexpr int kStagesMax = 4;
-constexpr int kColumns = 256;        // of tensor memory
+constexpr int kColumns = 512;        // of tensor memory
 constexpr float kLog2E = 1.44269504f;
 constexpr float kGrow = 8.f;
 
@@ -39,10 +40,22 @@ __device__ __forceinline__ float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
-__device__ __forceinline__ float warp_max(float x) {
-  float y;
-  asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(y) : "f"(x));
-  return y;
+// The 8 x 8 matrix of 16-bit elements that a warp holds (row lane / 4, columns 2 (lane & 3) and the next), transposed.
+__device__ __forceinline__ uint32_t transposed(uint32_t v) {
+  uint32_t r;
+  asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
+  return r;
+}
+__device__ __forceinline__ uint32_t pack2(float x, float y) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(x, y);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+// 16 lanes x 8 columns over the warp: lane / 4 (v0, v1) and 8 lanes on (v2, v3), columns 2 (lane & 3) and the next (no wait)
+__device__ __forceinline__ void tmem_ld_tile(uint32_t at, float (&v)[4]) {
+  uint32_t r[4];
+  asm volatile("tcgen05.ld.sync.aligned.16x256b.x1.b32 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at) : "memory");
+#pragma unroll
+  for (int x = 0; x < 4; ++x) v[x] = __uint_as_float(r[x]);
 }
 // NH columns of this thread's lane
 template <int NH>
@@ -74,7 +87,7 @@ __global__ void __launch_bounds__(kThreads, 1) flash_latent_kernel(const FlashAr
   __shared__ __align__(8) uint64_t full[kStagesMax], empty[kStagesMax], s_ready[2], p_ready[2], pv_done[2], q_full, finished;
   __shared__ uint32_t s_tmem;
   __shared__ int s_abort, s_grown, s_bad;
-  __shared__ float s_max[2][NH], s_ref[NH], s_alpha[NH], s_l[2][NH];
+  __shared__ __align__(16) float s_max[4][NH], s_ref[NH], s_alpha[NH], s_l[4][NH];
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   unsigned char* smem = reinterpret_cast<unsigned char*>((reinterpret_cast<uintptr_t>(s_raw) + 1023) & ~(uintptr_t)1023);
   const uint32_t k_at = smem_u32(smem), q_at = k_at + (uint32_t)(sh.stages * sh.stage_bytes), p_at = q_at + (uint32_t)(sh.panels * NH * 128);
@@ -129,35 +142,50 @@ __global__ void __launch_bounds__(kThreads, 1) flash_latent_kernel(const FlashAr
     }
   } else if (warp == 5) {
     if (lane == 0) {   // ---- MMA issue ----
-      constexpr uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(NH >> 3) << 17) | (8u << 24);
+      // scores: 64 rows, row k in lane k % 16 + 32 (k / 16); output: 128 rows, MN-major
+      constexpr uint32_t shape = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(NH >> 3) << 17);
+      constexpr uint32_t idesc_s = shape | (4u << 24), idesc_o = (shape + ((uint32_t)(NH >> 3) << 17)) | (1u << 15) | (8u << 24);   // both pieces
       const int ksteps = a.dpad >> 4;
       bool ok = mbar_wait(&q_full, 0u, &s_abort, &g_latent_fault);
-      for (int i = 0; ok && i <= n; ++i) {
-        if (i < n) {
-          const int s = i % sh.stages;
-          if (!(ok = mbar_wait(&full[s], (uint32_t)(i / sh.stages) & 1u, &s_abort, &g_latent_fault))) break;
-          tc_fence_after();
-          const uint32_t k_lo = ((k_at + (uint32_t)(s * sh.stage_bytes)) >> 4) | (1u << 16), q_lo = (q_at >> 4) | (1u << 16);
-          for (int ks = 0; ks < ksteps; ++ks)
-            mma_bf16_ss(tmem + (uint32_t)((i & 1) * NH), k_lo + (uint32_t)((ks >> 2) * (kPanel >> 4) + (ks & 3) * 2),
-                        q_lo + (uint32_t)((ks >> 2) * (NH * 8) + (ks & 3) * 2), idesc, ks > 0 ? 1u : 0u);
-          mma_commit(&s_ready[i & 1]);
-        }
-        if (i > 0) {
-          const int t = i - 1, s = t % sh.stages;
-          if (!(ok = mbar_wait(&p_ready[t & 1], (uint32_t)(t >> 1) & 1u, &s_abort, &g_latent_fault))) break;
+      int scored = 0, summed = 0;
+      long long idle = 0;
+      while (ok && summed < n) {   // whatever is ready first: the output of a tile, or the scores of one up to two ahead
+        bool did = false;
+        if (summed < scored && mbar_ready(&p_ready[summed & 1], (uint32_t)(summed >> 1) & 1u)) {
+          const int t = summed++, s = t % sh.stages;
           tc_fence_after();
           const uint32_t v_lo = ((k_at + (uint32_t)(s * sh.stage_bytes)) >> 4) | ((uint32_t)(kPanel >> 4) << 16);
           const uint32_t p_lo = ((p_at + (uint32_t)((t & 1) * 2 * NH * 128)) >> 4) | (1u << 16);
           for (int mt = 0; mt < sh.mtiles; ++mt)
 #pragma unroll
             for (int kk = 0; kk < kKeys / 16; ++kk)
-#pragma unroll
-              for (int piece = 0; piece < 2; ++piece)
-                mma_bf16_ss(o_at + (uint32_t)(mt * NH), v_lo + (uint32_t)(mt * 2 * (kPanel >> 4) + kk * 128), p_lo + (uint32_t)(piece * NH * 8 + kk * 2),
-                            idesc | (1u << 15), (t > 0 || kk > 0 || piece > 0) ? 1u : 0u);
+              mma_bf16_ss(o_at + (uint32_t)(mt * 2 * NH), v_lo + (uint32_t)(mt * 2 * (kPanel >> 4) + kk * 128), p_lo + (uint32_t)(kk * 2), idesc_o,
+                          (t > 0 || kk > 0) ? 1u : 0u);
           mma_commit(&empty[s]);
           mma_commit(&pv_done[t & 1]);
+          did = true;
+        }
+        if (scored < n && scored < summed + 2 && mbar_ready(&full[scored % sh.stages], (uint32_t)(scored / sh.stages) & 1u)) {
+          const int i = scored++, s = i % sh.stages;
+          tc_fence_after();
+          const uint32_t k_lo = ((k_at + (uint32_t)(s * sh.stage_bytes)) >> 4) | (1u << 16), q_lo = (q_at >> 4) | (1u << 16);
+#pragma unroll 4
+          for (int ks = 0; ks < ksteps; ++ks)
+            mma_bf16_ss(tmem + (uint32_t)((i & 1) * NH), k_lo + (uint32_t)((ks >> 2) * (kPanel >> 4) + (ks & 3) * 2),
+                        q_lo + (uint32_t)((ks >> 2) * (NH * 8) + (ks & 3) * 2), idesc_s, ks > 0 ? 1u : 0u);
+          mma_commit(&s_ready[i & 1]);
+          did = true;
+        }
+        if (did) {
+          idle = 0;
+        } else if (*reinterpret_cast<volatile int*>(&s_abort)) {
+          ok = false;
+        } else if (idle == 0) {
+          idle = clock64();
+        } else if (clock64() - idle > kWaitCycles) {
+          s_abort = 1;
+          atomicExch(&g_latent_fault, 1);
+          ok = false;
         }
       }
       mma_commit(&finished);
@@ -182,36 +210,50 @@ __global__ void __launch_bounds__(kThreads, 1) flash_latent_kernel(const FlashAr
     }
     const uint32_t lanes = (uint32_t)(warp * 32) << 16;
     const float scale = a.scale * kLog2E;
-    const int key = tid;                 // of the tile, in warps 0 and 1
-    float m = -INFINITY, l[NH];          // m: thread h of warp 0, head h;  l: this key's share of every head's sum
+    constexpr int NB = NH / 8;           // blocks of eight heads
+    // this lane's keys of a tile: 16 warp + lane / 4 and 8 on; heads 8 i + 2 (lane & 3) and the next
+    const int key = warp * 16 + (lane >> 2), col = (lane & 3) * 2;
+    float m = -INFINITY, l[NB][2];       // m: thread h of warp 0, head h;  l: these keys' share of the heads' sums
 #pragma unroll
-    for (int h = 0; h < NH; ++h) l[h] = 0.f;
+    for (int i = 0; i < NB; ++i) l[i][0] = l[i][1] = 0.f;
     bool ok = true;
     for (int t = 0; t < n; ++t) {
       ok = mbar_wait(&s_ready[t & 1], (uint32_t)(t >> 1) & 1u, &s_abort, &g_latent_fault);
       ok = __all_sync(0xffffffffu, ok);
       if (!ok) s_bad = 1;
-      float s[NH];
-      if (ok && warp < 2) {
+      float s[NB][4];
+      if (ok) {
         tc_fence_after();
-        tmem_load<NH>(tmem + lanes + (uint32_t)((t & 1) * NH), s);
-        const int p = begin + (t0 + t) * kKeys + key;
-        const bool seen = p >= lo && p <= pos;
-        float mine = -INFINITY;
 #pragma unroll
-        for (int h = 0; h < NH; ++h) {
-          s[h] = seen ? s[h] * scale : -INFINITY;
-          const float x = warp_max(s[h]);
-          if (lane == h) mine = x;
-        }
-        if (lane < NH) s_max[warp][lane] = mine;
+        for (int i = 0; i < NB; ++i) tmem_ld_tile(tmem + lanes + (uint32_t)((t & 1) * NH + i * 8), s[i]);
+        asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+        const int p = begin + (t0 + t) * kKeys + key;
+        const bool seen[2] = {p >= lo && p <= pos, p + 8 >= lo && p + 8 <= pos};
+        float mx[NB][2];
+#pragma unroll
+        for (int i = 0; i < NB; ++i)
+#pragma unroll
+          for (int y = 0; y < 2; ++y) {
+#pragma unroll
+            for (int z = 0; z < 2; ++z) s[i][2 * z + y] = seen[z] ? s[i][2 * z + y] * scale : -INFINITY;
+            mx[i][y] = fmaxf(s[i][y], s[i][2 + y]);
+          }
+#pragma unroll
+        for (int o = 16; o > 2; o >>= 1)
+#pragma unroll
+          for (int i = 0; i < NB; ++i)
+#pragma unroll
+            for (int y = 0; y < 2; ++y) mx[i][y] = fmaxf(mx[i][y], __shfl_xor_sync(0xffffffffu, mx[i][y], o));
+        if (lane < 4)
+#pragma unroll
+          for (int i = 0; i < NB; ++i) *reinterpret_cast<float2*>(&s_max[warp][i * 8 + col]) = make_float2(mx[i][0], mx[i][1]);
       }
       asm volatile("bar.sync 1, 128;" ::: "memory");
       const bool bad = *reinterpret_cast<volatile int*>(&s_bad) != 0;   // the same for all four warps: written in front of this barrier only
       if (warp == 0) {
         bool grow = false;
         if (lane < NH) {
-          const float mx = fmaxf(s_max[0][lane], s_max[1][lane]);
+          const float mx = fmaxf(fmaxf(s_max[0][lane], s_max[1][lane]), fmaxf(s_max[2][lane], s_max[3][lane]));
           grow = mx > m + kGrow || (m == -INFINITY && mx != -INFINITY);
           const float m1 = grow ? fmaxf(m, mx) : m;
           s_alpha[lane] = m == -INFINITY ? 0.f : ex2(m - m1);
@@ -231,30 +273,39 @@ __global__ void __launch_bounds__(kThreads, 1) flash_latent_kernel(const FlashAr
           mbar_wait(&pv_done[(t - 1) & 1], (uint32_t)((t - 1) >> 1) & 1u, &s_abort, &g_latent_fault);
           __syncwarp();
           tc_fence_after();
-          for (int mt = 0; mt < sh.mtiles; ++mt) {
+          for (int x = 0; x < 2 * sh.mtiles; ++x) {   // both pieces
             float o[NH];
-            tmem_load<NH>(o_at + lanes + (uint32_t)(mt * NH), o);
+            tmem_load<NH>(o_at + lanes + (uint32_t)(x * NH), o);
 #pragma unroll
             for (int h = 0; h < NH; ++h) o[h] *= s_alpha[h];
 #pragma unroll
-            for (int h = 0; h < NH; h += 8) tmem_st8(o_at + lanes + (uint32_t)(mt * NH + h), o + h);
+            for (int h = 0; h < NH; h += 8) tmem_st8(o_at + lanes + (uint32_t)(x * NH + h), o + h);
           }
           asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory");
         }
 #pragma unroll
-        for (int h = 0; h < NH; ++h) l[h] *= s_alpha[h];
+        for (int i = 0; i < NB; ++i)
+#pragma unroll
+          for (int y = 0; y < 2; ++y) l[i][y] *= s_alpha[i * 8 + col + y];
       }
       if (t > 1) mbar_wait(&pv_done[t & 1], (uint32_t)((t - 2) >> 1) & 1u, &s_abort, &g_latent_fault);   // the weights' place is free
-      if (warp < 2) {
-        unsigned char* p = smem + (p_at - k_at) + (size_t)(t & 1) * 2 * NH * 128 + (key & 7) * 2;
+      {
+        // [key][head] -> [head][key]: this lane then has head 8 i + lane / 4, keys 2 (lane & 3) and the next of each block of eight
+        unsigned char* p = smem + (p_at - k_at) + (size_t)(t & 1) * 2 * NH * 128 + (lane >> 2) * 128 + (lane & 3) * 4;
 #pragma unroll
-        for (int h = 0; h < NH; ++h) {
-          const float w = ex2(s[h] - s_ref[h]);
-          l[h] += w;
-          const __nv_bfloat16 hi = __float2bfloat16_rn(w);
-          unsigned char* at = p + h * 128 + (((key >> 3) ^ (h & 7)) << 4);
-          *reinterpret_cast<__nv_bfloat16*>(at) = hi;
-          *reinterpret_cast<__nv_bfloat16*>(at + NH * 128) = __float2bfloat16_rn(w - __bfloat162float(hi));
+        for (int i = 0; i < NB; ++i) {
+          const float2 ref = *reinterpret_cast<const float2*>(&s_ref[i * 8 + col]);
+#pragma unroll
+          for (int z = 0; z < 2; ++z) {
+            const float w0 = ex2(s[i][2 * z] - ref.x), w1 = ex2(s[i][2 * z + 1] - ref.y);
+            l[i][0] += w0;
+            l[i][1] += w1;
+            const uint32_t hi = pack2(w0, w1);
+            const uint32_t rest = pack2(w0 - __uint_as_float(hi << 16), w1 - __uint_as_float(hi & 0xFFFF0000u));
+            unsigned char* at = p + i * 1024 + (((warp * 2 + z) ^ (lane >> 2)) << 4);
+            *reinterpret_cast<uint32_t*>(at) = transposed(hi);
+            *reinterpret_cast<uint32_t*>(at + NH * 128) = transposed(rest);
+          }
         }
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
       }
@@ -264,38 +315,54 @@ __global__ void __launch_bounds__(kThreads, 1) flash_latent_kernel(const FlashAr
     if (ok && n > 0) mbar_wait(&pv_done[(n - 1) & 1], (uint32_t)((n - 1) >> 1) & 1u, &s_abort, &g_latent_fault);
     __syncwarp();
     tc_fence_after();
-    if (warp < 2) {
-      float mine = 0.f;
 #pragma unroll
-      for (int h = 0; h < NH; ++h) {
-        float x = l[h];
+    for (int o = 16; o > 2; o >>= 1)
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) x += __shfl_xor_sync(0xffffffffu, x, o);
-        if (lane == h) mine = x;
-      }
-      if (lane < NH) s_l[warp][lane] = mine;
-    }
+      for (int i = 0; i < NB; ++i)
+#pragma unroll
+        for (int y = 0; y < 2; ++y) l[i][y] += __shfl_xor_sync(0xffffffffu, l[i][y], o);
+    if (lane < 4)
+#pragma unroll
+      for (int i = 0; i < NB; ++i) *reinterpret_cast<float2*>(&s_l[warp][i * 8 + col]) = make_float2(l[i][0], l[i][1]);
     asm volatile("bar.sync 1, 128;" ::: "memory");
     const bool whole = sh.splits == 1;
-    if (!whole && warp == 0 && lane < nh) a.part_ml[((size_t)split * a.r.rows + r) * a.heads + h0 + lane] = make_float2(m, s_l[0][lane] + s_l[1][lane]);
-    for (int mt = 0; mt < sh.mtiles; ++mt) {
-      float o[NH];
-      if (n > 0) tmem_load<NH>(o_at + lanes + (uint32_t)(mt * NH), o);
-      const int c = mt * 128 + tid;
-#pragma unroll
-      for (int h = 0; h < NH; ++h) {
-        if (h >= nh) break;
-        const float sum = s_l[0][h] + s_l[1][h];
-        float v = n > 0 && sum > 0.f && c < a.vdim ? o[h] : 0.f;
-        if (!whole) {
-          if (c < a.vdim) a.parts[(((size_t)split * a.r.rows + r) * a.heads + h0 + h) * a.vdim + c] = v;
-          continue;
-        }
-        if (sum > 0.f) v /= sum;
-        if (a.gate) v *= a.gate[(size_t)r * a.heads + h0 + h];
-        if (c < flash_column_limit(a, h0 + h)) flash_store_column<true>(a, r, h0 + h, c, v);
+    if (warp == 0 && lane < NH) {
+      const float sum = (s_l[0][lane] + s_l[1][lane]) + (s_l[2][lane] + s_l[3][lane]);
+      float f = sum > 0.f ? 1.f : 0.f;
+      if (whole && sum > 0.f) {
+        f = 1.f / sum;
+        if (a.gate && lane < nh) f *= a.gate[(size_t)r * a.heads + h0 + lane];
       }
+      s_alpha[lane] = f;
+      if (!whole && lane < nh) a.part_ml[((size_t)split * a.r.rows + r) * a.heads + h0 + lane] = make_float2(m, sum);
+    }
+    asm volatile("bar.sync 1, 128;" ::: "memory");
+    float* parts = a.parts + (((size_t)split * a.r.rows + r) * a.heads + h0) * a.vdim + tid;
+    for (int mt = 0; mt < sh.mtiles; ++mt) {
+      const int c = mt * 128 + tid;
+      float o[NH];
+#pragma unroll
+      for (int h = 0; h < NH; ++h) o[h] = 0.f;
       __syncwarp();
+      if (n > 0) {
+        float rest[NH];
+        tmem_load<NH>(o_at + lanes + (uint32_t)(mt * 2 * NH), o);
+        tmem_load<NH>(o_at + lanes + (uint32_t)(mt * 2 * NH + NH), rest);
+#pragma unroll
+        for (int h = 0; h < NH; ++h) o[h] = c < a.vdim && s_alpha[h] > 0.f ? (o[h] + rest[h]) * s_alpha[h] : 0.f;
+      }
+      if (!whole) {
+        if (c < a.vdim) {
+          float* p = parts + mt * 128;
+#pragma unroll
+          for (int h = 0; h < NH; ++h, p += a.vdim)
+            if (h < nh) *p = o[h];
+        }
+      } else {
+#pragma unroll
+        for (int h = 0; h < NH; ++h)
+          if (h < nh && c < flash_column_limit(a, h0 + h)) flash_store_column<true>(a, r, h0 + h, c, o[h]);
+      }
     }
   }
   tc_fence_before();
@@ -309,10 +376,10 @@ __global__ void __launch_bounds__(kThreads, 1) flash_latent_kernel(const FlashAr
 bool latent_shape(const FlashArgs& a, int nh, LatentShape* sh, size_t* smem) {
   sh->panels = (a.dpad + 63) / 64;
   sh->mtiles = (a.vdim + 127) / 128;
-  if ((sh->mtiles + 2) * nh > kColumns) return false;
+  if ((2 * sh->mtiles + 2) * nh > kColumns) return false;
   sh->stage_bytes = (sh->panels > 2 * sh->mtiles ? sh->panels : 2 * sh->mtiles) * kPanel;
-  // behind the tiles: the queries, two buffers of weights in two pieces, and room for the rows that nobody reads
-  const size_t rest = (size_t)sh->panels * nh * 128 + (size_t)4 * nh * 128 + kPanel + 1024;
+  // behind the tiles: the queries, two buffers of weights in two pieces
+  const size_t rest = (size_t)sh->panels * nh * 128 + (size_t)4 * nh * 128 + 1024;
   const size_t fit = (224 * 1024 - rest) / sh->stage_bytes;
   if (rest > 224 * 1024 || fit < 2) return false;
   sh->stages = fit < kStagesMax ? (int)fit : kStagesMax;

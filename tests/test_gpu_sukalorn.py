@@ -32,6 +32,11 @@ MODELS = {
     "even": o.make_config(vocab=130, width=128, layers=[
         o.attention_layer(8, 2, 64, 64, 200, scale=0.1, cap=30.0, ff=256), o.latent_layer(6, 32, 16, 40, 136, 72, ff=None),
         o.attention_layer(6, 2, 48, 64, 77, scale=0.5, cap=5.0, ff=96), o.latent_layer(4, 128, 64, 128, 512, 96, scale=0.07, ff=80)]),
+    # head sizes of exactly 64, 128 and 256, many heads over a wide latent, more heads than a block of the decode kernel takes
+    "heads": o.make_config(vocab=100, width=160, layers=[
+        o.attention_layer(4, 2, 128, 128, 90, scale=0.1, cap=25.0, ff=72), o.latent_layer(24, 32, 16, 32, 512, 60, scale=0.15, ff=None),
+        o.attention_layer(2, 1, 256, 256, 64, scale=0.07, v_mix=False, ff=None), o.attention_layer(8, 1, 64, 64, 150, scale=0.2, v_mix=False, ff=96),
+        o.latent_layer(36, 16, 16, 24, 96, 48, scale=0.2, ff=None)]),
     # a latent beyond the tensor-core kernel's tiles
     "large": o.make_config(vocab=60, width=64, layers=[o.latent_layer(3, 12, 20, 16, 720, 48, ff=48)]),
 }
@@ -297,7 +302,7 @@ def test_far_positions_turn_by_their_angle(tmp_path, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", ["mixed", "many"])
+@pytest.mark.parametrize("name", ["mixed", "many", "even", "heads"])
 def test_unequal_requests_in_one_decoder(models, name, dtype):
     """Several sequences, prompts of unequal length, stepped together; ended sequences are used again."""
     path, cfg, w = models[name]
@@ -381,6 +386,36 @@ def test_flash_attention_with_windows_and_kept_positions(size, keep, vdim, dtype
     want = dab.forward(cfg, w, toks)
     got = np.concatenate([dec.extend(toks[:240], 0, list(range(240)))] + [dec.step(t, 240 + i)[None] for i, t in enumerate(toks[240:])])
     assert err(got, want) < TOL[dtype]
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("window,chunk,cap", [(50, 0, 0.0), (0, 64, 0.0), (70, 90, 4.0)])
+def test_latent_attention_with_the_other_masks_and_a_cap(tmp_path, monkeypatch, window, chunk, cap, dtype):
+    """The mechanisms are not tied to the design: latents behind a window, in chunks, with capped scores."""
+    import torchburn_b200 as tb
+    from torchburn_b200 import checkpoint, sukalorn
+
+    cfg = o.make_config(vocab=90, width=72, layers=[o.latent_layer(4, 64, 16, 32, 64, 48, scale=0.2, ff=88), o.latent_layer(4, 32, 16, 32, 128, 48, scale=0.2, ff=None)])
+    w = o.make_weights(cfg, 9)
+    n = 400
+    i, j = np.arange(n)[:, None], np.arange(n)[None, :]
+    mask = (j <= i) & (i - j < (window or n)) & (i // (chunk or n) == j // (chunk or n))
+    monkeypatch.setattr(o, "causal", lambda m: mask[:m, :m])
+    if cap:
+        plain = o.softmax
+        monkeypatch.setattr(o, "softmax", lambda s, m: plain(o.softcap(s, cap), m))
+    path = o.save_model(str(tmp_path), cfg, w)
+    t, specs = checkpoint.read_model_tensors(path), sukalorn.layer_specs(cfg)
+    for k, s in enumerate(specs):
+        s.tensors = sukalorn.layer_tensors(t, k, cfg["layers"][k], cfg["width"])
+        s.mask_window, s.mask_chunk, s.score_softcap = window, chunk, cap
+    dec = tb.LayeredDecoder(specs, t["embed"], t["final.norm"], embed_norm=t["embed.norm"], head=t["head"], hidden_size=72, vocab_size=90,
+                            norm_eps=1e-5, norm_offset=1.0, max_seq_len=n, dtype=dtype, prefill_rows=96)
+    toks = tokens_for(cfg, n, 5)
+    want = o.forward(cfg, w, toks)
+    got = np.concatenate([dec.extend(toks[:300], 0, list(range(300)))] + [dec.step(x, 300 + k)[None] for k, x in enumerate(toks[300:])])
+    assert err(got, want) < TOL[dtype]
+    assert fault() == 0
 
 
 def test_greedy_generation_and_schedulers(models):

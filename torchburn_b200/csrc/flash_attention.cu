@@ -548,43 +548,67 @@ __global__ void __launch_bounds__(kThreads) flash_decode_kernel(const FlashArgs 
 
 size_t decode_warp_bytes(const FlashArgs& a) { return (size_t)2 * kDecodeKeys * (a.dpad + a.vpad + 16) * 2; }
 
-// Merges the shares of a row's keys.  grid (heads, rows, columns / 128)
-__global__ void __launch_bounds__(128) flash_merge_kernel(const FlashArgs a, const int splits) {
-  __shared__ float s_w[kMaxSplits], s_red[4], s_sum[4];
-  const int tid = threadIdx.x, h = (int)blockIdx.x, r = (int)blockIdx.y, c = (int)blockIdx.z * 128 + tid;
+// Merges the shares of a row's keys.  A lane has four columns, each of W warps every W-th share; what they add up is
+// summed over the warps.  grid (heads, rows, columns / 128)
+template <int W>
+__global__ void __launch_bounds__(W * 32) flash_merge_kernel(const FlashArgs a, const int splits) {
+  constexpr int T = W * 32, AHEAD = 8;   // shares whose columns are requested before the weights are known
+  __shared__ float s_w[kMaxSplits], s_red[W], s_sum[W];
+  __shared__ float4 s_acc[W][32];
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, h = (int)blockIdx.x, r = (int)blockIdx.y, c = (int)blockIdx.z * 128 + lane * 4;
   grid_dep_launch();
   grid_dep_wait();
   const size_t stride = (size_t)a.r.rows * a.heads, at = (size_t)r * a.heads + h;
+  const float* p = a.parts + at * a.vdim + c;
+  auto load = [&](int z) {
+    const float* q = p + (size_t)z * stride * a.vdim;
+    if (a.vdim % 4 == 0) return c < a.vdim ? *reinterpret_cast<const float4*>(q) : make_float4(0.f, 0.f, 0.f, 0.f);
+    return make_float4(c < a.vdim ? q[0] : 0.f, c + 1 < a.vdim ? q[1] : 0.f, c + 2 < a.vdim ? q[2] : 0.f, c + 3 < a.vdim ? q[3] : 0.f);
+  };
+  float4 v[AHEAD];
+#pragma unroll
+  for (int i = 0; i < AHEAD; ++i)
+    if (warp + i * W < splits) v[i] = load(warp + i * W);
   float m = -INFINITY;
-  for (int z = tid; z < splits; z += 128) m = fmaxf(m, a.part_ml[z * stride + at].x);
+  for (int z = tid; z < splits; z += T) m = fmaxf(m, a.part_ml[z * stride + at].x);
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
-  if ((tid & 31) == 0) s_red[tid >> 5] = m;
+  if (lane == 0) s_red[warp] = m;
   __syncthreads();
-  m = fmaxf(fmaxf(s_red[0], s_red[1]), fmaxf(s_red[2], s_red[3]));
+#pragma unroll
+  for (int w = 0; w < W; ++w) m = fmaxf(m, s_red[w]);
   float l = 0.f;
-  for (int z = tid; z < splits; z += 128) {
-    const float2 p = a.part_ml[z * stride + at];
-    const float w = p.x == -INFINITY ? 0.f : exp2f(p.x - m);
+  for (int z = tid; z < splits; z += T) {
+    const float2 q = a.part_ml[z * stride + at];
+    const float w = q.x == -INFINITY ? 0.f : exp2f(q.x - m);   // a share that saw nothing left zeros
     s_w[z] = w;
-    l = fmaf(w, p.y, l);
+    l = fmaf(w, q.y, l);
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
-  if ((tid & 31) == 0) s_sum[tid >> 5] = l;
+  if (lane == 0) s_sum[warp] = l;
   __syncthreads();
-  l = (s_sum[0] + s_sum[1]) + (s_sum[2] + s_sum[3]);
-  if (c >= flash_column_limit(a, h)) return;
-  float v = 0.f;
-  if (c < a.vdim) {
-    const float* p = a.parts + at * a.vdim + c;
-#pragma unroll 16
-    for (int z = 0; z < splits; ++z) v = fmaf(s_w[z], p[(size_t)z * stride * a.vdim], v);   // a share that saw nothing left zeros
-    float f = l > 0.f ? 1.f / l : 0.f;
-    if (a.gate) f *= a.gate[at];
-    v *= f;
-  }
-  flash_store_column<true>(a, r, h, c, v);
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+  auto add = [&](float w, float4 x) { acc = make_float4(fmaf(w, x.x, acc.x), fmaf(w, x.y, acc.y), fmaf(w, x.z, acc.z), fmaf(w, x.w, acc.w)); };
+#pragma unroll
+  for (int i = 0; i < AHEAD; ++i)
+    if (warp + i * W < splits) add(s_w[warp + i * W], v[i]);
+  for (int z = warp + AHEAD * W; z < splits; z += W) add(s_w[z], load(z));
+  s_acc[warp][lane] = acc;
+  __syncthreads();
+  if (warp != 0) return;
+  l = 0.f;
+#pragma unroll
+  for (int w = 0; w < W; ++w) l += s_sum[w];
+  float f = l > 0.f ? 1.f / l : 0.f;
+  if (a.gate) f *= a.gate[at];
+  acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+  for (int w = 0; w < W; ++w) add(f, s_acc[w][lane]);
+  const float o[4] = {acc.x, acc.y, acc.z, acc.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+    if (c + i < flash_column_limit(a, h)) flash_store_column<true>(a, r, h, c + i, c + i < a.vdim ? o[i] : 0.f);
 }
 
 __device__ __forceinline__ float4 load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
@@ -728,7 +752,10 @@ tb_status launch_flash_attention(Precision p, const FlashArgs& a, cudaStream_t s
     if (splits == 1) return TB_OK;
     ++*launches;
     const int cols = a.out_per_head ? a.out.kp : a.out.kp - (a.heads - 1) * a.vdim;
-    return launch_kernel(flash_merge_kernel, dim3((unsigned)a.heads, (unsigned)rows, (unsigned)((cols + 127) / 128)), dim3(128), 0, st, a.pdl, 1, a, splits);
+    const dim3 grid((unsigned)a.heads, (unsigned)rows, (unsigned)((cols + 127) / 128));
+    if (splits <= 8) return launch_kernel(flash_merge_kernel<1>, grid, dim3(32), 0, st, a.pdl, 1, a, splits);
+    if (splits <= 32) return launch_kernel(flash_merge_kernel<4>, grid, dim3(128), 0, st, a.pdl, 1, a, splits);
+    return launch_kernel(flash_merge_kernel<8>, grid, dim3(256), 0, st, a.pdl, 1, a, splits);
   };
   if (flash_tc5_supported(a)) {
     int splits = 1;

@@ -37,8 +37,10 @@ MODELS = {
         o.attention_layer(4, 2, 128, 128, 90, scale=0.1, cap=25.0, ff=72), o.latent_layer(24, 32, 16, 32, 512, 60, scale=0.15, ff=None),
         o.attention_layer(2, 1, 256, 256, 64, scale=0.07, v_mix=False, ff=None), o.attention_layer(8, 1, 64, 64, 150, scale=0.2, v_mix=False, ff=96),
         o.latent_layer(36, 16, 16, 24, 96, 48, scale=0.2, ff=None)]),
-    # a latent beyond the tensor-core kernel's tiles
-    "large": o.make_config(vocab=60, width=64, layers=[o.latent_layer(3, 12, 20, 16, 720, 48, ff=48)]),
+    # latents and keys beyond the tensor-core kernels' tiles, and at the limit of their shared memory
+    "large": o.make_config(vocab=60, width=64, layers=[
+        o.latent_layer(3, 12, 20, 16, 720, 48, ff=48), o.attention_layer(2, 1, 240, 16, 60, scale=0.05, v_mix=False, ff=None),
+        o.latent_layer(4, 224, 32, 16, 64, 40, scale=0.06, ff=None), o.attention_layer(2, 2, 500, 300, 70, scale=0.05, v_mix=False, ff=40)]),
 }
 
 

@@ -35,6 +35,7 @@ constexpr int kKeys = 128;            // keys per tile
 constexpr int kPanel = 16384;         // 128 rows of 128 bytes
 constexpr int kThreads = 384;         // two softmax warpgroups, one warp for the MMAs, three for the copies
 constexpr int kLoaders = 96;
+constexpr size_t kSmemMax = 223 * 1024;   // what 227 KB leave beside the static part
 constexpr float kLog2E = 1.44269504f;
 constexpr float kGrow = 8.f;
 
@@ -249,55 +250,55 @@ __global__ void __launch_bounds__(kThreads, 1) flash_tc5_kernel(const FlashArgs 
         }
       }
     } else {
-    Rows ks, ks2, vs;
-    const int split_piece = a.key_rows ? a.key_cols >> 3 : kpieces, total = a.dim >> 3;
-    if (a.key_rows) {   // written out by position, the rest of a key in the cache
-      ks = Rows{static_cast<const __nv_bfloat16*>(a.key_rows) + (size_t)kv * a.key_cols, a.row_stride, begin - a.key_base, INT_MAX, 0};
-      vs = Rows{static_cast<const __nv_bfloat16*>(a.value_rows) + (size_t)kv * a.vdim, a.row_stride, begin - a.key_base, INT_MAX, 0};
-      ks2 = cache_rows(a, static_cast<const __nv_bfloat16*>(a.k_cache) + a.rest_col, 1, a.cache_row, 0, slot, begin);
-    } else {
-      ks = ks2 = cache_rows(a, a.k_cache, a.kv_heads, a.dpad, kv, slot, begin);
-      vs = cache_rows(a, a.v_cache, a.kv_heads, a.vpad, kv, slot, begin);
-    }
-    uint64_t* pending = nullptr;   // the load in flight in front of the one being issued
-    auto flush = [&] {
-      if (!pending) return;
-      asm volatile("cp.async.wait_all;" ::: "memory");
-      asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
-      mbar_arrive(pending);
-      pending = nullptr;
-    };
-    auto freed = [&](uint64_t* bar, int j) {   // the slot's last reader, tile j, is done
-      if (mbar_ready(bar, (uint32_t)j & 1u)) return true;
-      flush();
-      return mbar_wait(bar, (uint32_t)j & 1u, &s_abort, &g_flash_fault);
-    };
-    auto issued = [&](uint64_t* bar) {
-      asm volatile("cp.async.commit_group;" ::: "memory");
-      if (pending) {
-        asm volatile("cp.async.wait_group 1;" ::: "memory");
+      Rows ks, ks2, vs;
+      const int split_piece = a.key_rows ? a.key_cols >> 3 : kpieces, total = a.dim >> 3;
+      if (a.key_rows) {   // written out by position, the rest of a key in the cache
+        ks = Rows{static_cast<const __nv_bfloat16*>(a.key_rows) + (size_t)kv * a.key_cols, a.row_stride, begin - a.key_base, INT_MAX, 0};
+        vs = Rows{static_cast<const __nv_bfloat16*>(a.value_rows) + (size_t)kv * a.vdim, a.row_stride, begin - a.key_base, INT_MAX, 0};
+        ks2 = cache_rows(a, static_cast<const __nv_bfloat16*>(a.k_cache) + a.rest_col, 1, a.cache_row, 0, slot, begin);
+      } else {
+        ks = ks2 = cache_rows(a, a.k_cache, a.kv_heads, a.dpad, kv, slot, begin);
+        vs = cache_rows(a, a.v_cache, a.kv_heads, a.vpad, kv, slot, begin);
+      }
+      uint64_t* pending = nullptr;   // the load in flight in front of the one being issued
+      auto flush = [&] {
+        if (!pending) return;
+        asm volatile("cp.async.wait_all;" ::: "memory");
         asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
         mbar_arrive(pending);
+        pending = nullptr;
+      };
+      auto freed = [&](uint64_t* bar, int j) {   // the slot's last reader, tile j, is done
+        if (mbar_ready(bar, (uint32_t)j & 1u)) return true;
+        flush();
+        return mbar_wait(bar, (uint32_t)j & 1u, &s_abort, &g_flash_fault);
+      };
+      auto issued = [&](uint64_t* bar) {
+        asm volatile("cp.async.commit_group;" ::: "memory");
+        if (pending) {
+          asm volatile("cp.async.wait_group 1;" ::: "memory");
+          asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
+          mbar_arrive(pending);
+        }
+        pending = bar;
+      };
+      bool ok = true;
+      for (int j = 0; ok && j < nj[0]; ++j) {
+        for (int w = 0; ok && w < 2; ++w) {
+          if (j >= nj[w]) continue;
+          if (j > 0 && !(ok = freed(&s_ready[w], j - 1))) break;
+          load_tile(k_at + (uint32_t)(w * kbytes), ks, ks2, split_piece, a.key_rows ? total : kpieces, kpieces, (t0 + 2 * j + w) * kKeys, count, lt);
+          issued(&k_full[w]);
+        }
+        for (int w = 0; ok && w < 2; ++w) {
+          if (j >= nj[w]) continue;
+          if (j > 0 && !(ok = freed(&pv_done[w], j - 1))) break;
+          load_tile(v_at + (uint32_t)(w * vbytes), vs, vs, vpieces, a.key_rows ? a.vdim >> 3 : vpieces, vpieces, (t0 + 2 * j + w) * kKeys, count, lt);
+          issued(&v_full[w]);
+        }
       }
-      pending = bar;
-    };
-    bool ok = true;
-    for (int j = 0; ok && j < nj[0]; ++j) {
-      for (int w = 0; ok && w < 2; ++w) {
-        if (j >= nj[w]) continue;
-        if (j > 0 && !(ok = freed(&s_ready[w], j - 1))) break;
-        load_tile(k_at + (uint32_t)(w * kbytes), ks, ks2, split_piece, a.key_rows ? total : kpieces, kpieces, (t0 + 2 * j + w) * kKeys, count, lt);
-        issued(&k_full[w]);
-      }
-      for (int w = 0; ok && w < 2; ++w) {
-        if (j >= nj[w]) continue;
-        if (j > 0 && !(ok = freed(&pv_done[w], j - 1))) break;
-        load_tile(v_at + (uint32_t)(w * vbytes), vs, vs, vpieces, a.key_rows ? a.vdim >> 3 : vpieces, vpieces, (t0 + 2 * j + w) * kKeys, count, lt);
-        issued(&v_full[w]);
-      }
-    }
-    flush();
-    asm volatile("cp.async.wait_all;" ::: "memory");
+      flush();
+      asm volatile("cp.async.wait_all;" ::: "memory");
     }
   } else if (warp == 8) {
     if (lane == 0) {   // ---- MMA issue ----
@@ -525,7 +526,7 @@ int flash_fault_flag() {
 
 bool flash_tc5_fits(int dpad, int vdim) {
   const int vpad = (int)pad_to(vdim, 16);
-  return vdim % 8 == 0 && vpad <= 128 && dpad <= 768 && tc5_bytes(dpad, vpad) <= 226 * 1024;
+  return vdim % 8 == 0 && vpad <= 128 && dpad <= 768 && tc5_bytes(dpad, vpad) <= kSmemMax;
 }
 
 bool flash_tc5_supported(const FlashArgs& a) {
